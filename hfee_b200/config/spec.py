@@ -119,6 +119,8 @@ class ModelSpec:
     eos_token_ids: Tuple[int, ...] = ()
     bos_token_id: Optional[int] = None
     max_positions: int = 2048
+    # number of residual streams the blocks pass on (a ResidualStreams); None: the one residual stream itself
+    streams: Optional[int] = None
     # name patterns (fnmatch) of tensors that files of this architecture may carry without any part
     # asking for them; they are skipped with a warning instead of failing the load
     ignorable: Tuple[str, ...] = ()
@@ -127,6 +129,16 @@ class ModelSpec:
     def sequential(n_layers: int) -> Tuple[RunSpec, ...]:
         """Every layer once, in order, each with a cache of its own."""
         return tuple(RunSpec(layer=i, cache=i) for i in range(n_layers))
+
+    @staticmethod
+    def looped(n_layers: int, start: int, stop: int, times: int, adds_embedding: bool = False) -> Tuple[RunSpec, ...]:
+        """Every layer in order, layers ``start`` .. ``stop - 1`` ``times`` times in a row, each run with a cache of its
+        own; with ``adds_embedding`` the first run of every pass but the first takes the embedding's output on top."""
+        runs = [(i, False) for i in range(start)]
+        for r in range(times):
+            runs += [(i, adds_embedding and r > 0 and i == start) for i in range(start, stop)]
+        runs += [(i, False) for i in range(stop, n_layers)]
+        return tuple(RunSpec(layer=i, cache=j, adds_embedding=add) for j, (i, add) in enumerate(runs))
 
 
 def check_schedule(layers: Sequence[LayerSpec], schedule: Sequence[RunSpec]) -> None:

@@ -1,0 +1,534 @@
+// The gated delta rule with a decay per key channel.  Per request and head, with S [dim, vdim] float32 carried from
+// step to step:
+//
+//     S <- diag(g_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t
+//
+// q and k are first made unit vectors (x / sqrt(sum x^2 + 1e-6); q also times dim^-1/2), beta_t = sigmoid(b_t) and
+// g_t = exp(-exp(A_log) softplus(z_t + dt_bias)) per key channel, all float32.  `qk_heads` query/key heads serve `heads`
+// value heads; the decays belong to the value head.
+//
+// hfee_channel_delta, a step of single tokens: the recurrence itself, a block per (32 state columns, head, request).
+//
+// A step with longer portions: tiles of CD_TILE tokens.  With G_t the product of the decays of the tile's tokens up to t
+// (per channel), S_0 the state in front of the tile and `*` element by element over key channels,
+//
+//     u_t = beta_t (v_t - S_0^T (G_t * k_t) - sum_{j<t} A[t][j] u_j)       A[t][j] = k_t . (G_t / G_j * k_j)
+//     o_t = S_0^T (G_t * q_t) + sum_{j<=t} B[t][j] u_j                      B[t][j] = q_t . (G_t / G_j * k_j)
+//     S   = diag(G_last) S_0 + sum_j (G_last / G_j * k_j) u_j^T
+//
+// The first line is a triangular system with the same matrix for every column, so `channel_delta_prepare` solves it once
+// per tile and head for the right-hand sides that do not involve the state: u = U - W S_0 and o = O + P S_0 with
+//
+//     (I + diag(beta) A) [W | U] = diag(beta) [G * k | v]      P = G * q - B W      O = B U
+//
+// for all tiles at once, and `channel_delta_walk` goes through a request's tiles with three small products per tile.
+// The ratios G_t / G_j are running products of decays from j on (never a quotient of two products, which could be 0 / 0),
+// so strong decays underflow to zero and nothing overflows.  The result depends on how a prompt was cut only through the
+// order of float32 sums.
+//
+// A tile's part of the workspace (its place: (first token of the tile) / 16 + request, different for any two tiles of a
+// step), per head, rows of DP = dim rounded up to 32 floats:  W [16] | P [16] | Khat [16] (= G_last / G_j * k_j) | G_last,
+// and behind all of them, per head and group of CW_COLS columns, U [16][CW_COLS] | O [16][CW_COLS].
+#include "tcgen05.cuh"
+
+namespace {
+
+constexpr int CD_TILE = 16;
+constexpr int CD_MAX_DIM = 256;
+constexpr int CD_THREADS = 128;
+constexpr int CD_COLS = 32;                  // state columns per block of the one-token kernel
+
+struct ChannelDeltaArgs {
+  long long ld_qkv, ld_b, ld_z, ld_out;
+  int q_off, k_off, v_off;
+  int heads, qk_heads, dim, vdim;
+  int write_state;
+};
+
+__device__ __forceinline__ float softplus_cd(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+
+// ---------------------------------------------------------------------------------------------------------------
+// One token per request.  A thread keeps RPT rows of VEC neighbouring columns in registers; 32 / VEC threads side by
+// side make a row of CD_COLS columns.
+template <typename T, int VEC, int RPT>
+__global__ void __launch_bounds__(CD_THREADS)
+channel_delta_token_kernel(const T* __restrict__ qkv, const T* __restrict__ b, const float* __restrict__ z,
+                           const float* __restrict__ a_log, const float* __restrict__ dt_bias, float* __restrict__ state,
+                           const int* __restrict__ cu_tokens, const int* __restrict__ slots, float* __restrict__ out,
+                           ChannelDeltaArgs p) {
+  constexpr int LANES = CD_COLS / VEC, RG = CD_THREADS / LANES;        // threads of a row, rows taken side by side
+  __shared__ float k_s[CD_MAX_DIM], q_s[CD_MAX_DIM], g_s[CD_MAX_DIM];
+  __shared__ float sums_s[3][CD_THREADS / 32];
+  __shared__ float part_s[2][CD_THREADS / 32][CD_COLS];
+  const int h = blockIdx.y, req = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int cl = tid % LANES, rg = tid / LANES;
+  const int col = blockIdx.x * CD_COLS + cl * VEC;
+  const int dim = p.dim, vdim = p.vdim, kh = h / (p.heads / p.qk_heads);
+  const int slot = slots[req], tok = cu_tokens[req];
+  const float rate = expf(a_log[h]);
+  pdl_wait();
+  pdl_launch_dependents();
+  float* sp = state + ((long long)slot * p.heads + h) * (long long)dim * vdim;
+  float S[RPT][VEC];
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int d = rg + RG * i;
+    const bool in = d < dim && col < vdim;
+    if constexpr (VEC == 4) {
+      const float4 t = in ? *reinterpret_cast<const float4*>(sp + (long long)d * vdim + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[i][0] = t.x; S[i][1] = t.y; S[i][2] = t.z; S[i][3] = t.w;
+    } else {
+      S[i][0] = in ? sp[(long long)d * vdim + col] : 0.f;
+    }
+  }
+  const T* row = qkv + (long long)tok * p.ld_qkv;
+  float sk = 0.f, sq = 0.f, kq = 0.f;
+  for (int d = tid; d < dim; d += CD_THREADS) {
+    const float kv = to_f32<T>(row[p.k_off + (long long)kh * dim + d]), qv = to_f32<T>(row[p.q_off + (long long)kh * dim + d]);
+    const float zz = z[(long long)tok * p.ld_z + (long long)h * dim + d] + dt_bias[(long long)h * dim + d];
+    k_s[d] = kv;
+    q_s[d] = qv;
+    g_s[d] = expf(-rate * softplus_cd(zz));
+    sk = fmaf(kv, kv, sk);
+    sq = fmaf(qv, qv, sq);
+    kq = fmaf(kv, qv, kq);
+  }
+  sk = warp_sum(sk); sq = warp_sum(sq); kq = warp_sum(kq);
+  if (lane == 0) { sums_s[0][warp] = sk; sums_s[1][warp] = sq; sums_s[2][warp] = kq; }
+  __syncthreads();
+  sk = sq = kq = 0.f;
+#pragma unroll
+  for (int w = 0; w < CD_THREADS / 32; ++w) { sk += sums_s[0][w]; sq += sums_s[1][w]; kq += sums_s[2][w]; }
+  const float k_scale = 1.0f / sqrtf(sk + 1e-6f), q_scale = (1.0f / sqrtf((float)dim)) / sqrtf(sq + 1e-6f);
+  kq *= k_scale * q_scale;
+  float pk[VEC], pq[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) pk[e] = pq[e] = 0.f;
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int d = rg + RG * i;
+    const float g = d < dim ? g_s[d] : 0.f, kk = d < dim ? k_s[d] : 0.f, qq = d < dim ? q_s[d] : 0.f;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      S[i][e] *= g;
+      pk[e] = fmaf(S[i][e], kk, pk[e]);
+      pq[e] = fmaf(S[i][e], qq, pq[e]);
+    }
+  }
+#pragma unroll
+  for (int o = 16; o >= LANES; o >>= 1)
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      pk[e] += __shfl_xor_sync(0xffffffffu, pk[e], o);
+      pq[e] += __shfl_xor_sync(0xffffffffu, pq[e], o);
+    }
+  if (lane < LANES)
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      part_s[0][warp][cl * VEC + e] = pk[e];
+      part_s[1][warp][cl * VEC + e] = pq[e];
+    }
+  __syncthreads();
+  const float beta = 1.f / (1.f + expf(-to_f32<T>(b[(long long)tok * p.ld_b + h])));
+  float u[VEC], o[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) {
+    float sum_k = 0.f, sum_q = 0.f;
+#pragma unroll
+    for (int w = 0; w < CD_THREADS / 32; ++w) { sum_k += part_s[0][w][cl * VEC + e]; sum_q += part_s[1][w][cl * VEC + e]; }
+    const float v = col + e < vdim ? to_f32<T>(row[p.v_off + (long long)h * vdim + col + e]) : 0.f;
+    u[e] = beta * (v - sum_k * k_scale);
+    o[e] = fmaf(kq, u[e], sum_q * q_scale);
+  }
+  if (rg == 0)
+#pragma unroll
+    for (int e = 0; e < VEC; ++e)
+      if (col + e < vdim) out[(long long)tok * p.ld_out + (long long)h * vdim + col + e] = o[e];
+  if (!p.write_state) return;
+#pragma unroll
+  for (int i = 0; i < RPT; ++i) {
+    const int d = rg + RG * i;
+    if (d >= dim || col >= vdim) continue;
+    const float kk = k_s[d] * k_scale;
+    if constexpr (VEC == 4) {
+      *reinterpret_cast<float4*>(sp + (long long)d * vdim + col) =
+          make_float4(fmaf(kk, u[0], S[i][0]), fmaf(kk, u[1], S[i][1]), fmaf(kk, u[2], S[i][2]), fmaf(kk, u[3], S[i][3]));
+    } else {
+      sp[(long long)d * vdim + col] = fmaf(kk, u[0], S[i][0]);
+    }
+  }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int CW_COLS = 16;                                         // state columns per block of the walk
+constexpr int CW_WARPS = 4;                                         // each takes four of them
+constexpr int CW_STAGES = 3;
+
+__host__ __device__ inline int cd_pad(int dim) { return (dim + 31) / 32 * 32; }
+__host__ __device__ inline long long cd_head_floats(int dim) { return (3ll * CD_TILE + 1) * cd_pad(dim); }
+__host__ __device__ inline int cd_col_tiles(int vdim) { return (vdim + CW_COLS - 1) / CW_COLS; }
+constexpr int CD_UO = 2 * CD_TILE * CW_COLS;
+
+// NI: float4 per lane of a row (a row of DP = 32 * NI floats shared by 8 lanes)
+template <typename T, int NI>
+__global__ void __launch_bounds__(CD_THREADS)
+channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b, const float* __restrict__ z,
+                             const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+                             const int* __restrict__ cu_tokens, float* __restrict__ ws_head, float* __restrict__ ws_uo,
+                             ChannelDeltaArgs p) {
+  constexpr int DP = 32 * NI;
+  extern __shared__ __align__(128) float smem[];
+  float* k_s = smem;                         // [16][DP]
+  float* q_s = k_s + CD_TILE * DP;
+  float* g_s = q_s + CD_TILE * DP;
+  __shared__ __align__(16) float A_s[CD_TILE][CD_TILE], B_s[CD_TILE][CD_TILE];
+  __shared__ float beta_s[CD_TILE];
+  const int req = blockIdx.z, h = blockIdx.y, tile0 = blockIdx.x * CD_TILE;
+  const int begin = cu_tokens[req], count = cu_tokens[req + 1] - begin;
+  pdl_wait();
+  pdl_launch_dependents();
+  if (tile0 >= count) return;
+  const int tt = min(CD_TILE, count - tile0);
+  const long long tok0 = begin + tile0, place = tok0 / CD_TILE + req;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dim = p.dim, vdim = p.vdim, kh = h / (p.heads / p.qk_heads);
+  const float rate = expf(a_log[h]);
+  for (int e = tid; e < CD_TILE * DP; e += CD_THREADS) {
+    const int t = e / DP, d = e - t * DP;
+    const bool in = t < tt && d < dim;
+    float kv = 0.f, qv = 0.f, g = 1.f;       // a missing token is the identity: no write, no decay
+    if (in) {
+      const T* row = qkv + (tok0 + t) * p.ld_qkv + (long long)kh * dim + d;
+      kv = to_f32<T>(row[p.k_off]);
+      qv = to_f32<T>(row[p.q_off]);
+      g = expf(-rate * softplus_cd(z[(tok0 + t) * p.ld_z + (long long)h * dim + d] + dt_bias[(long long)h * dim + d]));
+    }
+    k_s[e] = kv;
+    q_s[e] = qv;
+    g_s[e] = g;
+  }
+  if (tid < CD_TILE) beta_s[tid] = tid < tt ? 1.f / (1.f + expf(-to_f32<T>(b[(tok0 + tid) * p.ld_b + h]))) : 0.f;
+  __syncthreads();
+  const float q_unit = 1.0f / sqrtf((float)dim);
+  for (int vid = warp; vid < 2 * tt; vid += CD_THREADS / 32) {
+    float* vec = vid < tt ? q_s + vid * DP : k_s + (vid - tt) * DP;
+    float x[NI], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) { x[i] = vec[lane + 32 * i]; ss = fmaf(x[i], x[i], ss); }
+    const float scale = (vid < tt ? q_unit : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) vec[lane + 32 * i] = x[i] * scale;
+  }
+  __syncthreads();
+  {
+    // the tables: eight lanes per row j, each with its share of the channels of G_t / G_j * k_j as t runs on from j
+    const int j = tid >> 3, sl = tid & 7;
+    const float4* k4 = reinterpret_cast<const float4*>(k_s);
+    const float4* q4 = reinterpret_cast<const float4*>(q_s);
+    const float4* g4 = reinterpret_cast<const float4*>(g_s);
+    float4 w[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) w[i] = k4[j * (DP / 4) + sl + 8 * i];
+    const int j_first = (warp * 4);            // smallest j of this warp: earlier tokens concern none of its rows
+    for (int t = j_first; t < tt; ++t) {
+      float a = 0.f, c = 0.f;
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int at = t * (DP / 4) + sl + 8 * i;
+        const float4 kk = k4[at], qq = q4[at];
+        if (t > j) {
+          const float4 g = g4[at];
+          w[i].x *= g.x; w[i].y *= g.y; w[i].z *= g.z; w[i].w *= g.w;
+        }
+        a = fmaf(w[i].x, kk.x, a); a = fmaf(w[i].y, kk.y, a); a = fmaf(w[i].z, kk.z, a); a = fmaf(w[i].w, kk.w, a);
+        c = fmaf(w[i].x, qq.x, c); c = fmaf(w[i].y, qq.y, c); c = fmaf(w[i].z, qq.z, c); c = fmaf(w[i].w, qq.w, c);
+      }
+#pragma unroll
+      for (int o = 4; o >= 1; o >>= 1) {
+        a += __shfl_xor_sync(0xffffffffu, a, o);
+        c += __shfl_xor_sync(0xffffffffu, c, o);
+      }
+      if (sl == 0) {
+        A_s[t][j] = t > j ? a : 0.f;
+        B_s[t][j] = t >= j ? c : 0.f;
+      }
+    }
+    if (sl == 0) {                             // what the loop did not reach
+      for (int t = 0; t < CD_TILE; ++t)
+        if (t < j_first || t >= tt) A_s[t][j] = B_s[t][j] = 0.f;
+    }
+  }
+  __syncthreads();
+  float* wh = ws_head + (place * p.heads + h) * cd_head_floats(dim);
+  const int tiles = cd_col_tiles(vdim);
+  float* wuo = ws_uo + (place * p.heads + h) * (long long)tiles * CD_UO;
+  // columns of the triangular system: the key channels, then the value columns
+  for (int c = tid; c < DP + tiles * CW_COLS; c += CD_THREADS) {
+    float x[CD_TILE];
+    if (c < DP) {
+      float run = 1.f;
+#pragma unroll
+      for (int t = 0; t < CD_TILE; ++t) {
+        run *= g_s[t * DP + c];
+        float r = run * k_s[t * DP + c];
+#pragma unroll
+        for (int j = 0; j < t; ++j) r = fmaf(-A_s[t][j], x[j], r);
+        x[t] = beta_s[t] * r;
+        wh[t * DP + c] = x[t];
+        float pr = run * q_s[t * DP + c];
+#pragma unroll
+        for (int j = 0; j <= t; ++j) pr = fmaf(-B_s[t][j], x[j], pr);
+        wh[(CD_TILE + t) * DP + c] = pr;
+      }
+      wh[3 * CD_TILE * DP + c] = run;
+      float after = 1.f;
+#pragma unroll
+      for (int t = CD_TILE - 1; t >= 0; --t) {
+        wh[(2 * CD_TILE + t) * DP + c] = after * k_s[t * DP + c];
+        after *= g_s[t * DP + c];
+      }
+    } else {
+      const int col = c - DP;
+      float* dst = wuo + (col / CW_COLS) * CD_UO + col % CW_COLS;
+      float v[CD_TILE];
+#pragma unroll
+      for (int t = 0; t < CD_TILE; ++t)
+        v[t] = (t < tt && col < vdim) ? to_f32<T>(qkv[(tok0 + t) * p.ld_qkv + p.v_off + (long long)h * vdim + col]) : 0.f;
+#pragma unroll
+      for (int t = 0; t < CD_TILE; ++t) {
+        float r = v[t];
+#pragma unroll
+        for (int j = 0; j < t; ++j) r = fmaf(-A_s[t][j], x[j], r);
+        x[t] = beta_s[t] * r;
+        dst[t * CW_COLS] = x[t];
+        float o = 0.f;
+#pragma unroll
+        for (int j = 0; j <= t; ++j) o = fmaf(B_s[t][j], x[j], o);
+        dst[(CD_TILE + t) * CW_COLS] = o;
+      }
+    }
+  }
+}
+
+// A block walks the tiles of one request and head for CW_COLS state columns; the tiles' parts of the workspace come in
+// through a ring of bulk copies.  A warp owns four columns; eight lanes share a column, lane dg of them holding the rows
+// 4 dg + 32 i + (0..3).  Rows of W and P times the lanes' rows of S are summed over the eight lanes so that lane dg ends
+// with those of the tokens dg and dg + 8; u is then handed around token by token for the update.
+template <int NI>
+__global__ void __launch_bounds__(CW_WARPS * 32)
+channel_delta_walk_kernel(const float* __restrict__ ws_head, const float* __restrict__ ws_uo, float* __restrict__ state,
+                          const int* __restrict__ cu_tokens, const int* __restrict__ slots, float* __restrict__ out,
+                          int* __restrict__ status, ChannelDeltaArgs p) {
+  constexpr int DP = 32 * NI;
+  constexpr int HEAD = (3 * CD_TILE + 1) * DP, STAGE = HEAD + CD_UO;      // floats of a tile
+  extern __shared__ __align__(128) float smem[];                          // [CW_STAGES][STAGE]
+  __shared__ __align__(8) uint64_t full[CW_STAGES];
+  __shared__ int abort_flag;
+  const int req = blockIdx.z, h = blockIdx.y, tile_col = blockIdx.x;
+  const int begin = cu_tokens[req], count = cu_tokens[req + 1] - begin;
+  const int slot = slots[req];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dg = lane & 7, cg = lane >> 3;
+  const int in_tile = warp * 4 + cg, col = tile_col * CW_COLS + in_tile;
+  const int dim = p.dim, vdim = p.vdim, tiles = (count + CD_TILE - 1) / CD_TILE;
+  if (tid == 0) {
+    abort_flag = 0;
+    for (int s = 0; s < CW_STAGES; ++s) tc::mbar_init(&full[s], 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  __syncthreads();
+  pdl_wait();
+  pdl_launch_dependents();
+  if (count <= 0) return;
+  const int col_tiles = cd_col_tiles(vdim);
+  auto bulk = [](float* dst, const float* src, uint32_t bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                 ::"r"(tc::smem_u32(dst)), "l"(src), "r"(bytes), "r"(tc::smem_u32(bar)) : "memory");
+  };
+  auto fetch = [&](int tile) {
+    const int s = tile % CW_STAGES;
+    const long long place = (begin + tile * CD_TILE) / CD_TILE + req, at = place * p.heads + h;
+    tc::mbar_expect_tx(&full[s], STAGE * 4u);
+    bulk(smem + s * STAGE, ws_head + at * HEAD, HEAD * 4u, &full[s]);
+    bulk(smem + s * STAGE + HEAD, ws_uo + (at * col_tiles + tile_col) * CD_UO, CD_UO * 4u, &full[s]);
+  };
+  if (tid == 0)
+    for (int t = 0; t < CW_STAGES - 1 && t < tiles; ++t) fetch(t);
+  float* sp = state + ((long long)slot * p.heads + h) * (long long)dim * vdim + col;
+  float S[NI][4];
+#pragma unroll
+  for (int i = 0; i < NI; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = 32 * i + 4 * dg + e;
+      S[i][e] = (d < dim && col < vdim) ? sp[(long long)d * vdim] : 0.f;
+    }
+  bool ok = true;
+  for (int tile = 0; tile < tiles; ++tile) {
+    const int s = tile % CW_STAGES;
+    ok = tc::mbar_wait(&full[s], (tile / CW_STAGES) & 1u, &abort_flag);
+    if (!__syncthreads_and(ok)) { ok = false; break; }        // also: every warp is done with the tile before
+    if (tid == 0 && tile + CW_STAGES - 1 < tiles) fetch(tile + CW_STAGES - 1);
+    const float4* M4 = reinterpret_cast<const float4*>(smem + s * STAGE);
+    const float* uo = smem + s * STAGE + HEAD;
+    float x[4];                                               // tokens dg, dg + 8 of W S and of P S
+#pragma unroll
+    for (int grp = 0; grp < 4; ++grp) {
+      float val[8];
+#pragma unroll
+      for (int r = 0; r < 8; ++r) {
+        float a = 0.f, c = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const float4 m = M4[(grp * 8 + r) * (DP / 4) + dg + 8 * i];
+          a = fmaf(m.x, S[i][0], a); c = fmaf(m.y, S[i][1], c);
+          a = fmaf(m.z, S[i][2], a); c = fmaf(m.w, S[i][3], c);
+        }
+        val[r] = a + c;
+      }
+#pragma unroll
+      for (int off = 4; off >= 1; off >>= 1) {
+        const bool upper = (lane & off) != 0;
+#pragma unroll
+        for (int i = 0; i < off; ++i) {
+          const float send = upper ? val[i] : val[i + off], keep = upper ? val[i + off] : val[i];
+          val[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+        }
+      }
+      x[grp] = val[0];
+    }
+    const float u0 = uo[dg * CW_COLS + in_tile] - x[0], u1 = uo[(dg + 8) * CW_COLS + in_tile] - x[1];
+    const float o0 = uo[(CD_TILE + dg) * CW_COLS + in_tile] + x[2], o1 = uo[(CD_TILE + dg + 8) * CW_COLS + in_tile] + x[3];
+    const int tt = min(CD_TILE, count - tile * CD_TILE);
+    float* orow = out + (long long)(begin + tile * CD_TILE) * p.ld_out + (long long)h * vdim + col;
+    if (col < vdim && dg < tt) orow[(long long)dg * p.ld_out] = o0;
+    if (col < vdim && dg + 8 < tt) orow[(long long)(dg + 8) * p.ld_out] = o1;
+    const float4* K4 = M4 + 2 * CD_TILE * (DP / 4);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const float4 g = K4[CD_TILE * (DP / 4) + dg + 8 * i];
+      S[i][0] *= g.x; S[i][1] *= g.y; S[i][2] *= g.z; S[i][3] *= g.w;
+    }
+#pragma unroll
+    for (int j = 0; j < CD_TILE; ++j) {
+      const float u = __shfl_sync(0xffffffffu, j < 8 ? u0 : u1, (lane & 24) + (j & 7));
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const float4 kk = K4[j * (DP / 4) + dg + 8 * i];
+        S[i][0] = fmaf(kk.x, u, S[i][0]); S[i][1] = fmaf(kk.y, u, S[i][1]);
+        S[i][2] = fmaf(kk.z, u, S[i][2]); S[i][3] = fmaf(kk.w, u, S[i][3]);
+      }
+    }
+  }
+  if (!ok) {                                                  // a copy never arrived: say so; copies in flight end on their own barriers
+    if (tid == 0) *status = 1;
+    for (int s = 0; s < CW_STAGES; ++s)
+      for (int i = 0; i < 64; ++i)
+        if (tc::mbar_try(&full[s], 0) || tc::mbar_try(&full[s], 1)) break;
+    return;
+  }
+  if (p.write_state)
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = 32 * i + 4 * dg + e;
+        if (d < dim && col < vdim) sp[(long long)d * vdim] = S[i][e];
+      }
+}
+
+template <typename T, int VEC, int RPT>
+int launch_token_r(const void* qkv, const void* b, const float* z, const float* a_log, const float* dt_bias, float* state,
+                   const int* cu_tokens, const int* slots, float* out, const ChannelDeltaArgs& p, int requests, cudaStream_t stream) {
+  hfee_launch(channel_delta_token_kernel<T, VEC, RPT>, dim3((unsigned)((p.vdim + CD_COLS - 1) / CD_COLS), (unsigned)p.heads, (unsigned)requests),
+              dim3(CD_THREADS), 0, stream, (const T*)qkv, (const T*)b, z, a_log, dt_bias, state, cu_tokens, slots, out, p);
+  return hfee_check_launch("channel_delta_token");
+}
+
+template <typename T>
+int launch_token(const void* qkv, const void* b, const float* z, const float* a_log, const float* dt_bias, float* state,
+                 const int* cu_tokens, const int* slots, float* out, const ChannelDeltaArgs& p, int requests, cudaStream_t stream) {
+#define HFEE_CD(V, R) return launch_token_r<T, V, R>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, stream)
+  if (p.vdim % 4 == 0 && (uintptr_t)state % 16 == 0) {       // 16 rows side by side
+    if (p.dim <= 32) HFEE_CD(4, 2);
+    if (p.dim <= 64) HFEE_CD(4, 4);
+    if (p.dim <= 128) HFEE_CD(4, 8);
+    HFEE_CD(4, 16);
+  }
+  if (p.dim <= 64) HFEE_CD(1, 16);                           // 4 rows side by side
+  HFEE_CD(1, 64);
+#undef HFEE_CD
+}
+
+template <typename T, int NI>
+int launch_tiles_n(const void* qkv, const void* b, const float* z, const float* a_log, const float* dt_bias, float* state,
+                   const int* cu_tokens, const int* slots, float* out, const ChannelDeltaArgs& p, int requests, int max_new,
+                   float* ws_head, float* ws_uo, int* status, cudaStream_t stream) {
+  const size_t prep = (size_t)3 * CD_TILE * 32 * NI * sizeof(float);
+  const size_t walk = (size_t)CW_STAGES * ((3 * CD_TILE + 1) * 32 * NI + CD_UO) * sizeof(float);
+  if (prep > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(channel_delta_prepare_kernel<T, NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep);
+    if (e != cudaSuccess) return hfee_fail(HFEE_ERR_CUDA, "channel_delta_prepare: %s", cudaGetErrorString(e));
+  }
+  if (walk > 40 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk);
+    if (e != cudaSuccess) return hfee_fail(HFEE_ERR_CUDA, "channel_delta_walk: %s", cudaGetErrorString(e));
+  }
+  hfee_launch(channel_delta_prepare_kernel<T, NI>, dim3((unsigned)((max_new + CD_TILE - 1) / CD_TILE), (unsigned)p.heads, (unsigned)requests),
+              dim3(CD_THREADS), prep, stream, (const T*)qkv, (const T*)b, z, a_log, dt_bias, cu_tokens, ws_head, ws_uo, p);
+  const int rc = hfee_check_launch("channel_delta_prepare");
+  if (rc != HFEE_OK) return rc;
+  hfee_launch(channel_delta_walk_kernel<NI>, dim3((unsigned)cd_col_tiles(p.vdim), (unsigned)p.heads, (unsigned)requests),
+              dim3(CW_WARPS * 32), walk, stream, ws_head, ws_uo, state, cu_tokens, slots, out, status, p);
+  return hfee_check_launch("channel_delta_walk");
+}
+
+template <typename T>
+int launch_tiles(const void* qkv, const void* b, const float* z, const float* a_log, const float* dt_bias, float* state,
+                 const int* cu_tokens, const int* slots, float* out, const ChannelDeltaArgs& p, int requests, int max_new,
+                 float* ws_head, float* ws_uo, int* status, cudaStream_t stream) {
+#define HFEE_CT(N) case N: return launch_tiles_n<T, N>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, max_new, ws_head, ws_uo, status, stream)
+  switch (cd_pad(p.dim) / 32) {
+    HFEE_CT(1); HFEE_CT(2); HFEE_CT(3); HFEE_CT(4); HFEE_CT(5); HFEE_CT(6); HFEE_CT(7);
+    default: return launch_tiles_n<T, 8>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, max_new, ws_head, ws_uo, status, stream);
+  }
+#undef HFEE_CT
+}
+
+long long cd_places(int requests, int n_tokens) { return n_tokens / CD_TILE + requests + 1; }
+
+}  // namespace
+
+// Floats of workspace for a step of n_tokens tokens in `requests` requests that has a portion of several tokens.
+HFEE_API long long hfee_channel_delta_workspace(int requests, int n_tokens, int heads, int dim, int vdim) {
+  return cd_places(requests, n_tokens) * heads * (cd_head_floats(dim) + (long long)cd_col_tiles(vdim) * CD_UO);
+}
+
+// qkv rows (dtype): head g's query at q_off + g * dim, its key at k_off + g * dim (g < qk_heads; head h of `heads` uses
+// g = h / (heads / qk_heads)), head h's value at v_off + h * vdim.  b rows (dtype): one number per head.  z rows
+// (float32): heads * dim.  dt_bias: [heads * dim].  state: [slots, heads, dim, vdim] float32.  out: float32 [n, heads *
+// vdim].  max_new: the longest portion of the step; 1 takes the one-token kernel, more takes the workspace.
+HFEE_API int hfee_channel_delta(const void* qkv, long long ld_qkv, int q_off, int k_off, int v_off, const void* b, long long ld_b,
+                                const float* z, long long ld_z, int dtype, const float* a_log, const float* dt_bias, float* state,
+                                const int* cu_tokens, const int* slots, float* out, long long ld_out, int requests, int heads,
+                                int qk_heads, int dim, int vdim, int write_state, int n_tokens, int max_new, float* workspace,
+                                long long workspace_floats, int* status, cudaStream_t stream) {
+  if (requests == 0 || max_new == 0) return HFEE_OK;
+  HFEE_REQUIRE(heads > 0 && qk_heads > 0 && heads % qk_heads == 0, "channel_delta: heads %d must be a multiple of %d", heads, qk_heads);
+  HFEE_REQUIRE(dim > 0 && dim <= CD_MAX_DIM && vdim > 0, "channel_delta: key size %d is outside 1..%d", dim, CD_MAX_DIM);
+  HFEE_REQUIRE(requests <= 65535 && heads <= 65535, "channel_delta: too many requests or heads");
+  HFEE_REQUIRE(dtype == HFEE_F32 || dtype == HFEE_BF16, "channel_delta: unknown dtype %d", dtype);
+  const ChannelDeltaArgs p{ld_qkv, ld_b, ld_z, ld_out, q_off, k_off, v_off, heads, qk_heads, dim, vdim, write_state};
+  if (max_new == 1) {
+    if (dtype == HFEE_F32) return launch_token<float>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, stream);
+    return launch_token<__nv_bfloat16>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, stream);
+  }
+  HFEE_REQUIRE(workspace != nullptr && workspace_floats >= hfee_channel_delta_workspace(requests, n_tokens, heads, dim, vdim) &&
+               (uintptr_t)workspace % 16 == 0 && status != nullptr, "channel_delta: the workspace is missing, too small or not 16-byte aligned");
+  float* ws_head = workspace;
+  float* ws_uo = workspace + cd_places(requests, n_tokens) * heads * cd_head_floats(dim);
+  if (dtype == HFEE_F32)
+    return launch_tiles<float>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, max_new, ws_head, ws_uo, status, stream);
+  return launch_tiles<__nv_bfloat16>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, max_new, ws_head, ws_uo, status, stream);
+}

@@ -33,6 +33,7 @@ struct LatentParams {
   int rows_per_token, tokens_per_tile;
   float scale_log2;
   int window;
+  const float* sink;               // per head, or null: one more term exp(sink[h]) of the softmax's denominator
 };
 
 __device__ __forceinline__ void la_cp_async16(void* smem, const void* gmem, bool valid) {
@@ -254,7 +255,12 @@ latent_attention_kernel(LatentParams p) {
       if (rowpos[row] < 0) continue;
       const int t = row / p.rows_per_token, h = head0 + row % p.rows_per_token;
       const float l = l_s[row];
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.sink != nullptr) {                 // joins the row's sum once; against the larger of the two exponents
+        const float s2 = p.sink[h] * 1.4426950408889634f, m = m_s[row], top = fmaxf(m, s2);
+        const float shrink = la_exp2(m - top);
+        inv = shrink / fmaf(l, shrink, la_exp2(s2 - top));
+      }
       bf16* dst = p.out + (long long)(begin + t0 + t) * p.ld_o + (long long)h * dv;
 #pragma unroll
       for (int g = 0; g < NG; ++g) {
@@ -295,7 +301,7 @@ HFEE_API int hfee_latent_attention_mma_supports(int heads, int dk, int dv) {
 HFEE_API int hfee_latent_attention_mma(const void* q, long long ld_q, const void* pool, const int* block_table, int max_pages,
                                        int page_size, const int* cu_tokens, const int* slots, const int* context_before,
                                        void* out, long long ld_o, int requests, int max_new, int heads, int dk, int dv,
-                                       float scale, int window, cudaStream_t stream) {
+                                       float scale, int window, const float* sink, cudaStream_t stream) {
   if (requests == 0 || max_new == 0) return HFEE_OK;
   HFEE_REQUIRE(hfee_latent_attention_mma_supports(heads, dk, dv), "latent_attention_mma: sizes %d heads, %d key, %d value dimensions are not taken", heads, dk, dv);
   HFEE_REQUIRE(page_size > 0 && (page_size & (page_size - 1)) == 0, "page_size %d must be a power of two", page_size);
@@ -315,6 +321,7 @@ HFEE_API int hfee_latent_attention_mma(const void* q, long long ld_q, const void
   p.tokens_per_tile = rows / p.rows_per_token;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window;
+  p.sink = sink;
   const dim3 grid((unsigned)((max_new + p.tokens_per_tile - 1) / p.tokens_per_tile),
                   (unsigned)((heads + p.rows_per_token - 1) / p.rows_per_token), (unsigned)requests);
   HFEE_REQUIRE(grid.y <= 65535, "latent_attention_mma: too many heads");

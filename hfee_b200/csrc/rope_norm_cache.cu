@@ -11,6 +11,9 @@
 //                               RMS-normed with its weight into a buffer, the key/value latent RMS-normed
 //                               with its weight into the leading dimensions of the token's cached vector,
 //                               the rotated tail behind it.
+//   hfee_latent_attend_prepare  one token of a latent attention whose queries come from one projection: the key/value
+//                               latent and the rotated tail into the cached vector as above, and the rotated part of
+//                               every query head to its place behind the head's part for the latent; either pairing.
 //   hfee_attention_prepare     one token's [q | k | v] projection on its way to the score kernel: a bias per column
 //                               (each optional), an RMS norm with a weight over the whole query and the whole key
 //                               projection (all heads at once; optional), then the rotation of the first `rope_dim`
@@ -146,6 +149,42 @@ latent_norm_rope_cache_kernel(const T* __restrict__ proj, long long ld, int q_of
   }
 }
 
+
+// One block per token.  The rotated parts pair dimension i with i + rot_dim/2, or 2i with 2i + 1 (interleaved).
+template <typename T>
+__global__ void __launch_bounds__(LT_THREADS)
+latent_attend_prepare_kernel(const T* __restrict__ proj, long long ld, int kv_off, int kv_rank, int rot_dim, int interleaved,
+                             const float* __restrict__ wkv, float eps, const float* __restrict__ cs,
+                             const int* __restrict__ positions, const int* __restrict__ slot_of_token, HeadGroup qg,
+                             T* __restrict__ q_out, long long ld_q, T* __restrict__ k_pool, PagedCache kc) {
+  __shared__ float partial[LT_THREADS / 32];
+  const int i = blockIdx.x;
+  const int pos = positions[i], slot = slot_of_token[i];
+  pdl_wait();
+  pdl_launch_dependents();
+  const T* row = proj + (long long)i * ld;
+  const float* csr = cs + (long long)i * rot_dim;
+  const int half = rot_dim >> 1;
+  // pair `i2` of a rotated part: its two dimensions, turned, from x to dst
+  auto turn = [&](const T* x, T* dst, int i2) {
+    const int a = interleaved ? 2 * i2 : i2, b = interleaved ? 2 * i2 + 1 : i2 + half;
+    const float u = to_f32<T>(x[a]), v = to_f32<T>(x[b]), c = csr[2 * i2], s = csr[2 * i2 + 1];
+    dst[a] = from_f32<T>(u * c - v * s);
+    dst[b] = from_f32<T>(v * c + u * s);
+  };
+  for (int e = threadIdx.x; e < qg.count * half; e += LT_THREADS) {
+    const int h = e / half, i2 = e - h * half;
+    turn(row + qg.src_off + (long long)h * qg.src_stride, q_out + (long long)i * ld_q + (long long)h * qg.dst_stride + qg.dst_off, i2);
+  }
+  if (k_pool == nullptr) return;
+  const T* x = row + kv_off;
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < kv_rank; d += LT_THREADS) { const float v = to_f32<T>(x[d]); ss = fmaf(v, v, ss); }
+  const float scale = 1.0f / sqrtf(block_sum_lt(ss, partial) / (float)kv_rank + eps);
+  T* dst = k_pool + paged_offset(kc, slot, pos, 0);
+  for (int d = threadIdx.x; d < kv_rank; d += LT_THREADS) dst[d] = from_f32<T>(to_f32<T>(x[d]) * scale * wkv[d]);
+  for (int i2 = threadIdx.x; i2 < half; i2 += LT_THREADS) turn(x + kv_rank, dst + kv_rank, i2);
+}
 
 constexpr int AP_THREADS = 128;
 
@@ -358,4 +397,31 @@ HFEE_API int hfee_latent_norm_rope_cache(const void* proj, long long ld, int dty
   else
     return hfee_fail(HFEE_ERR_ARG, "latent_norm_rope_cache: unknown dtype %d", dtype);
   return hfee_check_launch("latent_norm_rope_cache");
+}
+
+// proj rows hold [key/value latent | tail to rotate] at kv_off (kv_rank + rot_dim columns) and, per query head, rot_dim
+// columns to rotate at q_src_off + h * q_src_stride, which go to q_out at q_dst_off + h * q_dst_stride.  k_pool null:
+// queries only (a run that reads a cache another run filled).
+HFEE_API int hfee_latent_attend_prepare(const void* proj, long long ld, int dtype, int n, int kv_off, int kv_rank, int rot_dim,
+                                        int interleaved, const float* wkv, float eps, const float* cs, const int* positions,
+                                        const int* slot_of_token, int heads, int q_src_off, int q_src_stride, void* q_out,
+                                        long long ld_q, int q_dst_off, int q_dst_stride, void* k_pool, const int* block_table,
+                                        int max_pages, int page_size, cudaStream_t stream) {
+  if (n == 0) return HFEE_OK;
+  HFEE_REQUIRE(heads > 0 && kv_rank > 0 && rot_dim > 0 && rot_dim % 2 == 0 && cs != nullptr, "latent_attend_prepare: bad sizes");
+  HFEE_REQUIRE(q_dst_off >= 0 && ld_q >= (long long)(heads - 1) * q_dst_stride + q_dst_off + rot_dim, "latent_attend_prepare: queries leave their row");
+  const HeadGroup qg{heads, q_src_off, q_src_stride, rot_dim, 0, q_dst_off, q_dst_stride};
+  PagedCache kc{};
+  if (k_pool != nullptr)
+    HFEE_REQUIRE(make_paged_cache(&kc, block_table, max_pages, page_size, 1, kv_rank + rot_dim), "page_size %d must be a power of two", page_size);
+  if (dtype == HFEE_F32)
+    hfee_launch(latent_attend_prepare_kernel<float>, dim3(n), dim3(LT_THREADS), 0, stream, (const float*)proj, ld, kv_off, kv_rank,
+                rot_dim, interleaved, wkv, eps, cs, positions, slot_of_token, qg, (float*)q_out, ld_q, (float*)k_pool, kc);
+  else if (dtype == HFEE_BF16)
+    hfee_launch(latent_attend_prepare_kernel<__nv_bfloat16>, dim3(n), dim3(LT_THREADS), 0, stream, (const __nv_bfloat16*)proj, ld, kv_off,
+                kv_rank, rot_dim, interleaved, wkv, eps, cs, positions, slot_of_token, qg, (__nv_bfloat16*)q_out, ld_q,
+                (__nv_bfloat16*)k_pool, kc);
+  else
+    return hfee_fail(HFEE_ERR_ARG, "latent_attend_prepare: unknown dtype %d", dtype);
+  return hfee_check_launch("latent_attend_prepare");
 }

@@ -66,7 +66,10 @@ _SIGNATURES = {
     "hfee_rope_norm_cache": [_P, _L, _I, _I, _P, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I,
                              _I, _I, _I, _P, _I, _P, _I, _I, _P],
     "hfee_latent_norm_rope_cache": [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _P, _P, _L, _P, _P, _I, _I, _P],
-    "hfee_latent_attention_mma": [_P, _L, _P, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _F, _I, _P],
+    "hfee_latent_attention_mma": [_P, _L, _P, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _F, _I, _P, _P],
+    "hfee_latent_attend_prepare": [_P, _L, _I, _I, _I, _I, _I, _I, _P, _F, _P, _P, _P, _I, _I, _I, _P, _L, _I, _I, _P, _P, _I, _I, _P],
+    "hfee_stream_step": [_P, _L, _L, _P, _L, _P, _P, _P, _P, _P, _F, _I, _P, _P, _I, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _P],
+    "hfee_channel_delta": [_P, _L, _I, _I, _I, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _P, _L, _P, _P],
     "hfee_latent_attention_mma_supports": [_I, _I, _I],
     "hfee_head_linear": [_P, _L, _I, _I, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P, _L, _I, _P],
     "hfee_conv_act": [_P, _L, _I, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P],
@@ -140,6 +143,8 @@ def library() -> ctypes.CDLL:
     lib.hfee_linear_attention_chunked_workspace.argtypes = [_I, _I, _I, _I, _I]
     lib.hfee_delta_rule_workspace.restype = _L
     lib.hfee_delta_rule_workspace.argtypes = [_I, _I, _I, _I, _I]
+    lib.hfee_channel_delta_workspace.restype = _L
+    lib.hfee_channel_delta_workspace.argtypes = [_I, _I, _I, _I, _I]
     lib.hfee_gated_recurrence_workspace.restype = _L
     lib.hfee_gated_recurrence_workspace.argtypes = [_I, _I, _I, _I, _I]
     lib.hfee_moe_tile_rows.restype = _I
@@ -1105,11 +1110,13 @@ def softmax_attention_on_tensor_cores(q: torch.Tensor, out: torch.Tensor, heads:
 
 
 def latent_attention(q: torch.Tensor, k_pool: torch.Tensor, block_table: torch.Tensor, page_size: int, step,
-                     out: torch.Tensor, heads: int, cached_dim: int, value_dim: int, scale: float, window: int = 0) -> None:
+                     out: torch.Tensor, heads: int, cached_dim: int, value_dim: int, scale: float, window: int = 0,
+                     sink: Optional[torch.Tensor] = None) -> None:
     """Softmax attention of ``heads`` query heads over ONE cached vector per token (``k_pool`` [pages, 1, page_size,
     cached_dim]) whose leading ``value_dim`` dimensions are also the values: ``out`` [n, heads * value_dim].
-    bfloat16 with sizes the tensor-core kernel takes runs there (prompt portions and decode steps alike),
+    ``sink`` (float32 per head): the denominator also holds exp(sink[h]).  bfloat16 with sizes the tensor-core kernel takes runs there (prompt portions and decode steps alike),
     everything else on the CUDA cores in float32."""
+    assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == heads)
     if (USE_LATENT_MMA and q.dtype == torch.bfloat16 and latent_mma_supports(heads, cached_dim, value_dim)
             and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0 and _rows(out, "out") % 2 == 0 and out.data_ptr() % 4 == 0):
         lib = library()
@@ -1123,10 +1130,22 @@ def latent_attention(q: torch.Tensor, k_pool: torch.Tensor, block_table: torch.T
                                              block_table.shape[1], page_size, step.cu_tokens.data_ptr(), step.slots.data_ptr(),
                                              step.context_before.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r,
                                              step.max_new, heads, cached_dim, value_dim, float(scale), int(window or 0),
-                                             _stream()), lib)
+                                             _ptr(sink), _stream()), lib)
         return
-    attention_simt_general(q, k_pool, None, block_table, page_size, step.positions, step.slot_of_token, out, heads, 1,
-                           cached_dim, value_dim, scale, window)
+    if sink is None:
+        attention_simt_general(q, k_pool, None, block_table, page_size, step.positions, step.slot_of_token, out, heads, 1,
+                               cached_dim, value_dim, scale, window)
+        return
+    lib = library()
+    _i32(step.positions, "positions"); _i32(step.slot_of_token, "slot_of_token"); _i32(block_table, "block_table")
+    n = q.shape[0]
+    assert q.shape[1] == heads * cached_dim and tuple(out.shape) == (n, heads * value_dim) and q.dtype == k_pool.dtype == out.dtype
+    assert k_pool.is_contiguous() and tuple(k_pool.shape[1:]) == (1, page_size, cached_dim)
+    _check(lib.hfee_attention_simt_sink(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), None, block_table.data_ptr(),
+                                        block_table.shape[1], page_size, step.positions.data_ptr(), step.slot_of_token.data_ptr(),
+                                        out.data_ptr(), _rows(out, "out"), n, heads, 1, cached_dim, value_dim, 1, float(scale),
+                                        int(window or 0), 0, WEIGHTS_SOFTMAX, None, None, None, 0, GATE_NONE, None, None, 1.0,
+                                        sink.data_ptr(), _dt(q), _stream()), lib)
 
 
 USE_LATENT_MMA = True
@@ -1200,6 +1219,30 @@ def latent_norm_rope_cache(proj: torch.Tensor, q_off: int, q_rank: int, kv_off: 
                                            page_size, _stream()), lib)
 
 
+def latent_attend_prepare(proj: torch.Tensor, kv_off: int, kv_rank: int, rot_dim: int, interleaved: bool, kv_weight: torch.Tensor,
+                          eps: float, cs: torch.Tensor, step, heads: int, q_src_off: int, q_src_stride: int, q_out: torch.Tensor,
+                          q_dst_off: int, q_dst_stride: int, k_pool: Optional[torch.Tensor], block_table: torch.Tensor,
+                          page_size: int) -> None:
+    """What sits between the projection of a latent attention and its scores, per token: ``proj[:, kv_off : kv_off +
+    kv_rank]`` RMS-normed with ``kv_weight`` into the leading dimensions of the token's cached vector and the ``rot_dim``
+    columns behind it, rotated, into the rest (``k_pool`` None: not stored); the ``rot_dim`` columns of every query head at
+    ``q_src_off + h * q_src_stride``, rotated, into ``q_out`` at ``q_dst_off + h * q_dst_stride``."""
+    lib = library()
+    _i32(step.positions, "positions"); _i32(step.slot_of_token, "slot_of_token"); _i32(block_table, "block_table")
+    n = proj.shape[0]
+    assert kv_weight.dtype == torch.float32 and kv_weight.numel() == kv_rank and q_out.dtype == proj.dtype and q_out.shape[0] == n
+    assert cs.dtype == torch.float32 and cs.is_contiguous() and cs.numel() == n * rot_dim
+    assert kv_off + kv_rank + rot_dim <= proj.shape[1] and q_src_off + (heads - 1) * q_src_stride + rot_dim <= proj.shape[1]
+    assert q_dst_off + (heads - 1) * q_dst_stride + rot_dim <= q_out.shape[1]
+    if k_pool is not None:
+        assert k_pool.dtype == proj.dtype and k_pool.is_contiguous() and tuple(k_pool.shape[1:]) == (1, page_size, kv_rank + rot_dim)
+    _check(lib.hfee_latent_attend_prepare(proj.data_ptr(), _rows(proj, "proj"), _dt(proj), n, kv_off, kv_rank, rot_dim,
+                                          int(interleaved), kv_weight.data_ptr(), float(eps), cs.data_ptr(),
+                                          step.positions.data_ptr(), step.slot_of_token.data_ptr(), heads, q_src_off, q_src_stride,
+                                          q_out.data_ptr(), _rows(q_out, "q_out"), q_dst_off, q_dst_stride, _ptr(k_pool),
+                                          block_table.data_ptr(), block_table.shape[1], page_size, _stream()), lib)
+
+
 def head_linear(x: torch.Tensor, in_off: int, in_stride: int, w: torch.Tensor, out: torch.Tensor, out_off: int,
                 out_stride: int, gate: Optional[torch.Tensor] = None) -> None:
     """out[i, out_off + h * out_stride + o] = sum_k w[h, o, k] * x[i, in_off + h * in_stride + k], times
@@ -1264,6 +1307,79 @@ def delta_rule(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, ba: torch.
 def delta_rule_workspace(requests: int, tokens: int, heads: int, qk_heads: int, dim: int) -> int:
     """Floats of workspace the two-kernel delta rule needs for a step of ``tokens`` tokens in ``requests`` requests."""
     return int(library().hfee_delta_rule_workspace(requests, tokens, heads, qk_heads, dim))
+
+
+def channel_delta(qkv: torch.Tensor, q_off: int, k_off: int, v_off: int, b: torch.Tensor, z: torch.Tensor, a_log: torch.Tensor,
+                  dt_bias: torch.Tensor, state: torch.Tensor, step, out: torch.Tensor, heads: int, qk_heads: int, dim: int,
+                  vdim: int, write_state: bool = True, workspace: Optional[torch.Tensor] = None) -> None:
+    """:func:`delta_rule` with a decay per key channel: S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q with
+    g = exp(-exp(a_log[h]) softplus(z + dt_bias)).  ``z`` is float32 [n, heads * dim], ``dt_bias`` [heads * dim], ``b`` [n,
+    heads] in ``qkv``'s dtype.  A step with a portion of several tokens needs ``workspace`` (float32,
+    :func:`channel_delta_workspace`) and runs as two kernels: what does not depend on the state for all tiles of 16 tokens
+    at once, then the walk over each request's tiles."""
+    lib = library()
+    n = qkv.shape[0]
+    assert qkv.dtype == b.dtype and tuple(b.shape) == (n, heads) and out.dtype == torch.float32 and tuple(out.shape) == (n, heads * vdim)
+    assert z.dtype == torch.float32 and tuple(z.shape) == (n, heads * dim)
+    assert a_log.dtype == dt_bias.dtype == torch.float32 and a_log.numel() == heads and dt_bias.numel() == heads * dim
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, dim, vdim)
+    assert max(q_off, k_off) + qk_heads * dim <= qkv.shape[1] and v_off + heads * vdim <= qkv.shape[1]
+    assert workspace is None or (workspace.dtype == torch.float32 and workspace.is_contiguous())
+    _check(lib.hfee_channel_delta(qkv.data_ptr(), _rows(qkv, "qkv"), q_off, k_off, v_off, b.data_ptr(), _rows(b, "b"), z.data_ptr(),
+                                  _rows(z, "z"), _dt(qkv), a_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(),
+                                  step.cu_tokens.data_ptr(), step.slots.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r, heads,
+                                  qk_heads, dim, vdim, int(write_state), step.n, step.max_new, _ptr(workspace),
+                                  workspace.numel() if workspace is not None else 0, _status().data_ptr(), _stream()), lib)
+    if step.max_new > 1:
+        count_launches(1)
+
+
+def channel_delta_workspace(requests: int, tokens: int, heads: int, dim: int, vdim: int) -> int:
+    """Floats of workspace :func:`channel_delta` needs for a step of ``tokens`` tokens in ``requests`` requests."""
+    return int(library().hfee_channel_delta_workspace(requests, tokens, heads, dim, vdim))
+
+
+def stream_step(x: torch.Tensor, norm_weight: torch.Tensor, eps: float, groups: int, out: torch.Tensor,
+                in_weight: Optional[torch.Tensor] = None, update=None, x_out: Optional[torch.Tensor] = None,
+                shift=None, step=None, rows: Optional[torch.Tensor] = None) -> None:
+    """Between two sublayers of a model with several residual streams, per token (float32): with ``update`` = (y [n, width],
+    M [streams, streams] indexed [from, to], b [streams]) the streams become X_t = sum_s M[s, t] X_s + b[t] y and, with
+    ``x_out``, are stored there; then u = sum_s in_weight[s] X_s (None: the plain sum), the RMS norm of u in ``groups`` equal
+    parts times ``norm_weight``, and with ``shift`` = (mu [width], state [slots, width], write_state) the row becomes
+    h + (h of the token before - h) * mu, the row before a portion's first token taken from ``state``, which then takes the
+    request's last row.  The result goes to ``out`` in its dtype.  ``x``: [n, streams, width] or [n, width] (equal streams:
+    as many as ``in_weight`` or M has, else one).  ``rows`` chooses tokens (no shift, no ``x_out``)."""
+    lib = library()
+    _i32(rows, "rows")
+    width = x.shape[-1]
+    assert x.dtype == torch.float32 and x.is_contiguous() and x.dim() in (2, 3) and norm_weight.dtype == torch.float32
+    assert norm_weight.numel() == width and norm_weight.is_contiguous() and out.shape[1] == width
+    y = mix = out_w = None
+    if update is not None:
+        y, mix, out_w = update
+        assert y.dtype == torch.float32 and y.shape == (x.shape[0], width)
+    streams = x.shape[1] if x.dim() == 3 else (out_w if out_w is not None else in_weight).numel() if (out_w is not None or in_weight is not None) else 1
+    for t, size in ((mix, streams * streams), (out_w, streams), (in_weight, streams)):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == size)
+    assert x_out is None or (x_out.dtype == torch.float32 and x_out.is_contiguous() and tuple(x_out.shape) == (x.shape[0], streams, width))
+    mu = state = None
+    write_state = False
+    if shift is not None:
+        mu, state, write_state = shift
+        assert mu.dtype == state.dtype == torch.float32 and mu.numel() == width and state.is_contiguous() and state.shape[1] == width
+    n = out.shape[0]
+    assert n == (rows.numel() if rows is not None else x.shape[0])
+    _check(lib.hfee_stream_step(x.data_ptr(), x.stride(0), width if x.dim() == 3 else 0, _ptr(y), _rows(y, "y") if y is not None else 0,
+                                _ptr(mix), _ptr(out_w), _ptr(x_out), _ptr(in_weight), norm_weight.data_ptr(), float(eps), int(groups),
+                                _ptr(mu), _ptr(state), int(write_state), step.slot_of_token.data_ptr() if shift is not None else None,
+                                step.cu_tokens.data_ptr() if shift is not None else None, step.r if shift is not None else 0,
+                                _ptr(rows), out.data_ptr(), _rows(out, "out"), _dt(out), n, width, streams, _stream()), lib)
+
+
+def group_rmsnorm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, eps: float, groups: int,
+                  rows: Optional[torch.Tensor] = None) -> None:
+    """:func:`rmsnorm` over each of ``groups`` equal consecutive parts of a row."""
+    stream_step(x, weight, eps, groups, out, rows=rows)
 
 
 def head_norm_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, gate: torch.Tensor, out: torch.Tensor, heads: int,

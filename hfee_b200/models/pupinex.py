@@ -14,7 +14,7 @@ from __future__ import annotations
 from ..config.llama import LinearRopeScaling
 from ..config.pupinex import PupinexConfig, fill_from_tensors
 from ..config.registry import register_architecture
-from ..config.spec import LayerSpec, ModelSpec, PartSpec, RunSpec
+from ..config.spec import LayerSpec, ModelSpec, PartSpec
 
 SWISH_ALPHA = 1.702          # fixed by the design: g * sigmoid(1.702 g) in the dense feed-forward
 
@@ -72,11 +72,7 @@ def run_order(cfg: PupinexConfig):
     loop = cfg.loop
     if loop is None or loop.stop == loop.start:
         return ModelSpec.sequential(n)
-    runs = [(i, False) for i in range(loop.start)]
-    for r in range(loop.times):
-        runs += [(i, r > 0 and i == loop.start) for i in range(loop.start, loop.stop)]
-    runs += [(i, False) for i in range(loop.stop, n)]
-    return tuple(RunSpec(layer=i, cache=j, adds_embedding=add) for j, (i, add) in enumerate(runs))
+    return ModelSpec.looped(n, loop.start, loop.stop, loop.times, adds_embedding=True)
 
 
 def pupinex_spec(cfg: PupinexConfig) -> ModelSpec:

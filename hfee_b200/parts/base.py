@@ -16,6 +16,8 @@ Categories and what each must provide:
 ``merge``         ``begin(residual_f32[n,w], step)`` in front of the layer's sublayers and ``forward(residual_f32[n,w],
                   y_f32[n,w] or None, scale, step)`` after them: what the next layer reads, from this layer's result
                   ``residual + scale * y`` and what earlier layers left
+``streams``       the coefficients with which a sublayer reads and writes several residual streams
+``shift``         ``weight`` and ``cache_need()`` (one row per request) of a shift towards the row of the token before
 ``block``         ``forward(residual_f32[n,w], step, cache, writes_cache)``, arranging the above; it is
                   built with ``parts={key: part}`` for the keys its layer spec names
 ``embedding``     ``forward(step, residual_f32[n,w])``
@@ -37,7 +39,7 @@ import torch
 from ..config.spec import PartSpec
 from ..weights.loader import TensorNeed
 
-CATEGORIES = ("norm", "position", "mixer", "feed_forward", "conv", "merge", "block", "embedding", "head")
+CATEGORIES = ("norm", "position", "mixer", "feed_forward", "conv", "merge", "streams", "shift", "block", "embedding", "head")
 _PARTS: Dict[Tuple[str, str], Type["Part"]] = {}
 
 

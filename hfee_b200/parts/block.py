@@ -184,6 +184,56 @@ class ScaledPreNormBlock(Block):
             ops.scaled_add(y, self.scale, residual)
 
 
+class HyperConnectedBlock(Block):
+    """Sublayers on several residual streams: ``y = mixer(shift(norm(read(X)))); X = write(X, y)`` and likewise for the
+    feed-forward, with ``read`` and ``write`` the sublayer's own coefficients (parts ``mixer_streams``, ``ffn_streams``).
+    Optional: ``mixer_shift`` (the mixer's input leans towards the row of the token before) and ``ffn`` with ``ffn_norm``
+    and ``ffn_streams``.  Takes a :class:`~hfee_b200.parts.streams.ResidualStreams` in place of the residual stream.  The
+    layer's cache is a bundle: what the mixer asks for and the shift's row (``shift``)."""
+    needs = ("mixer", "mixer_norm", "mixer_streams")
+    graph_safe = True
+    on_streams = True
+
+    def __init__(self, spec, tensors, rt, parts):
+        super().__init__(spec, tensors, rt, parts)
+        self.mixer, self.mixer_norm, self.mixer_streams = parts["mixer"], parts["mixer_norm"], parts["mixer_streams"]
+        self.shift = parts.get("mixer_shift")
+        self.feed_forward = parts.get("ffn")
+        self.ffn_norm, self.ffn_streams = parts.get("ffn_norm"), parts.get("ffn_streams")
+        if (self.feed_forward is None) != (self.ffn_norm is None) or (self.feed_forward is None) != (self.ffn_streams is None):
+            raise ValueError("a feed-forward comes with its input norm and its streams' coefficients")
+        self.width = int(spec.width)
+
+    def cache_need(self):
+        from ..cache.needs import CacheBundle, FixedState, PagedKV
+        need = self.mixer.cache_need()
+        if self.shift is None:
+            return need
+        states = {"shift": self.shift.cache_need()}
+        paged = need if isinstance(need, PagedKV) else None
+        if isinstance(need, CacheBundle):
+            paged = need.paged
+            states.update(need.states)
+        elif isinstance(need, FixedState):
+            states["recurrent"] = need
+        return CacheBundle.of(paged, **states)
+
+    def forward(self, streams, step: Any, cache: Any, writes_cache: bool) -> None:
+        rt, n = self.rt, step.n
+        xn = rt.scratch("block_normed", (rt.max_tokens, self.width))[:n]
+        y = rt.scratch("block_sublayer_out", (rt.max_tokens, self.width), torch.float32)[:n]
+        state = cache.states["shift"] if self.shift is not None else None
+        streams.read(self.mixer_streams, self.mixer_norm, xn, step, self.shift, state, writes_cache)
+        OutputNormBlock._run(self.mixer, y, xn, step, cache, writes_cache)
+        streams.leave(self.mixer_streams, y)
+        if self.feed_forward is None:
+            return
+        streams.read(self.ffn_streams, self.ffn_norm, xn, step)
+        OutputNormBlock._run(self.feed_forward, y, xn, step)
+        streams.leave(self.ffn_streams, y)
+
+
+register_part("block", "hyper_connected", HyperConnectedBlock)
 register_part("block", "scaled_pre_norm", ScaledPreNormBlock)
 register_part("block", "sandwich_norm", SandwichNormBlock)
 register_part("block", "pre_norm", PreNormBlock)

@@ -16,6 +16,7 @@ from ..config.spec import LayerSpec, ModelSpec, PartSpec, check_schedule
 from ..weights.loader import Checkpoint, TensorNeed
 from .base import Runtime, build_part, part_class
 from .norm import LazyNormed
+from .streams import ResidualStreams
 
 
 def _named(needs: Mapping[str, TensorNeed], prefix: str, names: Mapping[str, str], where: str) -> Dict[str, Tuple[str, TensorNeed]]:
@@ -81,7 +82,13 @@ class DecoderModel:
         for layer, m in zip(spec.layers, layers):
             parts = {prefix: build_part(cat, ps, fetch(m, prefix), rt) for prefix, (cat, ps) in layer.parts.items()}
             self.blocks.append(part_class("block", layer.block.kind)(layer.block, {}, rt, parts=parts))
-        self.width, self.vocab = spec.width, spec.vocab
+        self.width, self.vocab, self.streams = spec.width, spec.vocab, spec.streams
+        for run in spec.schedule:
+            if getattr(self.blocks[run.layer], "on_streams", False) != (self.streams is not None):
+                raise ValueError(f"layer {run.layer}: a model with {self.streams or 'no'} residual streams has blocks of kind "
+                                 f"{spec.layers[run.layer].block.kind!r}")
+            if self.streams is not None and run.adds_embedding:
+                raise ValueError("the embedding is added to the one residual stream; this model has several")
         self.keeps_embedding = any(run.adds_embedding for run in spec.schedule)
         # decode steps may be captured in CUDA graphs only if every part of the schedule allows it
         self.graph_safe = (self.embedding.graph_safe and self.final_norm.graph_safe and self.head.graph_safe
@@ -122,6 +129,8 @@ class DecoderModel:
         if self.keeps_embedding:
             embedded = rt.scratch("embedding_out", (rt.max_tokens, self.width), torch.float32)[:step.n]
             embedded.copy_(residual)
+        if self.streams is not None:
+            residual = ResidualStreams(rt, residual, self.streams)
         for run in self.spec.schedule:
             block = self.blocks[run.layer]
             if run.adds_embedding:
@@ -136,7 +145,11 @@ class DecoderModel:
         if m == 0:
             return None
         xn = rt.scratch("head_normed", (rt.max_tokens, self.width))[:m]
-        lazy = LazyNormed(self.final_norm, residual, xn, rows=step.logit_rows)
         logits = rt.scratch("logits", (step.logits_capacity, self.vocab), torch.float32)[:m]
+        if self.streams is not None:
+            residual.collapse(self.final_norm, xn, rows=step.logit_rows)
+            self.head.forward(xn, logits)
+            return logits
+        lazy = LazyNormed(self.final_norm, residual, xn, rows=step.logit_rows)
         self.head.forward(lazy if getattr(self.head, "accepts_lazy_input", False) else lazy.tensor(), logits)
         return logits

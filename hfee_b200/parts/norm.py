@@ -1,6 +1,6 @@
 """Norm parts.  RMS norm, formula of hostfog/hfee internal/ggml/ops.go:125-134:
 ``dst = x * 1/sqrt(mean(x^2) + eps) * weight`` per row, with the sum in float32
-here (float64 in the reference); and layer norm with a weight and no bias:
+here (float64 in the reference), over the whole row or over each of several equal parts of it; and layer norm with a weight and no bias:
 ``dst = (x - mean) / sqrt(mean((x - mean)^2) + eps) * weight``."""
 from __future__ import annotations
 
@@ -55,6 +55,33 @@ class RMSNorm(Part):
         return self.weight, self.eps, self.add_unit
 
 
+class GroupRMSNorm(Part):
+    """spec: ``width``, ``eps``, ``groups``: every one of ``groups`` equal consecutive parts of a row is divided by its own
+    root mean square, then a weight per column."""
+    category = "norm"
+    graph_safe = True
+
+    @staticmethod
+    def tensor_needs(spec: PartSpec) -> Dict[str, TensorNeed]:
+        return {"weight": TensorNeed((spec.width,), role="scale")}
+
+    def __init__(self, spec, tensors, rt):
+        super().__init__(spec, tensors, rt)
+        self.weight = tensors["weight"]
+        self.eps, self.groups = float(spec.eps), int(spec.groups)
+        if self.groups < 1 or int(spec.width) % self.groups:
+            raise ValueError(f"{self.groups} groups do not divide a width of {spec.width}")
+
+    def forward(self, x: torch.Tensor, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+        before = ops.tag("norm")
+        ops.group_rmsnorm(x, self.weight, out, self.eps, self.groups, rows=rows)
+        ops.tag(before)
+
+    def group_params(self):
+        """(weight, eps, groups): what a kernel needs to apply this norm itself."""
+        return self.weight, self.eps, self.groups
+
+
 class LayerNorm(Part):
     """spec: ``width``, ``eps``.  Mean and variance (the mean of the squared deviations) per row in float32; a weight
     per column, no bias."""
@@ -104,4 +131,5 @@ class LazyNormed:
 
 
 register_part("norm", "rms_norm", RMSNorm)
+register_part("norm", "group_rms_norm", GroupRMSNorm)
 register_part("norm", "layer_norm", LayerNorm)
