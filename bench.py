@@ -25,7 +25,9 @@ Muvetar model (minGRU layers in turn with softmax attention under a logarithmic 
 scan; routed experts with a shared one whose active sizes add up to the dense feed-forward; depth averaging);
 ``--design pupinex`` for a Pupinex model (windowed attention with normed queries and keys beside a matrix memory, windowed
 attention with a sink, gated linear attention with a decay per key channel; a clamped gated feed-forward in turn with
-group-limited routed experts and a gated shared one; a hashed bigram embedding and layer norms).
+group-limited routed experts and a gated shared one; a hashed bigram embedding and layer norms); ``--design fokalorn``
+for a Fokalorn model (a delta rule with a decay per key channel in turn with latent attention over all earlier positions
+with a sink; four residual streams, norms in groups, a token shift, a relu^2 feed-forward), beside a Bamipel model as well.
 ``--breakdown`` prints, instead of the line above, what each class of kernels costs inside the decode
 step at batch 1, 8 and 64 and inside the prompt pass: the step is timed again with that class's
 launches left out (results wrong, timing not), and the difference is the class's cost in place.
@@ -252,10 +254,32 @@ def pupinex_like(model, layers, experts=16, top=2):
             "norm": {"eps": 1e-5}, "embedding": {"bigram": {"buckets": 65521, "mul_prev": 1000003, "mul_cur": 31}}}
 
 
-DESIGNS = {"dobelix": dobelix_like, "bamipel": bamipel_like, "muvetar": muvetar_like, "pupinex": pupinex_like}
+def fokalorn_like(model, layers, streams=4):
+    """A Fokalorn configuration of the layer sizes of the Llama configuration ``model``: in turn the channel-decay delta
+    rule (as many value heads, a query/key head per key/value head, four taps, low-rank projections of a head size) and
+    latent attention (a key/value latent of four head sizes, a rotated part of half a head, no window); ``streams``
+    residual streams, norms in two groups, the dense relu^2 feed-forward.  No stretch of layers is looped."""
+    h, kv, hd = model["num_attention_heads"], model["num_key_value_heads"], model["head_dim"]
+    ff = {"kind": "dense", "ff": model["intermediate_size"]}
+    kinds = [
+        {"type": "channel_delta", "mlp": ff,
+         "mixer": {"heads": h, "kv_heads": kv, "dim": hd, "vdim": hd, "conv": 4, "rank": hd, "gate_rank": hd}},
+        {"type": "latent_attention", "mlp": ff,
+         "mixer": {"heads": h, "dim": hd, "rot_dim": hd // 2, "vdim": hd, "kv_rank": 4 * hd,
+                   "rot": {"dims": hd // 2, "base": 10000.0}, "scale": (hd + hd // 2) ** -0.5}},
+    ]
+    return {"architecture": "Fokalorn", "vocab": model["vocab_size"], "width": model["hidden_size"], "streams": streams,
+            "layers": [kinds[i % 2] for i in range(layers)], "norm": {"eps": 1e-5, "groups": 2}, "embedding": {"scale": 1.0}}
+
+
+DESIGNS = {"fokalorn": fokalorn_like, "dobelix": dobelix_like, "bamipel": bamipel_like, "muvetar": muvetar_like, "pupinex": pupinex_like}
 # kernel classes (the names the parts tag their launches with) that only some layers of a design have: class -> the layer
 # types that have it; every other class is counted once per layer ("head": once per model)
+CLOSEST = {"fokalorn": ("bamipel",)}          # designs measured beside this one, after the Llama model
 DESIGN_CLASSES = {
+    "fokalorn": {"conv": ("channel_delta",), "low_rank": ("channel_delta",), "delta_rule": ("channel_delta",), "gate": ("channel_delta",),
+                 "rope": ("latent_attention",), "attention": ("latent_attention",), "fold": ("latent_attention",),
+                 "expand": ("latent_attention",)},
     "dobelix": {"conv": ("lightning", "attention"), "gate": ("lightning",), "linear_attention": ("lightning",),
                 "rope": ("attention",), "attention": ("attention",)},
     "bamipel": {"conv": ("delta",), "delta_rule": ("delta",), "gate": ("delta",), "rope": ("attention", "latent_attention"),
@@ -265,7 +289,7 @@ DESIGN_CLASSES = {
     "pupinex": {"rope": ("parallel", "attention"), "attention": ("parallel", "attention"), "scan_proj": ("parallel", "gla"),
                 "linear_attention": ("parallel", "gla"), "gate": ("parallel", "gla"), "router": ("attention",), "experts": ("attention",)},
 }
-CLASS_ORDER = ("conv", "norm", "qkv", "rope", "fold", "attention", "expand", "linear_attention", "delta_rule", "scan_proj", "scan",
+CLASS_ORDER = ("conv", "norm", "qkv", "rope", "fold", "attention", "expand", "linear_attention", "low_rank", "delta_rule", "scan_proj", "scan",
                "gate", "o", "router", "experts", "gate_up", "up", "down", "head")
 
 
@@ -283,7 +307,7 @@ def design_comparison(args):
     layers = args.layers or 6
     base = dict(base, num_hidden_layers=layers, vocab_size=32768, tie_word_embeddings=True,
                 max_position_embeddings=max(base["max_position_embeddings"], 2 * args.prompt))
-    designs = {"llama": base, args.design: DESIGNS[args.design](base, layers)}
+    designs = {"llama": base, **{d: DESIGNS[d](base, layers) for d in CLOSEST.get(args.design, ()) + (args.design,)}}
     rng = np.random.default_rng(0)
     out = {"design_comparison": f"{base_name} layer sizes, {layers} layers, vocabulary 32768, bf16, random weights",
            "prompt_tokens": args.prompt, "decode_batch": args.batch,
@@ -345,7 +369,7 @@ def design_comparison(args):
             kinds = [l["type"] for l in cfg["layers"]]
             having = {c: sum(kinds.count(k) for k in types) for c, types in DESIGN_CLASSES[name].items()}
             having.update({c: 0 for cs in DESIGN_CLASSES.values() for c in cs if c not in having})
-            having.update({"gate_up": 0, "up": layers} if name == "bamipel" else {"gate_up": layers, "up": 0})
+            having.update({"gate_up": 0, "up": layers} if name in ("bamipel", "fokalorn") else {"gate_up": layers, "up": 0})
 
         def classes_of(measure, rounds=3):
             res = {}

@@ -43,9 +43,50 @@ struct ChannelDeltaArgs {
   int q_off, k_off, v_off;
   int heads, qk_heads, dim, vdim;
   int write_state;
+  int vec;                     // rows of q, k, z and dt_bias can be fetched four channels at a time
 };
 
 __device__ __forceinline__ float softplus_cd(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+// the decay of one key channel; the bfloat16 instances take the fast exponential (relative error of some 1e-6)
+template <typename T> __device__ __forceinline__ float channel_decay(float rate, float z);
+template <> __device__ __forceinline__ float channel_decay<float>(float rate, float z) { return expf(-rate * softplus_cd(z)); }
+template <> __device__ __forceinline__ float channel_decay<__nv_bfloat16>(float rate, float z) {
+  return __expf(-rate * (fmaxf(z, 0.f) + log1pf(__expf(-fabsf(z)))));
+}
+template <typename T> __device__ __forceinline__ float4 load4(const T* p);
+template <> __device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
+template <> __device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(r.x << 16), __uint_as_float(r.x & 0xffff0000u), __uint_as_float(r.y << 16), __uint_as_float(r.y & 0xffff0000u));
+}
+
+// Two float32 numbers side by side, multiplied and added as a pair.
+__device__ __forceinline__ uint64_t pair_of(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float2 unpair(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma_pair(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul_pair(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t add_pair(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 
 // ---------------------------------------------------------------------------------------------------------------
 // One token per request.  A thread keeps RPT rows of VEC neighbouring columns in registers; 32 / VEC threads side by
@@ -89,7 +130,7 @@ channel_delta_token_kernel(const T* __restrict__ qkv, const T* __restrict__ b, c
     const float zz = z[(long long)tok * p.ld_z + (long long)h * dim + d] + dt_bias[(long long)h * dim + d];
     k_s[d] = kv;
     q_s[d] = qv;
-    g_s[d] = expf(-rate * softplus_cd(zz));
+    g_s[d] = channel_decay<T>(rate, zz);
     sk = fmaf(kv, kv, sk);
     sq = fmaf(qv, qv, sq);
     kq = fmaf(kv, qv, kq);
@@ -162,7 +203,6 @@ channel_delta_token_kernel(const T* __restrict__ qkv, const T* __restrict__ b, c
 
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int CW_COLS = 16;                                         // state columns per block of the walk
-constexpr int CW_WARPS = 4;                                         // each takes four of them
 constexpr int CW_STAGES = 3;
 
 __host__ __device__ inline int cd_pad(int dim) { return (dim + 31) / 32 * 32; }
@@ -172,7 +212,7 @@ constexpr int CD_UO = 2 * CD_TILE * CW_COLS;
 
 // NI: float4 per lane of a row (a row of DP = 32 * NI floats shared by 8 lanes)
 template <typename T, int NI>
-__global__ void __launch_bounds__(CD_THREADS)
+__global__ void __launch_bounds__(CD_THREADS, NI <= 4 ? 4 : 3)
 channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b, const float* __restrict__ z,
                              const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                              const int* __restrict__ cu_tokens, float* __restrict__ ws_head, float* __restrict__ ws_uo,
@@ -187,26 +227,47 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
   const int req = blockIdx.z, h = blockIdx.y, tile0 = blockIdx.x * CD_TILE;
   const int begin = cu_tokens[req], count = cu_tokens[req + 1] - begin;
   pdl_wait();
-  pdl_launch_dependents();
+  // the walk's few blocks are let in only when this kernel's last ones are done: let in earlier they would all settle on
+  // the first SMs with room
   if (tile0 >= count) return;
   const int tt = min(CD_TILE, count - tile0);
   const long long tok0 = begin + tile0, place = tok0 / CD_TILE + req;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dim = p.dim, vdim = p.vdim, kh = h / (p.heads / p.qk_heads);
   const float rate = expf(a_log[h]);
-  for (int e = tid; e < CD_TILE * DP; e += CD_THREADS) {
-    const int t = e / DP, d = e - t * DP;
-    const bool in = t < tt && d < dim;
-    float kv = 0.f, qv = 0.f, g = 1.f;       // a missing token is the identity: no write, no decay
-    if (in) {
-      const T* row = qkv + (tok0 + t) * p.ld_qkv + (long long)kh * dim + d;
-      kv = to_f32<T>(row[p.k_off]);
-      qv = to_f32<T>(row[p.q_off]);
-      g = expf(-rate * softplus_cd(z[(tok0 + t) * p.ld_z + (long long)h * dim + d] + dt_bias[(long long)h * dim + d]));
+  // a missing token is the identity: no write, no decay
+  if (p.vec) {
+#pragma unroll
+    for (int n = 0; n < NI; ++n) {
+      const int e = tid + n * CD_THREADS, t = e / (DP / 4), d = (e - t * (DP / 4)) * 4;
+      float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), qv = kv, g = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (t < tt && d < dim) {
+        const T* row = qkv + (tok0 + t) * p.ld_qkv + (long long)kh * dim + d;
+        kv = load4<T>(row + p.k_off);
+        qv = load4<T>(row + p.q_off);
+        const float4 zz = *reinterpret_cast<const float4*>(z + (tok0 + t) * p.ld_z + (long long)h * dim + d);
+        const float4 bb = *reinterpret_cast<const float4*>(dt_bias + (long long)h * dim + d);
+        g = make_float4(channel_decay<T>(rate, zz.x + bb.x), channel_decay<T>(rate, zz.y + bb.y), channel_decay<T>(rate, zz.z + bb.z),
+                        channel_decay<T>(rate, zz.w + bb.w));
+      }
+      reinterpret_cast<float4*>(k_s)[e] = kv;
+      reinterpret_cast<float4*>(q_s)[e] = qv;
+      reinterpret_cast<float4*>(g_s)[e] = g;
     }
-    k_s[e] = kv;
-    q_s[e] = qv;
-    g_s[e] = g;
+  } else {
+    for (int e = tid; e < CD_TILE * DP; e += CD_THREADS) {
+      const int t = e / DP, d = e - t * DP;
+      float kv = 0.f, qv = 0.f, g = 1.f;
+      if (t < tt && d < dim) {
+        const T* row = qkv + (tok0 + t) * p.ld_qkv + (long long)kh * dim + d;
+        kv = to_f32<T>(row[p.k_off]);
+        qv = to_f32<T>(row[p.q_off]);
+        g = channel_decay<T>(rate, z[(tok0 + t) * p.ld_z + (long long)h * dim + d] + dt_bias[(long long)h * dim + d]);
+      }
+      k_s[e] = kv;
+      q_s[e] = qv;
+      g_s[e] = g;
+    }
   }
   if (tid < CD_TILE) beta_s[tid] = tid < tt ? 1.f / (1.f + expf(-to_f32<T>(b[(tok0 + tid) * p.ld_b + h]))) : 0.f;
   __syncthreads();
@@ -224,26 +285,29 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
   {
     // the tables: eight lanes per row j, each with its share of the channels of G_t / G_j * k_j as t runs on from j
     const int j = tid >> 3, sl = tid & 7;
-    const float4* k4 = reinterpret_cast<const float4*>(k_s);
-    const float4* q4 = reinterpret_cast<const float4*>(q_s);
-    const float4* g4 = reinterpret_cast<const float4*>(g_s);
-    float4 w[NI];
+    const ulonglong2* k4 = reinterpret_cast<const ulonglong2*>(k_s);
+    const ulonglong2* q4 = reinterpret_cast<const ulonglong2*>(q_s);
+    const ulonglong2* g4 = reinterpret_cast<const ulonglong2*>(g_s);
+    ulonglong2 w[NI];
 #pragma unroll
     for (int i = 0; i < NI; ++i) w[i] = k4[j * (DP / 4) + sl + 8 * i];
     const int j_first = (warp * 4);            // smallest j of this warp: earlier tokens concern none of its rows
     for (int t = j_first; t < tt; ++t) {
-      float a = 0.f, c = 0.f;
+      uint64_t a2 = 0, c2 = 0;                 // pairs of zeros
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
         const int at = t * (DP / 4) + sl + 8 * i;
-        const float4 kk = k4[at], qq = q4[at];
+        const ulonglong2 kk = k4[at], qq = q4[at];
         if (t > j) {
-          const float4 g = g4[at];
-          w[i].x *= g.x; w[i].y *= g.y; w[i].z *= g.z; w[i].w *= g.w;
+          const ulonglong2 g = g4[at];
+          w[i].x = mul_pair(w[i].x, g.x);
+          w[i].y = mul_pair(w[i].y, g.y);
         }
-        a = fmaf(w[i].x, kk.x, a); a = fmaf(w[i].y, kk.y, a); a = fmaf(w[i].z, kk.z, a); a = fmaf(w[i].w, kk.w, a);
-        c = fmaf(w[i].x, qq.x, c); c = fmaf(w[i].y, qq.y, c); c = fmaf(w[i].z, qq.z, c); c = fmaf(w[i].w, qq.w, c);
+        a2 = fma_pair(w[i].x, kk.x, a2); a2 = fma_pair(w[i].y, kk.y, a2);
+        c2 = fma_pair(w[i].x, qq.x, c2); c2 = fma_pair(w[i].y, qq.y, c2);
       }
+      const float2 af = unpair(a2), cf = unpair(c2);
+      float a = af.x + af.y, c = cf.x + cf.y;
 #pragma unroll
       for (int o = 4; o >= 1; o >>= 1) {
         a += __shfl_xor_sync(0xffffffffu, a, o);
@@ -312,11 +376,14 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
 }
 
 // A block walks the tiles of one request and head for CW_COLS state columns; the tiles' parts of the workspace come in
-// through a ring of bulk copies.  A warp owns four columns; eight lanes share a column, lane dg of them holding the rows
-// 4 dg + 32 i + (0..3).  Rows of W and P times the lanes' rows of S are summed over the eight lanes so that lane dg ends
-// with those of the tokens dg and dg + 8; u is then handed around token by token for the update.
-template <int NI>
-__global__ void __launch_bounds__(CW_WARPS * 32)
+// through a ring of bulk copies.  A warp owns C neighbouring columns.  Lane (dg, cg), dg < 8 and cg < 4, holds the rows
+// 4 dg + 32 i + (0..3) of all C of them (the four lanes of a dg hold copies): for the products with W and P it takes the
+// rows t = 4 r + cg, r < 8, of the two matrices, so that a row is read from shared memory once per warp, and eight
+// lanes' partial sums leave lane (dg, cg) with those of t = 4 dg + cg: rows of W in the lanes with dg < 4, of P in the
+// others.  For the update it takes the tokens 4 r + cg, and the four partial sums meet by exchanges across cg, in an
+// order that gives every copy the same bits.
+template <int NI, int C>
+__global__ void __launch_bounds__(CW_COLS / C * 32, 1)
 channel_delta_walk_kernel(const float* __restrict__ ws_head, const float* __restrict__ ws_uo, float* __restrict__ state,
                           const int* __restrict__ cu_tokens, const int* __restrict__ slots, float* __restrict__ out,
                           int* __restrict__ status, ChannelDeltaArgs p) {
@@ -330,7 +397,7 @@ channel_delta_walk_kernel(const float* __restrict__ ws_head, const float* __rest
   const int slot = slots[req];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dg = lane & 7, cg = lane >> 3;
-  const int in_tile = warp * 4 + cg, col = tile_col * CW_COLS + in_tile;
+  const int in_tile = warp * C, col = tile_col * CW_COLS + in_tile;
   const int dim = p.dim, vdim = p.vdim, tiles = (count + CD_TILE - 1) / CD_TILE;
   if (tid == 0) {
     abort_flag = 0;
@@ -356,86 +423,125 @@ channel_delta_walk_kernel(const float* __restrict__ ws_head, const float* __rest
   if (tid == 0)
     for (int t = 0; t < CW_STAGES - 1 && t < tiles; ++t) fetch(t);
   float* sp = state + ((long long)slot * p.heads + h) * (long long)dim * vdim + col;
-  float S[NI][4];
+  uint64_t S[NI][C][2];                                       // rows (0, 1) and (2, 3) of the lane's four, per column
 #pragma unroll
   for (int i = 0; i < NI; ++i)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int d = 32 * i + 4 * dg + e;
-      S[i][e] = (d < dim && col < vdim) ? sp[(long long)d * vdim] : 0.f;
-    }
+    for (int c = 0; c < C; ++c)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int d = 32 * i + 4 * dg + 2 * e;
+        S[i][c][e] = pair_of((d < dim && col + c < vdim) ? sp[(long long)d * vdim + c] : 0.f,
+                             (d + 1 < dim && col + c < vdim) ? sp[(long long)(d + 1) * vdim + c] : 0.f);
+      }
+  const bool wide = C == 4 && vdim % 4 == 0 && p.ld_out % 4 == 0 && (uintptr_t)out % 16 == 0;
   bool ok = true;
   for (int tile = 0; tile < tiles; ++tile) {
     const int s = tile % CW_STAGES;
     ok = tc::mbar_wait(&full[s], (tile / CW_STAGES) & 1u, &abort_flag);
     if (!__syncthreads_and(ok)) { ok = false; break; }        // also: every warp is done with the tile before
     if (tid == 0 && tile + CW_STAGES - 1 < tiles) fetch(tile + CW_STAGES - 1);
-    const float4* M4 = reinterpret_cast<const float4*>(smem + s * STAGE);
-    const float* uo = smem + s * STAGE + HEAD;
-    float x[4];                                               // tokens dg, dg + 8 of W S and of P S
+    const ulonglong2* M = reinterpret_cast<const ulonglong2*>(smem + s * STAGE) + dg;
+    float val[8 * C];                                         // [r][c]
 #pragma unroll
-    for (int grp = 0; grp < 4; ++grp) {
-      float val[8];
-#pragma unroll
-      for (int r = 0; r < 8; ++r) {
-        float a = 0.f, c = 0.f;
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-          const float4 m = M4[(grp * 8 + r) * (DP / 4) + dg + 8 * i];
-          a = fmaf(m.x, S[i][0], a); c = fmaf(m.y, S[i][1], c);
-          a = fmaf(m.z, S[i][2], a); c = fmaf(m.w, S[i][3], c);
-        }
-        val[r] = a + c;
-      }
-#pragma unroll
-      for (int off = 4; off >= 1; off >>= 1) {
-        const bool upper = (lane & off) != 0;
-#pragma unroll
-        for (int i = 0; i < off; ++i) {
-          const float send = upper ? val[i] : val[i + off], keep = upper ? val[i + off] : val[i];
-          val[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
-        }
-      }
-      x[grp] = val[0];
-    }
-    const float u0 = uo[dg * CW_COLS + in_tile] - x[0], u1 = uo[(dg + 8) * CW_COLS + in_tile] - x[1];
-    const float o0 = uo[(CD_TILE + dg) * CW_COLS + in_tile] + x[2], o1 = uo[(CD_TILE + dg + 8) * CW_COLS + in_tile] + x[3];
-    const int tt = min(CD_TILE, count - tile * CD_TILE);
-    float* orow = out + (long long)(begin + tile * CD_TILE) * p.ld_out + (long long)h * vdim + col;
-    if (col < vdim && dg < tt) orow[(long long)dg * p.ld_out] = o0;
-    if (col < vdim && dg + 8 < tt) orow[(long long)(dg + 8) * p.ld_out] = o1;
-    const float4* K4 = M4 + 2 * CD_TILE * (DP / 4);
-#pragma unroll
-    for (int i = 0; i < NI; ++i) {
-      const float4 g = K4[CD_TILE * (DP / 4) + dg + 8 * i];
-      S[i][0] *= g.x; S[i][1] *= g.y; S[i][2] *= g.z; S[i][3] *= g.w;
-    }
-#pragma unroll
-    for (int j = 0; j < CD_TILE; ++j) {
-      const float u = __shfl_sync(0xffffffffu, j < 8 ? u0 : u1, (lane & 24) + (j & 7));
+    for (int r = 0; r < 8; ++r) {
+      uint64_t acc[C];
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
-        const float4 kk = K4[j * (DP / 4) + dg + 8 * i];
-        S[i][0] = fmaf(kk.x, u, S[i][0]); S[i][1] = fmaf(kk.y, u, S[i][1]);
-        S[i][2] = fmaf(kk.z, u, S[i][2]); S[i][3] = fmaf(kk.w, u, S[i][3]);
+        const ulonglong2 m = M[(4 * r + cg) * (DP / 4) + 8 * i];
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          acc[c] = i == 0 ? mul_pair(m.x, S[i][c][0]) : fma_pair(m.x, S[i][c][0], acc[c]);
+          acc[c] = fma_pair(m.y, S[i][c][1], acc[c]);
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const float2 f = unpair(acc[c]);
+        val[r * C + c] = f.x + f.y;
+      }
+    }
+#pragma unroll
+    for (int off = 4; off >= 1; off >>= 1) {
+      const bool upper = (lane & off) != 0;
+#pragma unroll
+      for (int i = 0; i < off * C; ++i) {
+        const float send = upper ? val[i] : val[i + off * C], keep = upper ? val[i + off * C] : val[i];
+        val[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
+      }
+    }
+    const int t = 4 * dg + cg;                                // below 16: u of token t, else o of token t - 16
+    const float* uo = smem + s * STAGE + HEAD + t * CW_COLS + in_tile;
+    float x[C];
+#pragma unroll
+    for (int c = 0; c < C; ++c) x[c] = uo[c] + (dg < 4 ? -val[c] : val[c]);
+    if (dg >= 4 && tile * CD_TILE + t - CD_TILE < count) {
+      float* o = out + (long long)(begin + tile * CD_TILE + t - CD_TILE) * p.ld_out + (long long)h * vdim + col;
+      if (wide && C == 4) {
+        if (col < vdim) *reinterpret_cast<float4*>(o) = make_float4(x[0], x[1 % C], x[2 % C], x[3 % C]);
+      } else {
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+          if (col + c < vdim) o[c] = x[c];
+      }
+    }
+    uint64_t u[4][C];                                         // of the tokens 4 r + cg, twice side by side
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        const float v = __shfl_sync(0xffffffffu, x[c], (lane & 24) + r);
+        u[r][c] = pair_of(v, v);
+      }
+    const ulonglong2* K = M + 2 * CD_TILE * (DP / 4);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      uint64_t d[C][2];
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        const ulonglong2 k = K[(4 * r + cg) * (DP / 4) + 8 * i];
+#pragma unroll
+        for (int c = 0; c < C; ++c) {
+          d[c][0] = r == 0 ? mul_pair(k.x, u[r][c]) : fma_pair(k.x, u[r][c], d[c][0]);
+          d[c][1] = r == 0 ? mul_pair(k.y, u[r][c]) : fma_pair(k.y, u[r][c], d[c][1]);
+        }
+      }
+#pragma unroll
+      for (int off = 8; off <= 16; off <<= 1)
+#pragma unroll
+        for (int c = 0; c < C; ++c)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const float2 f = unpair(d[c][e]);
+            d[c][e] = add_pair(d[c][e], pair_of(__shfl_xor_sync(0xffffffffu, f.x, off), __shfl_xor_sync(0xffffffffu, f.y, off)));
+          }
+      const ulonglong2 g = K[CD_TILE * (DP / 4) + 8 * i];
+#pragma unroll
+      for (int c = 0; c < C; ++c) {
+        S[i][c][0] = fma_pair(g.x, S[i][c][0], d[c][0]);
+        S[i][c][1] = fma_pair(g.y, S[i][c][1], d[c][1]);
       }
     }
   }
-  if (!ok) {                                                  // a copy never arrived: say so; copies in flight end on their own barriers
+  if (!ok) {                                                  // a copy never arrived: say so; copies in flight get a while to end
     if (tid == 0) *status = 1;
     for (int s = 0; s < CW_STAGES; ++s)
       for (int i = 0; i < 64; ++i)
         if (tc::mbar_try(&full[s], 0) || tc::mbar_try(&full[s], 1)) break;
     return;
   }
-  if (p.write_state)
+  if (p.write_state && cg == 0)
 #pragma unroll
     for (int i = 0; i < NI; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = 32 * i + 4 * dg + e;
-        if (d < dim && col < vdim) sp[(long long)d * vdim] = S[i][e];
-      }
+      for (int c = 0; c < C; ++c)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int d = 32 * i + 4 * dg + 2 * e;
+          const float2 f = unpair(S[i][c][e]);
+          if (d < dim && col + c < vdim) sp[(long long)d * vdim + c] = f.x;
+          if (d + 1 < dim && col + c < vdim) sp[(long long)(d + 1) * vdim + c] = f.y;
+        }
 }
 
 template <typename T, int VEC, int RPT>
@@ -465,6 +571,7 @@ template <typename T, int NI>
 int launch_tiles_n(const void* qkv, const void* b, const float* z, const float* a_log, const float* dt_bias, float* state,
                    const int* cu_tokens, const int* slots, float* out, const ChannelDeltaArgs& p, int requests, int max_new,
                    float* ws_head, float* ws_uo, int* status, cudaStream_t stream) {
+  constexpr int C = NI <= 4 ? 4 : 2;                          // columns per warp of the walk: what its registers hold
   const size_t prep = (size_t)3 * CD_TILE * 32 * NI * sizeof(float);
   const size_t walk = (size_t)CW_STAGES * ((3 * CD_TILE + 1) * 32 * NI + CD_UO) * sizeof(float);
   if (prep > 40 * 1024) {
@@ -472,15 +579,15 @@ int launch_tiles_n(const void* qkv, const void* b, const float* z, const float* 
     if (e != cudaSuccess) return hfee_fail(HFEE_ERR_CUDA, "channel_delta_prepare: %s", cudaGetErrorString(e));
   }
   if (walk > 40 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk);
+    cudaError_t e = cudaFuncSetAttribute(channel_delta_walk_kernel<NI, C>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)walk);
     if (e != cudaSuccess) return hfee_fail(HFEE_ERR_CUDA, "channel_delta_walk: %s", cudaGetErrorString(e));
   }
   hfee_launch(channel_delta_prepare_kernel<T, NI>, dim3((unsigned)((max_new + CD_TILE - 1) / CD_TILE), (unsigned)p.heads, (unsigned)requests),
               dim3(CD_THREADS), prep, stream, (const T*)qkv, (const T*)b, z, a_log, dt_bias, cu_tokens, ws_head, ws_uo, p);
   const int rc = hfee_check_launch("channel_delta_prepare");
   if (rc != HFEE_OK) return rc;
-  hfee_launch(channel_delta_walk_kernel<NI>, dim3((unsigned)cd_col_tiles(p.vdim), (unsigned)p.heads, (unsigned)requests),
-              dim3(CW_WARPS * 32), walk, stream, ws_head, ws_uo, state, cu_tokens, slots, out, status, p);
+  hfee_launch(channel_delta_walk_kernel<NI, C>, dim3((unsigned)cd_col_tiles(p.vdim), (unsigned)p.heads, (unsigned)requests),
+              dim3(CW_COLS / C * 32), walk, stream, ws_head, ws_uo, state, cu_tokens, slots, out, status, p);
   return hfee_check_launch("channel_delta_walk");
 }
 
@@ -519,7 +626,9 @@ HFEE_API int hfee_channel_delta(const void* qkv, long long ld_qkv, int q_off, in
   HFEE_REQUIRE(dim > 0 && dim <= CD_MAX_DIM && vdim > 0, "channel_delta: key size %d is outside 1..%d", dim, CD_MAX_DIM);
   HFEE_REQUIRE(requests <= 65535 && heads <= 65535, "channel_delta: too many requests or heads");
   HFEE_REQUIRE(dtype == HFEE_F32 || dtype == HFEE_BF16, "channel_delta: unknown dtype %d", dtype);
-  const ChannelDeltaArgs p{ld_qkv, ld_b, ld_z, ld_out, q_off, k_off, v_off, heads, qk_heads, dim, vdim, write_state};
+  const int vec = dim % 4 == 0 && ld_qkv % 4 == 0 && ld_z % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
+                  (uintptr_t)qkv % (dtype == HFEE_F32 ? 16 : 8) == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)dt_bias % 16 == 0;
+  const ChannelDeltaArgs p{ld_qkv, ld_b, ld_z, ld_out, q_off, k_off, v_off, heads, qk_heads, dim, vdim, write_state, vec};
   if (max_new == 1) {
     if (dtype == HFEE_F32) return launch_token<float>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, stream);
     return launch_token<__nv_bfloat16>(qkv, b, z, a_log, dt_bias, state, cu_tokens, slots, out, p, requests, stream);

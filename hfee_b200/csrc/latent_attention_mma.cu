@@ -12,6 +12,10 @@
 // registers, so the four warps split a block twice: for S = Q K^T each warp takes 16 of the block's keys (queries
 // and keys both come from shared memory), the row maxima and sums meet in shared memory, the weights go to shared
 // memory as bfloat16, and for O += P V each warp takes every fourth group of 16 value columns for all rows.
+//
+// A step of single tokens leaves most SMs idle at one CTA per request (and slice of the heads), so its keys may be split
+// among `splits` CTAs, each with an equal share of the visible key blocks: they leave unnormalised float32 outputs with
+// their rows' maxima and sums, and latent_combine_kernel puts the shares together.
 #include "mma_tiles.cuh"
 
 namespace {
@@ -33,6 +37,9 @@ struct LatentParams {
   int rows_per_token, tokens_per_tile;
   float scale_log2;
   int window;
+  int splits;                      // CTAs that share a tile's keys (1: each writes its outputs itself)
+  float* partial;                  // [splits][tokens][heads][dv + 2]: output, maximum (log2 units), sum
+  int n_tokens;
   const float* sink;               // per head, or null: one more term exp(sink[h]) of the softmax's denominator
 };
 
@@ -74,7 +81,8 @@ latent_attention_kernel(LatentParams p) {
 
   const int req = blockIdx.z, head0 = blockIdx.y * p.rows_per_token;
   const int begin = p.cu_tokens[req], count = p.cu_tokens[req + 1] - begin;     // host-written batch layout
-  const int t0 = blockIdx.x * p.tokens_per_tile;
+  const int split = blockIdx.x % p.splits;
+  const int t0 = blockIdx.x / p.splits * p.tokens_per_tile;
   pdl_wait();
   pdl_launch_dependents();
   if (t0 >= count) return;
@@ -82,8 +90,14 @@ latent_attention_kernel(LatentParams p) {
   const int slot = p.slots[req], before = p.context_before[req];
   const int tid = threadIdx.x, warp = (tid >> 5) % LA_WARPS, lane = tid & 31;
   const int rb = (tid >> 5) / LA_WARPS * LA_ROWS;              // first row of this set of warps
-  const int p_first = before + t0, p_last = before + t0 + tokens - 1;
-  const int lo = p.window > 0 ? max(0, p_first - p.window + 1) : 0;
+  const int p_first = before + t0;
+  int p_last = before + t0 + tokens - 1;
+  int lo = p.window > 0 ? max(0, p_first - p.window + 1) : 0;
+  if (p.splits > 1) {                                          // this CTA's share of the blocks that hold keys lo .. p_last
+    const int b0 = lo / LA_BN, blocks = p_last / LA_BN - b0 + 1, share = (blocks + p.splits - 1) / p.splits;
+    lo = max(lo, (b0 + split * share) * LA_BN);
+    p_last = min(p_last, (b0 + (split + 1) * share) * LA_BN - 1);        // may leave nothing: lo > p_last
+  }
   const int* table = p.block_table + (long long)slot * p.max_pages;
   const long long page_stride = (long long)(p.page_mask + 1) * dk;
 
@@ -246,6 +260,7 @@ latent_attention_kernel(LatentParams p) {
       }
     }
   }
+  la_wait_all();
   __syncthreads();
 #pragma unroll
   for (int mt = 0; mt < 2; ++mt)
@@ -255,6 +270,22 @@ latent_attention_kernel(LatentParams p) {
       if (rowpos[row] < 0) continue;
       const int t = row / p.rows_per_token, h = head0 + row % p.rows_per_token;
       const float l = l_s[row];
+      if (p.splits > 1) {
+        float* part = p.partial + (((long long)split * p.n_tokens + begin + t0 + t) * p.heads + h) * (dv + 2);
+#pragma unroll
+        for (int g = 0; g < NG; ++g) {
+          const int grp = warp + LA_WARPS * g;
+          if (grp >= groups) break;
+#pragma unroll
+          for (int nt = 0; nt < 2; ++nt)
+            *reinterpret_cast<float2*>(part + 16 * grp + 8 * nt + quad_col) = make_float2(o[g][nt][mt][2 * half], o[g][nt][mt][2 * half + 1]);
+        }
+        if (warp == 0 && (lane & 3) == 0) {
+          part[dv] = m_s[row];
+          part[dv + 1] = l;
+        }
+        continue;
+      }
       float inv = l > 0.f ? 1.f / l : 0.f;
       if (p.sink != nullptr) {                 // joins the row's sum once; against the larger of the two exponents
         const float s2 = p.sink[h] * 1.4426950408889634f, m = m_s[row], top = fmaxf(m, s2);
@@ -272,6 +303,44 @@ latent_attention_kernel(LatentParams p) {
               __floats2bfloat162_rn(o[g][nt][mt][2 * half] * inv, o[g][nt][mt][2 * half + 1] * inv);
       }
     }
+}
+
+// One (token, head) per warp: the shares' outputs against the largest of their maxima (and the sink's).
+__global__ void __launch_bounds__(128)
+latent_combine_kernel(const float* __restrict__ partial, int splits, int n_tokens, int heads, int dv, const float* __restrict__ sink,
+                      bf16* __restrict__ out, long long ld_o) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int task = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (task >= n_tokens * heads) return;
+  const int t = task / heads, h = task - t * heads;
+  const long long stride = (long long)n_tokens * heads * (dv + 2);
+  const float* mine = partial + (long long)task * (dv + 2);
+  float m = -INFINITY, l = 0.f;                                // lane s: share s (at most 32 of them)
+  if (lane < splits) {
+    m = mine[lane * stride + dv];
+    l = mine[lane * stride + dv + 1];
+  }
+  float top = warp_max(m);
+  const float s2 = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
+  top = fmaxf(top, s2);
+  const float w = m == -INFINITY ? 0.f : la_exp2(m - top);
+  const float total = warp_sum(w * l) + (sink != nullptr ? la_exp2(s2 - top) : 0.f);
+  const float inv = total > 0.f ? 1.f / total : 0.f;
+  bf16* dst = out + (long long)t * ld_o + (long long)h * dv;
+  for (int base = 0; base < dv; base += 64) {                  // the same for all lanes: they hand their weights around
+    const int d = base + 2 * lane;
+    float a = 0.f, b = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float ws = __shfl_sync(0xffffffffu, w, s);
+      if (d < dv) {
+        const float2 v = *reinterpret_cast<const float2*>(mine + s * stride + d);
+        a = fmaf(ws, v.x, a);
+        b = fmaf(ws, v.y, b);
+      }
+    }
+    if (d < dv) *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(a * inv, b * inv);
+  }
 }
 
 size_t latent_smem(int dk, int rows) {
@@ -298,16 +367,20 @@ HFEE_API int hfee_latent_attention_mma_supports(int heads, int dk, int dv) {
   return heads > 0 && dk > 0 && dk % 16 == 0 && dv > 0 && dv % 16 == 0 && dv <= dk && dv <= 512 && latent_smem(dk, LA_ROWS) <= 227 * 1024;
 }
 
+// splits > 1 (at most 32): that many CTAs share a tile's keys through `partial`, [splits][n_tokens][heads][dv + 2] floats.
 HFEE_API int hfee_latent_attention_mma(const void* q, long long ld_q, const void* pool, const int* block_table, int max_pages,
                                        int page_size, const int* cu_tokens, const int* slots, const int* context_before,
                                        void* out, long long ld_o, int requests, int max_new, int heads, int dk, int dv,
-                                       float scale, int window, const float* sink, cudaStream_t stream) {
+                                       float scale, int window, const float* sink, int splits, float* partial, int n_tokens,
+                                       cudaStream_t stream) {
   if (requests == 0 || max_new == 0) return HFEE_OK;
   HFEE_REQUIRE(hfee_latent_attention_mma_supports(heads, dk, dv), "latent_attention_mma: sizes %d heads, %d key, %d value dimensions are not taken", heads, dk, dv);
   HFEE_REQUIRE(page_size > 0 && (page_size & (page_size - 1)) == 0, "page_size %d must be a power of two", page_size);
   HFEE_REQUIRE(ld_q % 8 == 0 && (uintptr_t)q % 16 == 0 && (uintptr_t)pool % 16 == 0, "latent_attention_mma: queries and cache must be 16-byte aligned");
   HFEE_REQUIRE(ld_o % 2 == 0 && (uintptr_t)out % 4 == 0, "latent_attention_mma: the output's rows must start on 4 bytes");
   HFEE_REQUIRE(requests <= 65535 && window >= 0, "latent_attention_mma: bad batch or window");
+  HFEE_REQUIRE(splits >= 1 && splits <= 32 && (splits == 1 || (partial != nullptr && (uintptr_t)partial % 8 == 0 && n_tokens > 0)),
+               "latent_attention_mma: %d splits of the keys need their workspace", splits);
   LatentParams p{};
   p.q = (const bf16*)q; p.ld_q = ld_q; p.out = (bf16*)out; p.ld_o = ld_o; p.pool = (const bf16*)pool;
   p.block_table = block_table; p.max_pages = max_pages; p.page_mask = page_size - 1;
@@ -322,18 +395,27 @@ HFEE_API int hfee_latent_attention_mma(const void* q, long long ld_q, const void
   p.scale_log2 = scale * 1.4426950408889634f;
   p.window = window;
   p.sink = sink;
-  const dim3 grid((unsigned)((max_new + p.tokens_per_tile - 1) / p.tokens_per_tile),
+  p.splits = splits;
+  p.partial = partial;
+  p.n_tokens = n_tokens;
+  const dim3 grid((unsigned)((max_new + p.tokens_per_tile - 1) / p.tokens_per_tile * splits),
                   (unsigned)((heads + p.rows_per_token - 1) / p.rows_per_token), (unsigned)requests);
   HFEE_REQUIRE(grid.y <= 65535, "latent_attention_mma: too many heads");
   const int per_warp = (dv / 16 + LA_WARPS - 1) / LA_WARPS;
+  int rc;
   if (sets == 2) {
-    if (per_warp <= 1) return launch_latent<1, 2>(p, grid, stream);
-    if (per_warp <= 2) return launch_latent<2, 2>(p, grid, stream);
-    if (per_warp <= 4) return launch_latent<4, 2>(p, grid, stream);
-    return launch_latent<8, 2>(p, grid, stream);
+    if (per_warp <= 1) rc = launch_latent<1, 2>(p, grid, stream);
+    else if (per_warp <= 2) rc = launch_latent<2, 2>(p, grid, stream);
+    else if (per_warp <= 4) rc = launch_latent<4, 2>(p, grid, stream);
+    else rc = launch_latent<8, 2>(p, grid, stream);
+  } else {
+    if (per_warp <= 1) rc = launch_latent<1, 1>(p, grid, stream);
+    else if (per_warp <= 2) rc = launch_latent<2, 1>(p, grid, stream);
+    else if (per_warp <= 4) rc = launch_latent<4, 1>(p, grid, stream);
+    else rc = launch_latent<8, 1>(p, grid, stream);
   }
-  if (per_warp <= 1) return launch_latent<1, 1>(p, grid, stream);
-  if (per_warp <= 2) return launch_latent<2, 1>(p, grid, stream);
-  if (per_warp <= 4) return launch_latent<4, 1>(p, grid, stream);
-  return launch_latent<8, 1>(p, grid, stream);
+  if (rc != HFEE_OK || splits == 1) return rc;
+  hfee_launch(latent_combine_kernel, dim3((unsigned)(((long long)n_tokens * heads + 3) / 4)), dim3(128), 0, stream, partial, splits,
+              n_tokens, heads, dv, sink, (bf16*)out, ld_o);
+  return hfee_check_launch("latent_combine");
 }

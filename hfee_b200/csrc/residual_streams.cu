@@ -63,7 +63,7 @@ template <> __device__ __forceinline__ void store_row<__nv_bfloat16, 4>(__nv_bfl
 
 // S: number of streams, or 0 for any number (the streams are then read again for every output stream).
 template <typename T, int S, int VEC>
-__global__ void __launch_bounds__(ST_THREADS)
+__global__ void __launch_bounds__(ST_THREADS, S > 0 ? 3 : 2)
 stream_step_kernel(StreamArgs p, T* __restrict__ h_out) {
   extern __shared__ __align__(16) float row_s[];       // [width]: u of the token in work; with a shift [width]: the row before
   __shared__ float coef_s[ST_MAX_STREAMS * 2 + (S > 0 ? S * S : ST_MAX_STREAMS * ST_MAX_STREAMS)];
@@ -181,30 +181,28 @@ stream_step_kernel(StreamArgs p, T* __restrict__ h_out) {
     turn ^= 1;                                         // the next token's sums go to the other half of red_s
   };
 
-  if (p.shift_w == nullptr) {
-    for (int i = i0; i < i1; ++i)
-      normed(i, true, [&](int c, const Pack<VEC>& h) { store_row<T, VEC>(h_out + (long long)i * p.ld_h + c, h); });
-    return;
-  }
-  auto first_of_request = [&](int i) { return i == 0 || p.slot_of_token[i - 1] != p.slot_of_token[i]; };
+  const bool shift = p.shift_w != nullptr;
   bool reads_state = false;                            // the request in work has its first token of the step in this block
-  if (!first_of_request(i0))
-    normed(i0 - 1, false, [&](int c, const Pack<VEC>& h) { h.store(prev_s + c); });
-  for (int i = i0; i < i1; ++i) {
-    const bool first = first_of_request(i);
-    const bool last = i + 1 == p.n || p.slot_of_token[i + 1] != p.slot_of_token[i];
+  auto first_of_request = [&](int i) { return i == 0 || p.slot_of_token[i - 1] != p.slot_of_token[i]; };
+  // the run, behind the token in front of it if that is needed, and in front of the last request's last token likewise
+  int i = shift && !first_of_request(i0) ? i0 - 1 : i0;
+  for (; i < i1; ++i) {
+    const bool own = i >= i0, first = shift && own && first_of_request(i);
     reads_state = reads_state || first;
-    float* state = p.shift_state + (long long)p.slot_of_token[i] * p.width;
-    const bool renew = last && reads_state && p.write_state;
-    normed(i, true, [&](int c, const Pack<VEC>& h) {
-      Pack<VEC> before, mu, out;
-      before.load((first ? state : prev_s) + c);
-      mu.load(p.shift_w + c);
+    float* state = shift ? p.shift_state + (long long)p.slot_of_token[i] * p.width : nullptr;
+    const bool renew = shift && own && reads_state && p.write_state && (i + 1 == p.n || p.slot_of_token[i + 1] != p.slot_of_token[i]);
+    normed(i, own, [&](int c, const Pack<VEC>& h) {
+      Pack<VEC> out = h;
+      if (shift && own) {
+        Pack<VEC> before, mu;
+        before.load((first ? state : prev_s) + c);
+        mu.load(p.shift_w + c);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) out.v[e] = fmaf(before.v[e] - h.v[e], mu.v[e], h.v[e]);
-      store_row<T, VEC>(h_out + (long long)i * p.ld_h + c, out);
-      h.store(prev_s + c);
-      if (renew) h.store(state + c);
+        for (int e = 0; e < VEC; ++e) out.v[e] = fmaf(before.v[e] - h.v[e], mu.v[e], h.v[e]);
+        if (renew) h.store(state + c);
+      }
+      if (own) store_row<T, VEC>(h_out + (long long)i * p.ld_h + c, out);
+      if (shift) h.store(prev_s + c);
     });
   }
   if (reads_state && p.write_state && i1 < p.n && p.slot_of_token[i1] == p.slot_of_token[i1 - 1]) {
@@ -263,8 +261,8 @@ HFEE_API int hfee_stream_step(const float* x, long long token_stride, long long 
   const int sms = hfee_sm_count();
   HFEE_REQUIRE(sms > 0, "stream_step: cannot ask the device for its number of SMs");
   int run = 1;
-  if (shift_w != nullptr) {                            // a longer run computes fewer rows twice; about four blocks an SM
-    run = (n + 4 * sms - 1) / (4 * sms);
+  if (shift_w != nullptr) {                            // a longer run computes fewer rows twice; one wave of three blocks an SM
+    run = (n + 3 * sms - 1) / (3 * sms);
     run = run < 1 ? 1 : (run > 8 ? 8 : run);
   }
   const StreamArgs p{x, token_stride, stream_stride, y, ld_y, mix, out_w, x_out, in_w, norm_w, eps, groups, shift_w, shift_state,

@@ -11,6 +11,8 @@ where that matters, and prints what it achieved against the roofline that bounds
     python -m hfee_b200.kernels.microbench sigmoid_attention --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64 --chunk 128
     python -m hfee_b200.kernels.microbench linear_attention  --tokens 2048 --heads 32 --head-dim 64 [--batch 8 for a decode step]
     python -m hfee_b200.kernels.microbench delta_rule        --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64 [--decode --batch 8]
+    python -m hfee_b200.kernels.microbench channel_delta     --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64 [--decode --batch 8]
+    python -m hfee_b200.kernels.microbench stream_step       --tokens 2048 --k 2048 --streams 4
     python -m hfee_b200.kernels.microbench conv_act          --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64
     python -m hfee_b200.kernels.microbench latent_attention  --tokens 2048 --heads 32 --head-dim 64 --rank 256 --window 512 [--decode --batch 8]
     python -m hfee_b200.kernels.microbench head_linear       --tokens 2048 --heads 32 --head-dim 64 --rank 256
@@ -244,7 +246,9 @@ def _latent_attention(args) -> dict:
     q = (torch.randn(b.n, heads * dk, device=DEV) * 0.3).to(torch.bfloat16)
     out = torch.empty(b.n, heads * rank, dtype=torch.bfloat16, device=DEV)
     ops.USE_LATENT_MMA = not args.no_tc_attention
-    fn = lambda i: ops.latent_attention(q, pool, table, page, b, out, heads, dk, rank, dk ** -0.5, window)
+    scratch = torch.empty(160 * heads * (rank + 2), device=DEV)
+    b.planning_context, b.attention_splits = b.max_context, args.splits or None
+    fn = lambda i: ops.latent_attention(q, pool, table, page, b, out, heads, dk, rank, dk ** -0.5, window, None, scratch)
     sec = _time(fn, args.warmup, args.iters)
     keys = sum(min(p + 1, window) if window else p + 1 for s, c in zip(before, new) for p in range(s, s + c))
     flops = 2.0 * heads * (dk + rank) * keys
@@ -459,6 +463,45 @@ def _gated_recurrence(args, mode: int) -> dict:
             "io_gbs": round(io / sec / 1e9, 1)}
 
 
+def _channel_delta(args) -> dict:
+    """The delta rule with a decay per key channel, ``--heads`` value heads on ``--kv-heads`` query/key heads."""
+    heads, qk, d, vd = args.heads, args.kv_heads, args.head_dim, args.value_dim or args.head_dim
+    before, new = ([args.context] * args.batch, [1] * args.batch) if args.decode else ([0] * args.requests, [args.tokens // args.requests] * args.requests)
+    b = _batch_of(before, new)
+    qc, vc = qk * d, heads * vd
+    qkv = torch.randn(b.n, 2 * qc + vc, device=DEV).to(torch.bfloat16)
+    beta = torch.randn(b.n, heads, device=DEV).to(torch.bfloat16)
+    z = torch.randn(b.n, heads * d, device=DEV)
+    a_log, dt = torch.linspace(-4.0, -1.0, heads, device=DEV), torch.full((heads * d,), -2.0, device=DEV)
+    states = [torch.zeros(b.r, heads, d, vd, device=DEV) for _ in range(args.rotate if args.decode else 1)]
+    out = torch.empty(b.n, vc, device=DEV)
+    ws = torch.empty(ops.channel_delta_workspace(b.r, b.n, heads, d, vd), device=DEV)
+    fn = lambda i: ops.channel_delta(qkv, 0, qc, 2 * qc, beta, z, a_log, dt, states[i % len(states)], b, out, heads, qk, d, vd, True, ws)
+    sec = _time(fn, args.warmup, args.iters)
+    io = b.n * ((2 * qc + vc) * 2 + heads * d * 4 + vc * 4) + 2 * b.r * heads * d * vd * 4
+    return {"kernel": "channel_delta", "heads": heads, "qk_heads": qk, "key_dim": d, "value_dim": vd, "tokens": b.n, "requests": b.r,
+            "us": round(sec * 1e6, 2), "io_gbs": round(io / sec / 1e9, 1), "fp32_tflops": round(6.0 * b.n * heads * d * vd / sec / 1e12, 2)}
+
+
+def _stream_step(args) -> dict:
+    """From one sublayer's output to the next one's input with ``--streams`` residual streams of width ``--k``: plain,
+    with the token shift, and the final sum; buffers rotate so that decode steps do not find them in L2 either."""
+    n, w, s = args.tokens, args.k, args.streams
+    b = _batch_of([0], [n])
+    xs = [torch.randn(n, s, w, device=DEV) for _ in range(max(2, min(args.rotate, (1 << 31) // (n * s * w * 4))))]
+    y, nw, mu = torch.randn(n, w, device=DEV), torch.ones(w, device=DEV), torch.rand(w, device=DEV)
+    a, mix = torch.rand(s, device=DEV), torch.rand(s, s, device=DEV) / s
+    state = torch.zeros(b.r, w, device=DEV)
+    out = torch.empty(n, w, dtype=torch.bfloat16, device=DEV)
+    res = {"kernel": "stream_step", "tokens": n, "width": w, "streams": s}
+    nbytes = n * w * (8 * s + 4 + 2)
+    step = lambda i, shift: ops.stream_step(xs[i % len(xs)], nw, 1e-5, 2, out, a, (y, mix, a), xs[(i + 1) % len(xs)], shift, b)
+    for name, shift in (("plain", None), ("token_shift", (mu, state, True))):
+        sec = _time(lambda i: step(i, shift), args.warmup, args.iters)
+        res[name] = {"us": round(sec * 1e6, 2), "gbs": round(nbytes / sec / 1e9, 1)}
+    return res
+
+
 def _pupinex_rows(args) -> dict:
     """Row kernels of the Pupinex parts on ``--tokens`` rows of width ``--k``: layer norm, the bigram embedding, the bias,
     the step between the q/k/v projection and the attention, and the per-head norm with its gate."""
@@ -506,7 +549,7 @@ def main(argv=None) -> int:
                                        "gemm_tcgen05", "gemm_stream", "gemm_skinny", "gemm_ring", "gemm_pair", "attention_decode", "attention_prefill",
                                       "sigmoid_attention", "linear_attention", "mingru", "selective_scan",
                                        "distance_attention", "moe_experts", "row_ops", "softmax_attention", "gla", "matrix_memory",
-                                       "pupinex_rows"])
+                                       "pupinex_rows", "channel_delta", "stream_step"])
     ap.add_argument("--m", type=int, default=2048)
     ap.add_argument("--n", type=int, default=16384)
     ap.add_argument("--k", type=int, default=2048)
@@ -529,6 +572,8 @@ def main(argv=None) -> int:
     ap.add_argument("--channels", type=int, default=2048, help="mingru / selective_scan: channels of the recurrence")
     ap.add_argument("--state", type=int, default=16, help="selective_scan: state entries per channel")
     ap.add_argument("--value-dim", type=int, default=0, help="distance_attention: value size per head (0: the key size)")
+    ap.add_argument("--streams", type=int, default=4, help="stream_step: residual streams")
+    ap.add_argument("--requests", type=int, default=1, help="channel_delta: equal portions that --tokens is divided into")
     ap.add_argument("--experts", type=int, default=16)
     ap.add_argument("--top", type=int, default=2)
     ap.add_argument("--inner", type=int, default=2048, help="moe_experts / row_ops: inner size of an expert")
@@ -560,6 +605,8 @@ def main(argv=None) -> int:
         res = _softmax_attention(args)
     elif args.kernel in ("gla", "matrix_memory"):
         res = _gated_recurrence(args, 0 if args.kernel == "gla" else 1)
+    elif args.kernel in ("channel_delta", "stream_step"):
+        res = {"channel_delta": _channel_delta, "stream_step": _stream_step}[args.kernel](args)
     elif args.kernel == "pupinex_rows":
         res = _pupinex_rows(args)
     else:

@@ -66,7 +66,7 @@ _SIGNATURES = {
     "hfee_rope_norm_cache": [_P, _L, _I, _I, _P, _I, _F, _P, _P, _I, _I, _I, _I, _I, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _I, _I,
                              _I, _I, _I, _P, _I, _P, _I, _I, _P],
     "hfee_latent_norm_rope_cache": [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _P, _P, _L, _P, _P, _I, _I, _P],
-    "hfee_latent_attention_mma": [_P, _L, _P, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _F, _I, _P, _P],
+    "hfee_latent_attention_mma": [_P, _L, _P, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _P],
     "hfee_latent_attend_prepare": [_P, _L, _I, _I, _I, _I, _I, _I, _P, _F, _P, _P, _P, _I, _I, _I, _P, _L, _I, _I, _P, _P, _I, _I, _P],
     "hfee_stream_step": [_P, _L, _L, _P, _L, _P, _P, _P, _P, _P, _F, _I, _P, _P, _I, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _P],
     "hfee_channel_delta": [_P, _L, _I, _I, _I, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _P, _L, _P, _P],
@@ -1111,10 +1111,11 @@ def softmax_attention_on_tensor_cores(q: torch.Tensor, out: torch.Tensor, heads:
 
 def latent_attention(q: torch.Tensor, k_pool: torch.Tensor, block_table: torch.Tensor, page_size: int, step,
                      out: torch.Tensor, heads: int, cached_dim: int, value_dim: int, scale: float, window: int = 0,
-                     sink: Optional[torch.Tensor] = None) -> None:
+                     sink: Optional[torch.Tensor] = None, scratch: Optional[torch.Tensor] = None) -> None:
     """Softmax attention of ``heads`` query heads over ONE cached vector per token (``k_pool`` [pages, 1, page_size,
     cached_dim]) whose leading ``value_dim`` dimensions are also the values: ``out`` [n, heads * value_dim].
-    ``sink`` (float32 per head): the denominator also holds exp(sink[h]).  bfloat16 with sizes the tensor-core kernel takes runs there (prompt portions and decode steps alike),
+    ``sink`` (float32 per head): the denominator also holds exp(sink[h]).  ``scratch`` (float32) lets a step of single
+    tokens split its keys among CTAs.  bfloat16 with sizes the tensor-core kernel takes runs there (prompt portions and decode steps alike),
     everything else on the CUDA cores in float32."""
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == heads)
     if (USE_LATENT_MMA and q.dtype == torch.bfloat16 and latent_mma_supports(heads, cached_dim, value_dim)
@@ -1126,11 +1127,19 @@ def latent_attention(q: torch.Tensor, k_pool: torch.Tensor, block_table: torch.T
         assert k_pool.dtype == out.dtype == torch.bfloat16 and k_pool.is_contiguous()
         assert tuple(k_pool.shape[1:]) == (1, page_size, cached_dim)
         assert tuple(q.shape) == (step.n, heads * cached_dim) and tuple(out.shape) == (step.n, heads * value_dim)
+        splits = 1
+        if step.max_new == 1 and scratch is not None:
+            assert scratch.dtype == torch.float32 and scratch.is_contiguous()
+            splits = getattr(step, "attention_splits", None) or latent_splits(
+                step.r, heads, getattr(step, "planning_context", step.max_context), int(window or 0))
+            splits = max(1, min(splits, scratch.numel() // max(1, step.n * heads * (value_dim + 2))))
         _check(lib.hfee_latent_attention_mma(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), block_table.data_ptr(),
                                              block_table.shape[1], page_size, step.cu_tokens.data_ptr(), step.slots.data_ptr(),
                                              step.context_before.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r,
                                              step.max_new, heads, cached_dim, value_dim, float(scale), int(window or 0),
-                                             _ptr(sink), _stream()), lib)
+                                             _ptr(sink), splits, _ptr(scratch) if splits > 1 else None, step.n, _stream()), lib)
+        if splits > 1:
+            count_launches(1)
         return
     if sink is None:
         attention_simt_general(q, k_pool, None, block_table, page_size, step.positions, step.slot_of_token, out, heads, 1,
@@ -1146,6 +1155,13 @@ def latent_attention(q: torch.Tensor, k_pool: torch.Tensor, block_table: torch.T
                                         out.data_ptr(), _rows(out, "out"), n, heads, 1, cached_dim, value_dim, 1, float(scale),
                                         int(window or 0), 0, WEIGHTS_SOFTMAX, None, None, None, 0, GATE_NONE, None, None, 1.0,
                                         sink.data_ptr(), _dt(q), _stream()), lib)
+
+
+def latent_splits(requests: int, heads: int, max_context: int, window: int) -> int:
+    """How many CTAs share the keys of one request in a decode step of the latent attention: about one CTA an SM (a CTA
+    takes up to 64 heads and most of an SM's shared memory), at least two key blocks of 64 each."""
+    keys = min(max_context, window + 64) if window else max_context
+    return max(1, min(MAX_SPLITS, sm_count() // max(1, requests * -(-heads // 64)), keys // 128))
 
 
 USE_LATENT_MMA = True

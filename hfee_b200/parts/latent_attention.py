@@ -121,8 +121,12 @@ class LatentAttention(Mixer):
                                 q=(h, d, d + r, r, 0, qf, rank, self.cached_dim))
         ol = rt.scratch("lattn_latent_out", (rt.max_tokens, pad8(h * rank)))[:n, :h * rank]
         ops.tag("attention")
+        # a decode step's keys may be split among CTAs; room for about one CTA an SM, or two per request
+        scratch = None
+        if rt.dtype == torch.bfloat16:
+            scratch = rt.scratch("lattn_partial", (max(2 * rt.max_requests, 160) * h * (rank + 2),), torch.float32)
         ops.latent_attention(qf, cache.k, cache.block_table, cache.page_size, step, ol, h, self.cached_dim, rank,
-                             self.scale, int(self.window or 0), self.sink)
+                             self.scale, int(self.window or 0), self.sink, scratch)
         att = rt.scratch("lattn_out", (rt.max_tokens, pad8(h * v)))[:n, :h * v]
         gate = proj[:, self.g_at:self.g_at + h] if self.g_at is not None else None
         ops.tag("expand")
