@@ -72,23 +72,23 @@ class FokalornConfig:
             m = _get(entry, "mixer", where)
             mw = where + ".mixer"
             if kind == "channel_delta":
-                heads, kv = _at_least_one(m, "heads", mw), _at_least_one(m, "kv_heads", mw)
+                heads, kv = _int(m, "heads", mw), _int(m, "kv_heads", mw)
                 if heads % kv:
                     raise ConfigError(f"config.json: {mw}.heads {heads} must be a multiple of kv_heads {kv}")
                 for key, tensor in (("rank", "a1"), ("gate_rank", "g1")):
                     if not isinstance(m, Mapping) or m.get(key) is None:
                         raise ConfigError(f"config.json: {mw}: {key} is neither given nor known from the tensor l{i}.mix.{tensor}")
-                mixer = ChannelDeltaMixer(heads, kv, _at_least_one(m, "dim", mw), _at_least_one(m, "vdim", mw),
-                                          _at_least_one(m, "conv", mw), int(m["rank"]), int(m["gate_rank"]))
+                mixer = ChannelDeltaMixer(heads, kv, _int(m, "dim", mw), _int(m, "vdim", mw),
+                                          _int(m, "conv", mw), int(m["rank"]), int(m["gate_rank"]))
             elif kind == "latent_attention":
-                rot_dim = _at_least_one(m, "rot_dim", mw)
+                rot_dim = _int(m, "rot_dim", mw)
                 rot = _get(m, "rot", mw)
                 dims = _int(rot, "dims", mw + ".rot")
                 if dims != rot_dim or dims % 2:
                     raise ConfigError(f"config.json: {mw}.rot.dims {dims} must be even and equal rot_dim {rot_dim}: the whole "
                                       "shared key part is rotated")
-                mixer = LatentMixer(_at_least_one(m, "heads", mw), _at_least_one(m, "dim", mw), rot_dim, _at_least_one(m, "vdim", mw),
-                                    _at_least_one(m, "kv_rank", mw), _num(m, "scale", mw), _positive(rot, "base", mw + ".rot"))
+                mixer = LatentMixer(_int(m, "heads", mw), _int(m, "dim", mw), rot_dim, _int(m, "vdim", mw),
+                                    _int(m, "kv_rank", mw), _num(m, "scale", mw), _positive(rot, "base", mw + ".rot"))
             else:
                 raise ConfigError(f"config.json: {where}.type {kind!r} is not a mixer of this design (known: channel_delta, latent_attention)")
             mlp = entry.get("mlp") if isinstance(entry, Mapping) else None
@@ -96,7 +96,7 @@ class FokalornConfig:
                 mk = _get(mlp, "kind", where + ".mlp")
                 if mk != "dense":
                     raise ConfigError(f"config.json: {where}.mlp.kind {mk!r} is not a feed-forward of this design (known: dense)")
-                mlp = DenseMlp(_at_least_one(mlp, "ff", where + ".mlp"))
+                mlp = DenseMlp(_int(mlp, "ff", where + ".mlp"))
             out.append(FokalornLayer(kind, mixer, mlp))
         loop = d.get("loop")
         if loop is not None:
@@ -104,20 +104,13 @@ class FokalornConfig:
             if not (0 <= loop.start <= loop.stop <= len(out)) or loop.times < 1:
                 raise ConfigError(f"config.json: loop {loop.start}..{loop.stop} x {loop.times} does not fit {len(out)} layers")
         norm = _get(d, "norm", "config")
-        width, groups = _at_least_one(d, "width", "config"), _at_least_one(norm, "groups", "norm")
+        width, groups = _int(d, "width", "config"), _int(norm, "groups", "norm")
         if width % groups:
             raise ConfigError(f"config.json: norm.groups {groups} does not divide the width {width}")
         max_positions = d.get("max_positions", d.get("max_position_embeddings", 1 << 20))
-        return cls(vocab=_at_least_one(d, "vocab", "config"), width=width, streams=_at_least_one(d, "streams", "config"),
+        return cls(vocab=_int(d, "vocab", "config"), width=width, streams=_int(d, "streams", "config"),
                    layers=tuple(out), loop=loop, eps=_num(norm, "eps", "norm"), groups=groups,
                    embedding_scale=_num(_get(d, "embedding", "config"), "scale", "embedding"), max_positions=int(max_positions))
-
-
-def _at_least_one(d: Mapping[str, Any], key: str, where: str) -> int:
-    v = _int(d, key, where)
-    if v < 1:
-        raise ConfigError(f"config.json: {where}.{key} must be positive, got {v}")
-    return v
 
 
 def fill_from_tensors(config_json: Mapping[str, Any], shapes: Mapping[str, Tuple[int, ...]]) -> Mapping[str, Any]:

@@ -212,7 +212,7 @@ constexpr int CD_UO = 2 * CD_TILE * CW_COLS;
 
 // NI: float4 per lane of a row (a row of DP = 32 * NI floats shared by 8 lanes)
 template <typename T, int NI>
-__global__ void __launch_bounds__(CD_THREADS, NI <= 4 ? 4 : 3)
+__global__ void __launch_bounds__(CD_THREADS, NI <= 4 ? 5 : 3)
 channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b, const float* __restrict__ z,
                              const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                              const int* __restrict__ cu_tokens, float* __restrict__ ws_head, float* __restrict__ ws_uo,
@@ -272,14 +272,21 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
   if (tid < CD_TILE) beta_s[tid] = tid < tt ? 1.f / (1.f + expf(-to_f32<T>(b[(tok0 + tid) * p.ld_b + h]))) : 0.f;
   __syncthreads();
   const float q_unit = 1.0f / sqrtf((float)dim);
-  for (int vid = warp; vid < 2 * tt; vid += CD_THREADS / 32) {
-    float* vec = vid < tt ? q_s + vid * DP : k_s + (vid - tt) * DP;
-    float x[NI], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < NI; ++i) { x[i] = vec[lane + 32 * i]; ss = fmaf(x[i], x[i], ss); }
-    const float scale = (vid < tt ? q_unit : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+  for (int half = 0; half < 2; ++half) {       // eight lanes per vector: 16 keys, then 16 queries
+    float4* vec = reinterpret_cast<float4*>(half ? q_s : k_s) + (tid >> 3) * (DP / 4) + (tid & 7);
+    float4 x[NI];
+    float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < NI; ++i) vec[lane + 32 * i] = x[i] * scale;
+    for (int i = 0; i < NI; ++i) {
+      x[i] = vec[8 * i];
+      ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss);
+    }
+#pragma unroll
+    for (int o = 4; o >= 1; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float scale = (half ? q_unit : 1.f) / sqrtf(ss + 1e-6f);
+#pragma unroll
+    for (int i = 0; i < NI; ++i) vec[8 * i] = make_float4(x[i].x * scale, x[i].y * scale, x[i].z * scale, x[i].w * scale);
   }
   __syncthreads();
   {
