@@ -37,7 +37,7 @@ def config(width, vocab, layers, streams=3, groups=4, loop=None, eps=1e-5, scale
 FOK_A = config(64, 200, [delta(4, 2, 16, 24, 4, ff=80), latent(4, 24, 8, 16, 40, 0.3, 500.0, ff=96), delta(3, 1, 32, 16, 2, ff=48),
                          latent(2, 16, 16, 40, 24, 0.25, 2.0e4, ff=72)], streams=3, groups=4, loop=(1, 3, 3), eps=1e-5, scale=3.0)
 FOK_B = config(96, 310, [latent(5, 16, 32, 24, 64, 0.2, 77.0), delta(2, 2, 48, 40, 1, ff=64, ranks=(3, 17)),
-                         latent(3, 8, 4, 8, 28, 0.4, 1.0e5, ff=56), delta(1, 1, 72, 88, 5)], streams=5, groups=1, eps=1e-6, scale=0.6)
+                         latent(3, 8, 4, 8, 28, 0.4, 1.0e5, ff=56), delta(1, 1, 72, 88, 5)], streams=5, groups=1, eps=1e-6, scale=4.0)
 STD = 0.15
 MARK_A, MARK_B, MARK_LATER = 0, 1, 2      # embedding dimensions that mark the tokens of the far-token tests
 
@@ -89,7 +89,7 @@ def write_model(path, cfg, seed, dtype="bfloat16", edit=None):
         elif name.endswith(".dt_bias"):
             uniform(t, -4.0, 1.0)
         elif name.endswith((".a2", ".g2", ".mix.b")):
-            t.mul_(4.0)                       # gates that move with the token
+            t.mul_(3.0)                       # gates that move with the token
     if edit is not None:
         edit(tensors)
     store = {"bfloat16": torch.bfloat16, "float32": torch.float32}[dtype]
