@@ -212,7 +212,7 @@ constexpr int CD_UO = 2 * CD_TILE * CW_COLS;
 
 // NI: float4 per lane of a row (a row of DP = 32 * NI floats shared by 8 lanes)
 template <typename T, int NI>
-__global__ void __launch_bounds__(CD_THREADS, NI <= 4 ? 5 : 3)
+__global__ void __launch_bounds__(CD_THREADS, NI <= 4 ? 6 : 3)
 channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b, const float* __restrict__ z,
                              const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                              const int* __restrict__ cu_tokens, float* __restrict__ ws_head, float* __restrict__ ws_uo,
@@ -222,7 +222,7 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
   float* k_s = smem;                         // [16][DP]
   float* q_s = k_s + CD_TILE * DP;
   float* g_s = q_s + CD_TILE * DP;
-  __shared__ __align__(16) float A_s[CD_TILE][CD_TILE], B_s[CD_TILE][CD_TILE];
+  __shared__ __align__(16) float2 A_s[CD_TILE][CD_TILE], B_s[CD_TILE][CD_TILE];      // -A and B, every number twice: operands of pairs
   __shared__ float beta_s[CD_TILE];
   const int req = blockIdx.z, h = blockIdx.y, tile0 = blockIdx.x * CD_TILE;
   const int begin = cu_tokens[req], count = cu_tokens[req + 1] - begin;
@@ -234,6 +234,11 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
   const long long tok0 = begin + tile0, place = tok0 / CD_TILE + req;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dim = p.dim, vdim = p.vdim, kh = h / (p.heads / p.qk_heads);
+  // work of the last part: pairs of columns of the triangular system (key channels, then values), then pairs of key
+  // channels once more
+  const int value_cols = cd_col_tiles(vdim) * CW_COLS, items = DP + value_cols / 2;
+  float* v_s = g_s + CD_TILE * DP;           // [16][value_cols]
+  const float b_own = tid < tt ? to_f32<T>(b[(tok0 + tid) * p.ld_b + h]) : 0.f;
   const float rate = expf(a_log[h]);
   // a missing token is the identity: no write, no decay
   if (p.vec) {
@@ -269,7 +274,19 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
       g_s[e] = g;
     }
   }
-  if (tid < CD_TILE) beta_s[tid] = tid < tt ? 1.f / (1.f + expf(-to_f32<T>(b[(tok0 + tid) * p.ld_b + h]))) : 0.f;
+  if (p.vec && vdim % 4 == 0) {
+    for (int e = tid; e < CD_TILE * value_cols / 4; e += CD_THREADS) {
+      const int t = e / (value_cols / 4), c = (e - t * (value_cols / 4)) * 4;
+      reinterpret_cast<float4*>(v_s)[e] = t < tt && c < vdim ? load4<T>(qkv + (tok0 + t) * p.ld_qkv + p.v_off + (long long)h * vdim + c)
+                                                             : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  } else {
+    for (int e = tid; e < CD_TILE * value_cols; e += CD_THREADS) {
+      const int t = e / value_cols, c = e - t * value_cols;
+      v_s[e] = t < tt && c < vdim ? to_f32<T>(qkv[(tok0 + t) * p.ld_qkv + p.v_off + (long long)h * vdim + c]) : 0.f;
+    }
+  }
+  if (tid < CD_TILE) beta_s[tid] = tid < tt ? 1.f / (1.f + expf(-b_own)) : 0.f;
   __syncthreads();
   const float q_unit = 1.0f / sqrtf((float)dim);
 #pragma unroll
@@ -321,63 +338,68 @@ channel_delta_prepare_kernel(const T* __restrict__ qkv, const T* __restrict__ b,
         c += __shfl_xor_sync(0xffffffffu, c, o);
       }
       if (sl == 0) {
-        A_s[t][j] = t > j ? a : 0.f;
-        B_s[t][j] = t >= j ? c : 0.f;
+        A_s[t][j] = t > j ? make_float2(-a, -a) : make_float2(0.f, 0.f);
+        B_s[t][j] = t >= j ? make_float2(c, c) : make_float2(0.f, 0.f);
       }
     }
     if (sl == 0) {                             // what the loop did not reach
       for (int t = 0; t < CD_TILE; ++t)
-        if (t < j_first || t >= tt) A_s[t][j] = B_s[t][j] = 0.f;
+        if (t < j_first || t >= tt) A_s[t][j] = B_s[t][j] = make_float2(0.f, 0.f);
     }
   }
   __syncthreads();
   float* wh = ws_head + (place * p.heads + h) * cd_head_floats(dim);
-  const int tiles = cd_col_tiles(vdim);
-  float* wuo = ws_uo + (place * p.heads + h) * (long long)tiles * CD_UO;
-  // columns of the triangular system: the key channels, then the value columns
-  for (int c = tid; c < DP + tiles * CW_COLS; c += CD_THREADS) {
-    float x[CD_TILE];
-    if (c < DP) {
-      float run = 1.f;
-#pragma unroll
-      for (int t = 0; t < CD_TILE; ++t) {
-        run *= g_s[t * DP + c];
-        float r = run * k_s[t * DP + c];
-#pragma unroll
-        for (int j = 0; j < t; ++j) r = fmaf(-A_s[t][j], x[j], r);
-        x[t] = beta_s[t] * r;
-        wh[t * DP + c] = x[t];
-        float pr = run * q_s[t * DP + c];
-#pragma unroll
-        for (int j = 0; j <= t; ++j) pr = fmaf(-B_s[t][j], x[j], pr);
-        wh[(CD_TILE + t) * DP + c] = pr;
-      }
-      wh[3 * CD_TILE * DP + c] = run;
-      float after = 1.f;
+  float* wuo = ws_uo + (place * p.heads + h) * (long long)value_cols * 2 * CD_TILE;
+  const ulonglong2* A2 = reinterpret_cast<const ulonglong2*>(A_s);      // [t][j / 2]
+  const ulonglong2* B2 = reinterpret_cast<const ulonglong2*>(B_s);
+  for (int item = tid; item < items; item += CD_THREADS) {
+    if (item >= DP / 2 + value_cols / 2) {     // a pair of key channels: what a token's write is worth at the tile's end
+      const int c = 2 * (item - DP / 2 - value_cols / 2);
+      uint64_t after = pair_of(1.f, 1.f);
 #pragma unroll
       for (int t = CD_TILE - 1; t >= 0; --t) {
-        wh[(2 * CD_TILE + t) * DP + c] = after * k_s[t * DP + c];
-        after *= g_s[t * DP + c];
+        const uint64_t k = *reinterpret_cast<const uint64_t*>(k_s + t * DP + c), g = *reinterpret_cast<const uint64_t*>(g_s + t * DP + c);
+        *reinterpret_cast<uint64_t*>(wh + (2 * CD_TILE + t) * DP + c) = mul_pair(after, k);
+        after = mul_pair(after, g);
       }
-    } else {
-      const int col = c - DP;
-      float* dst = wuo + (col / CW_COLS) * CD_UO + col % CW_COLS;
-      float v[CD_TILE];
+      *reinterpret_cast<uint64_t*>(wh + 3 * CD_TILE * DP + c) = after;
+      continue;
+    }
+    // two columns of the triangular system side by side, the second product behind it
+    const bool key = item < DP / 2;
+    const int c = key ? 2 * item : 2 * (item - DP / 2);
+    float* dst = key ? wh + c : wuo + (c / CW_COLS) * CD_UO + c % CW_COLS;
+    const int ld = key ? DP : CW_COLS;
+    uint64_t x[CD_TILE], run = pair_of(1.f, 1.f);
 #pragma unroll
-      for (int t = 0; t < CD_TILE; ++t)
-        v[t] = (t < tt && col < vdim) ? to_f32<T>(qkv[(tok0 + t) * p.ld_qkv + p.v_off + (long long)h * vdim + col]) : 0.f;
-#pragma unroll
-      for (int t = 0; t < CD_TILE; ++t) {
-        float r = v[t];
-#pragma unroll
-        for (int j = 0; j < t; ++j) r = fmaf(-A_s[t][j], x[j], r);
-        x[t] = beta_s[t] * r;
-        dst[t * CW_COLS] = x[t];
-        float o = 0.f;
-#pragma unroll
-        for (int j = 0; j <= t; ++j) o = fmaf(B_s[t][j], x[j], o);
-        dst[(CD_TILE + t) * CW_COLS] = o;
+    for (int t = 0; t < CD_TILE; ++t) {
+      asm volatile("" ::: "memory");           // or all the tokens' loads would be moved up here and overflow the registers
+      uint64_t r, second;
+      if (key) {
+        run = mul_pair(run, *reinterpret_cast<const uint64_t*>(g_s + t * DP + c));
+        r = mul_pair(run, *reinterpret_cast<const uint64_t*>(k_s + t * DP + c));
+        second = mul_pair(run, *reinterpret_cast<const uint64_t*>(q_s + t * DP + c));
+      } else {
+        r = *reinterpret_cast<const uint64_t*>(v_s + t * value_cols + c);
+        second = 0;
       }
+#pragma unroll
+      for (int j = 0; j < t; j += 2) {         // A holds -A, and zero from the diagonal on
+        const ulonglong2 m = A2[t * (CD_TILE / 2) + j / 2];
+        r = fma_pair(m.x, x[j], r);
+        if (j + 1 < t) r = fma_pair(m.y, x[j + 1], r);
+      }
+      const float bt = beta_s[t];
+      x[t] = mul_pair(pair_of(bt, bt), r);
+      *reinterpret_cast<uint64_t*>(dst + t * ld) = x[t];
+      uint64_t o = 0;
+#pragma unroll
+      for (int j = 0; j <= t; j += 2) {
+        const ulonglong2 m = B2[t * (CD_TILE / 2) + j / 2];
+        o = fma_pair(m.x, x[j], o);
+        if (j + 1 <= t) o = fma_pair(m.y, x[j + 1], o);
+      }
+      *reinterpret_cast<uint64_t*>(dst + (CD_TILE + t) * ld) = key ? fma_pair(o, pair_of(-1.f, -1.f), second) : o;
     }
   }
 }
@@ -579,7 +601,8 @@ int launch_tiles_n(const void* qkv, const void* b, const float* z, const float* 
                    const int* cu_tokens, const int* slots, float* out, const ChannelDeltaArgs& p, int requests, int max_new,
                    float* ws_head, float* ws_uo, int* status, cudaStream_t stream) {
   constexpr int C = NI <= 4 ? 4 : 2;                          // columns per warp of the walk: what its registers hold
-  const size_t prep = (size_t)3 * CD_TILE * 32 * NI * sizeof(float);
+  const size_t prep = (size_t)CD_TILE * (3 * 32 * NI + cd_col_tiles(p.vdim) * CW_COLS) * sizeof(float);
+  HFEE_REQUIRE(prep <= 200 * 1024, "channel_delta: values of %d numbers per head do not fit shared memory", p.vdim);
   const size_t walk = (size_t)CW_STAGES * ((3 * CD_TILE + 1) * 32 * NI + CD_UO) * sizeof(float);
   if (prep > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(channel_delta_prepare_kernel<T, NI>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep);
@@ -633,7 +656,7 @@ HFEE_API int hfee_channel_delta(const void* qkv, long long ld_qkv, int q_off, in
   HFEE_REQUIRE(dim > 0 && dim <= CD_MAX_DIM && vdim > 0, "channel_delta: key size %d is outside 1..%d", dim, CD_MAX_DIM);
   HFEE_REQUIRE(requests <= 65535 && heads <= 65535, "channel_delta: too many requests or heads");
   HFEE_REQUIRE(dtype == HFEE_F32 || dtype == HFEE_BF16, "channel_delta: unknown dtype %d", dtype);
-  const int vec = dim % 4 == 0 && ld_qkv % 4 == 0 && ld_z % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 &&
+  const int vec = dim % 4 == 0 && ld_qkv % 4 == 0 && ld_z % 4 == 0 && q_off % 4 == 0 && k_off % 4 == 0 && v_off % 4 == 0 &&
                   (uintptr_t)qkv % (dtype == HFEE_F32 ? 16 : 8) == 0 && (uintptr_t)z % 16 == 0 && (uintptr_t)dt_bias % 16 == 0;
   const ChannelDeltaArgs p{ld_qkv, ld_b, ld_z, ld_out, q_off, k_off, v_off, heads, qk_heads, dim, vdim, write_state, vec};
   if (max_new == 1) {
