@@ -245,7 +245,7 @@ def _latent_attention(args) -> dict:
     pool = torch.randn(b.r * max_pages, 1, page, dk, device=DEV).to(torch.bfloat16)
     q = (torch.randn(b.n, heads * dk, device=DEV) * 0.3).to(torch.bfloat16)
     out = torch.empty(b.n, heads * rank, dtype=torch.bfloat16, device=DEV)
-    ops.USE_LATENT_MMA = not args.no_tc_attention
+    ops.USE_LATENT_TC = not args.no_tc_attention
     scratch = torch.empty(160 * heads * (rank + 2), device=DEV)
     b.planning_context, b.attention_splits = b.max_context, args.splits or None
     fn = lambda i: ops.latent_attention(q, pool, table, page, b, out, heads, dk, rank, dk ** -0.5, window, None, scratch)

@@ -67,6 +67,8 @@ _SIGNATURES = {
                              _I, _I, _I, _P, _I, _P, _I, _I, _P],
     "hfee_latent_norm_rope_cache": [_P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _P, _F, _P, _P, _P, _P, _L, _P, _P, _I, _I, _P],
     "hfee_latent_attention_mma": [_P, _L, _P, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _I, _P],
+    "hfee_latent_attention_tc": [_P, _L, _P, _I, _P, _I, _I, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P, _P],
+    "hfee_latent_attention_tc_supports": [_I, _I, _I, _I],
     "hfee_latent_attend_prepare": [_P, _L, _I, _I, _I, _I, _I, _I, _P, _F, _P, _P, _P, _I, _I, _I, _P, _L, _I, _I, _P, _P, _I, _I, _P],
     "hfee_stream_step": [_P, _L, _L, _P, _L, _P, _P, _P, _P, _P, _F, _I, _P, _P, _I, _P, _P, _I, _P, _P, _L, _I, _I, _I, _I, _P],
     "hfee_channel_delta": [_P, _L, _I, _I, _I, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _I, _P, _L, _P, _P],
@@ -1115,9 +1117,25 @@ def latent_attention(q: torch.Tensor, k_pool: torch.Tensor, block_table: torch.T
     """Softmax attention of ``heads`` query heads over ONE cached vector per token (``k_pool`` [pages, 1, page_size,
     cached_dim]) whose leading ``value_dim`` dimensions are also the values: ``out`` [n, heads * value_dim].
     ``sink`` (float32 per head): the denominator also holds exp(sink[h]).  ``scratch`` (float32) lets a step of single
-    tokens split its keys among CTAs.  bfloat16 with sizes the tensor-core kernel takes runs there (prompt portions and decode steps alike),
-    everything else on the CUDA cores in float32."""
+    tokens split its keys among CTAs.  bfloat16 runs on the tensor cores where the sizes allow it (portions of LATENT_TC_MIN_ROWS
+    (token, head) rows and more on tcgen05, shorter ones and decode steps on ``mma.sync`` tiles), everything else on the CUDA cores in float32."""
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == heads)
+    if (USE_LATENT_TC and q.dtype == torch.bfloat16 and step.max_new * heads >= LATENT_TC_MIN_ROWS and scale > 0
+            and latent_tc_supports(heads, cached_dim, value_dim, page_size) and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0
+            and _rows(out, "out") % 8 == 0 and out.data_ptr() % 16 == 0):
+        lib = library()
+        for t, what in ((block_table, "block_table"), (step.cu_tokens, "cu_tokens"), (step.slots, "slots"),
+                        (step.context_before, "context_before")):
+            _i32(t, what)
+        assert k_pool.dtype == out.dtype == torch.bfloat16 and k_pool.is_contiguous()
+        assert tuple(k_pool.shape[1:]) == (1, page_size, cached_dim)
+        assert tuple(q.shape) == (step.n, heads * cached_dim) and tuple(out.shape) == (step.n, heads * value_dim)
+        _check(lib.hfee_latent_attention_tc(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), k_pool.shape[0], block_table.data_ptr(),
+                                            block_table.shape[1], page_size, step.cu_tokens.data_ptr(), step.slots.data_ptr(),
+                                            step.context_before.data_ptr(), out.data_ptr(), _rows(out, "out"), step.n, step.r,
+                                            step.max_new, heads, cached_dim, value_dim, float(scale), int(window or 0), _ptr(sink),
+                                            _status().data_ptr(), _stream()), lib)
+        return
     if (USE_LATENT_MMA and q.dtype == torch.bfloat16 and latent_mma_supports(heads, cached_dim, value_dim)
             and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0 and _rows(out, "out") % 2 == 0 and out.data_ptr() % 4 == 0):
         lib = library()
@@ -1164,7 +1182,18 @@ def latent_splits(requests: int, heads: int, max_context: int, window: int) -> i
     return max(1, min(MAX_SPLITS, sm_count() // max(1, requests * -(-heads // 64)), keys // 128))
 
 
-USE_LATENT_MMA = True
+USE_LATENT_MMA = USE_LATENT_TC = True
+LATENT_TC_MIN_ROWS = 128
+_LATENT_TC_TAKES: dict = {}
+
+
+def latent_tc_supports(heads: int, cached_dim: int, value_dim: int, page_size: int) -> bool:
+    key = (heads, cached_dim, value_dim, page_size)
+    if key not in _LATENT_TC_TAKES:
+        _LATENT_TC_TAKES[key] = bool(library().hfee_latent_attention_tc_supports(*key))
+    return _LATENT_TC_TAKES[key]
+
+
 _LATENT_MMA_TAKES: dict = {}
 
 

@@ -239,3 +239,45 @@ def test_latent_attention_with_a_sink(dtype, heads, dk, dv, window, level):
             step.attention_splits, step.planning_context = splits, step.max_context
             ops.latent_attention(q, pool, table, page, step, out, heads, dk, dv, 0.2, window, dev_sink, scratch)
             assert np.max(np.abs(host(out) - ref)) <= tol * max(scale, 1e-3), (counts, splits)
+
+
+@pytest.mark.parametrize("heads,dk,dv,window", [(8, 96, 64, 0), (32, 288, 256, 0), (3, 144, 128, 70), (128, 80, 64, 0), (5, 576, 512, 0),
+                                                (16, 320, 320, 33), (1, 64, 64, 0)])
+@pytest.mark.parametrize("page", [64, 128])
+def test_latent_attention_of_prompt_portions(heads, dk, dv, window, page):
+    """The tcgen05 kernel: portions that start at 0, inside a key block and at its edge, beside a single token and a short
+    portion; pages in any order with stale not-a-numbers wherever no key of the request lies; sinks of every size."""
+    from hfee_b200.kernels import ops
+    rng = np.random.default_rng(dk + heads)
+    assert ops.latent_tc_supports(heads, dk, dv, page)
+    before, new = [0, 64, 131, 200], [150, 67, 1, 9]
+    pages = 4
+    table = torch.tensor(rng.permutation(4 * pages).reshape(4, pages), dtype=torch.int32, device=DEV)
+    pool = torch.full((4 * pages, 1, page, dk), float("nan"), dtype=torch.bfloat16, device=DEV)
+    keys = [dev(rng.normal(size=(b + n, dk)), torch.bfloat16) for b, n in zip(before, new)]
+    for r in range(4):
+        for p in range(before[r] + new[r]):
+            pool[table[r, p // page], 0, p % page] = keys[r][p]
+    step = make_step(new, lengths=before, slots=[0, 1, 2, 3])
+    q = dev(rng.normal(size=(step.n, heads * dk)), torch.bfloat16)
+    qh, scale = q.float().reshape(step.n, heads, dk), 2.0 * dk ** -0.5
+    for level in (None, 0.0, 40.0):
+        sink = None if level is None else dev(level + rng.normal(size=heads))
+        want, at = [], 0
+        for r in range(4):
+            k = keys[r].float()
+            s = torch.einsum("thd,kd->htk", qh[at:at + new[r]].double(), k.double()) * scale
+            pos = torch.arange(before[r], before[r] + new[r], device=DEV)[:, None]
+            j = torch.arange(k.shape[0], device=DEV)[None]
+            s = s.masked_fill(~((j <= pos) & ((j > pos - window) if window else (j >= 0)))[None], -torch.inf)
+            if sink is not None:
+                s = torch.cat([s, sink.double()[:, None, None].expand(heads, new[r], 1)], dim=2)
+            w = torch.softmax(s, dim=2)[:, :, :k.shape[0]]
+            want.append(torch.einsum("htk,kd->thd", w, k[:, :dv].double()).reshape(new[r], heads * dv))
+            at += new[r]
+        want = torch.cat(want)
+        out = torch.full((step.n, heads * dv), 9.0, dtype=torch.bfloat16, device=DEV)
+        ops.latent_attention(q, pool, table, page, step, out, heads, dk, dv, scale, window, sink)
+        err = (out.double() - want).abs()
+        assert torch.isfinite(out).all() and float(err.max()) <= 1.5e-2 * max(float(want.abs().max()), 1e-2), level
+    ops.check_status()
