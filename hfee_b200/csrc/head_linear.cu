@@ -68,7 +68,7 @@ __device__ __forceinline__ void hm_cp_async16(void* smem, const void* gmem, bool
 __global__ void __launch_bounds__(HM_THREADS)
 head_linear_mma_kernel(const bf16* __restrict__ in, long long ld_in, int in_off, int in_stride, const bf16* __restrict__ w,
                        bf16* __restrict__ out, long long ld_out, int out_off, int out_stride, int n, int n_in, int n_out,
-                       const bf16* __restrict__ gate, long long ld_gate) {
+                       const bf16* __restrict__ gate, long long ld_gate, int wide) {
   __shared__ __align__(16) bf16 a_s[HM_TILE * HM_LD];
   __shared__ __align__(16) bf16 b_s[HM_TILE * HM_LD];
   pdl_wait();
@@ -110,23 +110,36 @@ head_linear_mma_kernel(const bf16* __restrict__ in, long long ld_in, int in_off,
       mma_bf16(acc[1][2], a1, b1[0], b1[1]); mma_bf16(acc[1][3], a1, b1[2], b1[3]);
     }
   }
+  if (wide) __syncthreads();                             // the last operand tiles have been read: a_s takes the result
 #pragma unroll
   for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-      const int row = row0 + wr + mt * 16 + (lane >> 2) + 8 * half;
+      const int r = wr + mt * 16 + (lane >> 2) + 8 * half, row = row0 + r;
       if (row >= n) continue;
       float gv = 1.f;
       if (gate != nullptr) gv = 1.f / (1.f + expf(-__bfloat162float(gate[(long long)row * ld_gate + h])));
       bf16* dst = out + (long long)row * ld_out + out_off + (long long)h * out_stride;
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int col = col0 + wc + nt * 8 + 2 * (lane & 3) + e;
-          if (col < n_out) dst[col] = __float2bfloat16_rn(acc[mt][nt][2 * half + e] * gv);
+      for (int nt = 0; nt < 4; ++nt) {
+        const int c = wc + nt * 8 + 2 * (lane & 3);
+        const __nv_bfloat162 v = __floats2bfloat162_rn(acc[mt][nt][2 * half] * gv, acc[mt][nt][2 * half + 1] * gv);
+        if (wide) {
+          *reinterpret_cast<__nv_bfloat162*>(a_s + r * HM_LD + c) = v;
+        } else {
+          if (col0 + c < n_out) dst[col0 + c] = v.x;
+          if (col0 + c + 1 < n_out) dst[col0 + c + 1] = v.y;
         }
+      }
     }
+  if (!wide) return;
+  __syncthreads();
+  for (int e = tid; e < HM_TILE * (HM_TILE / 8); e += HM_THREADS) {       // 16 bytes a thread, a tile's row by eight neighbours
+    const int r = e / (HM_TILE / 8), c = (e % (HM_TILE / 8)) * 8;
+    if (row0 + r < n && col0 + c < n_out)
+      *reinterpret_cast<uint4*>(out + (long long)(row0 + r) * ld_out + out_off + (long long)h * out_stride + col0 + c) =
+          *reinterpret_cast<const uint4*>(a_s + r * HM_LD + c);
+  }
 }
 
 bool head_linear_mma_takes(const void* in, long long ld_in, int in_off, int in_stride, const void* w, int n_in) {
@@ -158,9 +171,11 @@ HFEE_API int hfee_head_linear(const void* in, long long ld_in, int in_off, int i
   if (dtype == HFEE_F32)
     return launch_head_linear<float>(in, ld_in, in_off, in_stride, w, out, ld_out, out_off, out_stride, n, heads, n_in, n_out, gate, ld_gate, stream);
   if (dtype == HFEE_BF16 && head_linear_mma_takes(in, ld_in, in_off, in_stride, w, n_in)) {
+    // rows of the output that start on 16 bytes and hold whole 16-byte pieces leave through shared memory
+    const int wide = n_out % 8 == 0 && ld_out % 8 == 0 && out_off % 8 == 0 && out_stride % 8 == 0 && (uintptr_t)out % 16 == 0;
     hfee_launch(head_linear_mma_kernel, dim3((unsigned)((n + HM_TILE - 1) / HM_TILE), (unsigned)((n_out + HM_TILE - 1) / HM_TILE), (unsigned)heads),
                 dim3(HM_THREADS), 0, stream, (const bf16*)in, ld_in, in_off, in_stride, (const bf16*)w, (bf16*)out, ld_out, out_off,
-                out_stride, n, n_in, n_out, (const bf16*)gate, ld_gate);
+                out_stride, n, n_in, n_out, (const bf16*)gate, ld_gate, wide);
     return hfee_check_launch("head_linear_mma");
   }
   if (dtype == HFEE_BF16)

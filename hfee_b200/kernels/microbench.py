@@ -13,6 +13,7 @@ where that matters, and prints what it achieved against the roofline that bounds
     python -m hfee_b200.kernels.microbench delta_rule        --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64 [--decode --batch 8]
     python -m hfee_b200.kernels.microbench channel_delta     --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64 [--decode --batch 8]
     python -m hfee_b200.kernels.microbench stream_step       --tokens 2048 --k 2048 --streams 4
+    python -m hfee_b200.kernels.microbench latent_prepare    --tokens 2048 --heads 32 --head-dim 64 --rank 256
     python -m hfee_b200.kernels.microbench conv_act          --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64
     python -m hfee_b200.kernels.microbench latent_attention  --tokens 2048 --heads 32 --head-dim 64 --rank 256 --window 512 [--decode --batch 8]
     python -m hfee_b200.kernels.microbench head_linear       --tokens 2048 --heads 32 --head-dim 64 --rank 256
@@ -502,6 +503,24 @@ def _stream_step(args) -> dict:
     return res
 
 
+def _latent_prepare(args) -> dict:
+    """Between the projection of a latent attention without a query latent and its scores: latent norm, rotations, cache."""
+    heads, d, rank, page, n = args.heads, args.head_dim, args.rank, args.page_size, args.tokens
+    r = d // 2
+    b = _batch_of([0], [n])
+    cols = heads * (d + r) + rank + r
+    proj = torch.randn(n, cols, device=DEV).to(torch.bfloat16)
+    pages = -(-n // page)
+    table = torch.arange(pages, dtype=torch.int32, device=DEV).reshape(1, pages)
+    pool = torch.zeros(pages, 1, page, rank + r, dtype=torch.bfloat16, device=DEV)
+    q = torch.zeros(n, heads * (rank + r), dtype=torch.bfloat16, device=DEV)
+    cs, w = torch.rand(n, r // 2, 2, device=DEV), torch.ones(rank, device=DEV)
+    sec = _time(lambda i: ops.latent_attend_prepare(proj, heads * (d + r), rank, r, True, w, 1e-5, cs, b, heads, d, d + r, q, rank,
+                                                    rank + r, pool, table, page), args.warmup, args.iters)
+    moved = n * 4 * (heads * r + rank + r)
+    return {"kernel": "latent_prepare", "tokens": n, "heads": heads, "rank": rank, "us": round(sec * 1e6, 2), "gbs": round(moved / sec / 1e9, 1)}
+
+
 def _pupinex_rows(args) -> dict:
     """Row kernels of the Pupinex parts on ``--tokens`` rows of width ``--k``: layer norm, the bigram embedding, the bias,
     the step between the q/k/v projection and the attention, and the per-head norm with its gate."""
@@ -549,7 +568,7 @@ def main(argv=None) -> int:
                                        "gemm_tcgen05", "gemm_stream", "gemm_skinny", "gemm_ring", "gemm_pair", "attention_decode", "attention_prefill",
                                       "sigmoid_attention", "linear_attention", "mingru", "selective_scan",
                                        "distance_attention", "moe_experts", "row_ops", "softmax_attention", "gla", "matrix_memory",
-                                       "pupinex_rows", "channel_delta", "stream_step"])
+                                       "pupinex_rows", "channel_delta", "stream_step", "latent_prepare"])
     ap.add_argument("--m", type=int, default=2048)
     ap.add_argument("--n", type=int, default=16384)
     ap.add_argument("--k", type=int, default=2048)
@@ -605,8 +624,8 @@ def main(argv=None) -> int:
         res = _softmax_attention(args)
     elif args.kernel in ("gla", "matrix_memory"):
         res = _gated_recurrence(args, 0 if args.kernel == "gla" else 1)
-    elif args.kernel in ("channel_delta", "stream_step"):
-        res = {"channel_delta": _channel_delta, "stream_step": _stream_step}[args.kernel](args)
+    elif args.kernel in ("channel_delta", "stream_step", "latent_prepare"):
+        res = {"channel_delta": _channel_delta, "stream_step": _stream_step, "latent_prepare": _latent_prepare}[args.kernel](args)
     elif args.kernel == "pupinex_rows":
         res = _pupinex_rows(args)
     else:

@@ -2099,6 +2099,7 @@ for _name in ("rmsnorm_add_norm", "latent_attention", "linear_act", "attention_s
               "qk_norm_rope_cache", "embed", "rmsnorm", "rope_table", "rope_cache_write", "swiglu", "linear", "linear_normed", "linear_swiglu", "linear_rope_cache",
               "linear_swiglu_normed", "paged_attention", "paged_attention_rope", "sample", "argmax", "sample_chain",
               "mingru", "selective_scan", "distance_attention", "moe_route", "moe_plan", "moe_experts", "moe_experts_grouped", "moe_combine",
-              "clamped_glu", "linear_clamped_glu", "depth_average", "scaled_add_norm", "scaled_add", "add_sinusoid", "softcap_"):
+              "clamped_glu", "linear_clamped_glu", "depth_average", "scaled_add_norm", "scaled_add", "add_sinusoid", "softcap_",
+              "channel_delta", "stream_step", "latent_attend_prepare"):
     globals()[_name] = _measurable(globals()[_name])
 del _name
