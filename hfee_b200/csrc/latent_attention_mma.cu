@@ -305,41 +305,41 @@ latent_attention_kernel(LatentParams p) {
     }
 }
 
-// One (token, head) per warp: the shares' outputs against the largest of their maxima (and the sink's).
-__global__ void __launch_bounds__(128)
+// A block per (token, head), a thread per pair of value columns: the shares' outputs against the largest of their maxima
+// (and the sink's).
+constexpr int LC_THREADS = 128;
+__global__ void __launch_bounds__(LC_THREADS)
 latent_combine_kernel(const float* __restrict__ partial, int splits, int n_tokens, int heads, int dv, const float* __restrict__ sink,
                       bf16* __restrict__ out, long long ld_o) {
+  __shared__ float w_s[32];
   pdl_wait();
   pdl_launch_dependents();
-  const int task = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (task >= n_tokens * heads) return;
-  const int t = task / heads, h = task - t * heads;
+  const int h = blockIdx.x, t = blockIdx.y, lane = threadIdx.x & 31;
   const long long stride = (long long)n_tokens * heads * (dv + 2);
-  const float* mine = partial + (long long)task * (dv + 2);
-  float m = -INFINITY, l = 0.f;                                // lane s: share s (at most 32 of them)
-  if (lane < splits) {
-    m = mine[lane * stride + dv];
-    l = mine[lane * stride + dv + 1];
-  }
-  float top = warp_max(m);
-  const float s2 = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
-  top = fmaxf(top, s2);
-  const float w = m == -INFINITY ? 0.f : la_exp2(m - top);
-  const float total = warp_sum(w * l) + (sink != nullptr ? la_exp2(s2 - top) : 0.f);
-  const float inv = total > 0.f ? 1.f / total : 0.f;
-  bf16* dst = out + (long long)t * ld_o + (long long)h * dv;
-  for (int base = 0; base < dv; base += 64) {                  // the same for all lanes: they hand their weights around
-    const int d = base + 2 * lane;
-    float a = 0.f, b = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float ws = __shfl_sync(0xffffffffu, w, s);
-      if (d < dv) {
-        const float2 v = *reinterpret_cast<const float2*>(mine + s * stride + d);
-        a = fmaf(ws, v.x, a);
-        b = fmaf(ws, v.y, b);
-      }
+  const float* mine = partial + ((long long)t * heads + h) * (dv + 2);
+  if (threadIdx.x < 32) {                                      // lane s: share s (at most 32 of them)
+    float m = -INFINITY, l = 0.f;
+    if (lane < splits) {
+      m = mine[lane * stride + dv];
+      l = mine[lane * stride + dv + 1];
     }
-    if (d < dv) *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(a * inv, b * inv);
+    const float s2 = sink != nullptr ? sink[h] * 1.4426950408889634f : -INFINITY;
+    const float top = fmaxf(warp_max(m), s2);
+    const float w = m == -INFINITY ? 0.f : la_exp2(m - top);
+    const float total = warp_sum(w * l) + (sink != nullptr ? la_exp2(s2 - top) : 0.f);
+    w_s[lane] = total > 0.f ? w / total : 0.f;
+  }
+  __syncthreads();
+  bf16* dst = out + (long long)t * ld_o + (long long)h * dv;
+  for (int d = 2 * threadIdx.x; d < dv; d += 2 * LC_THREADS) {
+    float a = 0.f, b = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < splits; ++s) {
+      const float2 v = *reinterpret_cast<const float2*>(mine + s * stride + d);
+      a = fmaf(w_s[s], v.x, a);
+      b = fmaf(w_s[s], v.y, b);
+    }
+    *reinterpret_cast<__nv_bfloat162*>(dst + d) = __floats2bfloat162_rn(a, b);
   }
 }
 
@@ -415,7 +415,7 @@ HFEE_API int hfee_latent_attention_mma(const void* q, long long ld_q, const void
     else rc = launch_latent<8, 1>(p, grid, stream);
   }
   if (rc != HFEE_OK || splits == 1) return rc;
-  hfee_launch(latent_combine_kernel, dim3((unsigned)(((long long)n_tokens * heads + 3) / 4)), dim3(128), 0, stream, partial, splits,
+  hfee_launch(latent_combine_kernel, dim3((unsigned)heads, (unsigned)n_tokens), dim3(LC_THREADS), 0, stream, partial, splits,
               n_tokens, heads, dv, sink, (bf16*)out, ld_o);
   return hfee_check_launch("latent_combine");
 }
