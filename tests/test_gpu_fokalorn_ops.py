@@ -241,7 +241,7 @@ def test_latent_attention_with_a_sink(dtype, heads, dk, dv, window, level):
             assert np.max(np.abs(host(out) - ref)) <= tol * max(scale, 1e-3), (counts, splits)
 
 
-@pytest.mark.parametrize("heads,dk,dv,window", [(8, 96, 64, 0), (32, 288, 256, 0), (3, 144, 128, 70), (128, 80, 64, 0), (5, 576, 512, 0),
+@pytest.mark.parametrize("heads,dk,dv,window", [(8, 112, 64, 0), (32, 288, 256, 0), (3, 144, 128, 70), (128, 80, 64, 0), (5, 576, 512, 0),
                                                 (16, 320, 320, 33), (1, 64, 64, 0)])
 @pytest.mark.parametrize("page", [64, 128])
 def test_latent_attention_of_prompt_portions(heads, dk, dv, window, page):
