@@ -406,3 +406,14 @@ def test_command_line_generates(models):
     draws = [subprocess.run(base + ["--temperature", "0.9", "--top-k", "20", "--seed", "7"], capture_output=True, text=True,
                             timeout=300).stdout.split("\n")[0] for _ in range(2)]
     assert draws[0] == draws[1] and len(draws[0].split()) == 6
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_pages_of_64(models, dtype):
+    """Pages that the tcgen05 attention takes: long portions beside short ones and single tokens, in and across key blocks."""
+    d, cfg, _, _ = models["B"]
+    c, w = plain.load(d)
+    seqs = fu.sequences(cfg["vocab"], (300, 130, 65, 64), seed=12)
+    ref = [plain.forward(c, w, s) for s in seqs]
+    for steps in (ru.whole(seqs), ru.portions(seqs, sizes=(130, 2, 63, 1, 64)), ru.mixed(seqs, live=3, seed=4, chunk_sizes=(2, 40, 64, 90))):
+        check(ru.run_in_process(fu.make_runner(d, dtype, 10 * 64, page_size=64, max_requests=3, context=320), steps), ref, dtype)
