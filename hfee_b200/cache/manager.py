@@ -8,7 +8,7 @@ a paged group owns a pool of pages (one page id addresses the page in every cach
 of the group) and one block table ``[max_requests, max_pages]`` whose row is the
 request's slot; a state group owns ``[max_requests, ...]`` rows.  Pages go back to
 the pool when a request is closed or, in a windowed group, once the window has
-passed them.
+passed them (pages of first positions that stay visible behind the window are held until then).
 """
 from __future__ import annotations
 
@@ -47,7 +47,9 @@ class _PagedGroup:
         self.pool = PagePool(num_pages)
         self.page_size = page_size
         self.table = np.full((max_requests, max_pages), -1, dtype=np.int32)
-        self.first_live = [0] * max_requests       # logical pages [first_live, held_to) are held
+        # logical pages [first_live, held_to) are held, and so are the first ``kept_pages``
+        self.kept_pages = -(-int(need.keep_first) // page_size) if need.window is not None else 0
+        self.first_live = [0] * max_requests
         self.held_to = [0] * max_requests
         self.dirty = True
         shape = (len(cache_ids), num_pages, need.kv_heads, page_size, need.head_dim)
@@ -63,7 +65,7 @@ class _PagedGroup:
         self.staging_turn = 0
 
     def first_needed_page(self, length: int) -> int:
-        """First logical page a token at position >= ``length`` can still read."""
+        """First logical page a token at position >= ``length`` can still read (the kept first pages aside)."""
         lowest = 0
         if self.need.window is not None:
             lowest = max(0, length - int(self.need.window) + 1) // self.page_size
@@ -182,11 +184,12 @@ class CacheManager:
         self.length[slot] = new_length
         for g in self.paged:
             first = min(g.first_needed_page(new_length), g.held_to[slot])
-            if first > g.first_live[slot]:
+            start = max(g.first_live[slot], g.kept_pages)
+            if first > start:
                 row = g.table[slot]
-                gone = [int(p) for p in row[g.first_live[slot]:first] if p >= 0]
+                gone = [int(p) for p in row[start:first] if p >= 0]
                 g.pool.give_back(gone)
-                row[g.first_live[slot]:first] = -1
+                row[start:first] = -1
                 g.first_live[slot] = first
                 g.dirty = True
 
@@ -257,7 +260,8 @@ class CacheManager:
                     seen[p] = (slot, logical)
                 if self.open_slots[slot]:
                     need_to = -(-self.length[slot] // self.page_size)
-                    for logical in range(g.first_needed_page(self.length[slot]), need_to):
+                    first = g.first_needed_page(self.length[slot])
+                    for logical in [*range(min(g.kept_pages, first, need_to)), *range(first, need_to)]:
                         if row[logical] < 0:
                             raise AssertionError(f"slot {slot} has no page for logical page {logical}")
             if len(seen) + g.pool.free_pages != g.pool.num_pages:

@@ -10,6 +10,7 @@ class PagedKV:
     """Keys and values for every cached position (or, with ``window``, for the last
     ``window`` positions only; with ``chunk``, for the positions of the current block of
     ``chunk`` positions counted from 0 only), stored in pages of ``page_size`` tokens.
+    ``keep_first``: beside a window, the first ``keep_first`` positions stay cached as long as the request.
     ``value_dim``: size of a cached value; None = ``head_dim``; 0 = nothing is cached beside the keys (the
     values are read out of the cached keys, as with a latent that serves as both)."""
     kv_heads: int
@@ -17,6 +18,7 @@ class PagedKV:
     window: Optional[int] = None
     chunk: Optional[int] = None
     value_dim: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

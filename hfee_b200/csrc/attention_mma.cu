@@ -51,6 +51,9 @@ struct AttnParams {
   const float* dist_r1; const float* dist_r2;     // both null: no penalty
   float out_scale;
   const float* sink;           // DIST only: per query head, one more term exp(sink[h]) of the softmax's denominator; null: none
+  int keep_first;              // DIST only: this many positions from the start stay visible behind the window
+  float cap_log2;              // DIST only: > 0: the score becomes cap * tanh(score / cap); cap in log2 units, and
+  float cap_in;                //   2 * log2(e) * scale / cap, which turns q.k into the exponent of e^(2 score / cap)
 };
 
 // Rotates the 16-byte piece of a head that starts at dim `a` (a multiple of 8): pairs (i, i + half)
@@ -126,6 +129,11 @@ __device__ __forceinline__ float fast_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float fast_reciprocal(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&v);
@@ -172,8 +180,14 @@ attention_mma_kernel(AttnParams p) {
   const int key_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
   const int rows_used = t_count * p.group;
 
-  // key blocks of this CTA
+  // Key blocks of this CTA, numbered b_lo .. b_hi.  Where first positions stay visible behind the window, their n_front
+  // blocks come in front of the window's: number v is block v below n_front, block v + skip from there on.
   int b_lo = key_lo / BLOCK_N, b_hi = pos_last / BLOCK_N;
+  const int kept = DIST ? min(p.keep_first, key_lo) : 0;
+  const int n_front = DIST ? min((kept + BLOCK_N - 1) / BLOCK_N, b_lo) : 0;
+  const int skip = DIST && n_front > 0 ? b_lo - n_front : 0;
+  if (DIST && n_front > 0) { b_lo = 0; b_hi -= skip; }
+  auto block_of = [&](int v) { return DIST && v >= n_front ? v + skip : v; };
   if (p.num_splits > 1) {
     // The launch (and a captured graph) fixes the number of splits for the longest context the
     // engine allows; a shorter context uses only as many of them as leave each at least two key
@@ -196,7 +210,7 @@ attention_mma_kernel(AttnParams p) {
   else if (wrow + 15 >= rows_used) row_pos_min = -1;          // padding rows in the tile: keep masking
 
   if (b_lo <= b_hi && tid <= b_hi - b_lo) {
-    int warm = p.cache.block_table[(long long)slot * p.cache.max_pages + (b_lo + tid) * BLOCK_N / p.cache.page_size];
+    int warm = p.cache.block_table[(long long)slot * p.cache.max_pages + block_of(b_lo + tid) * BLOCK_N / p.cache.page_size];
     asm volatile("" ::"r"(warm));
   }
   // A block's 64 rows x CHUNKS 16-byte pieces are spread over the threads.  Page ids are looked
@@ -221,7 +235,7 @@ attention_mma_kernel(AttnParams p) {
         const int idx = tid + i * THREADS;
         const int row = idx / CHUNKS, ch = idx % CHUNKS;
         const int pos = pos0 + row;
-        ok[i] = idx < BLOCK_N * CHUNKS && pos >= key_lo && pos <= pos_last;
+        ok[i] = idx < BLOCK_N * CHUNKS && (pos >= key_lo || pos < kept) && pos <= pos_last;
         off[i] = ok[i] ? (DIST ? base + row : base + (long long)row * HD + ch * 8) : 0;
       }
     } else {
@@ -230,7 +244,7 @@ attention_mma_kernel(AttnParams p) {
         const int idx = tid + i * THREADS;
         const int row = idx / CHUNKS, ch = idx % CHUNKS;
         const int pos = block * BLOCK_N + row;
-        ok[i] = idx < BLOCK_N * CHUNKS && pos >= key_lo && pos <= pos_last;
+        ok[i] = idx < BLOCK_N * CHUNKS && (pos >= key_lo || pos < kept) && pos <= pos_last;
         off[i] = ok[i] ? (DIST ? paged_offset(p.cache, slot, pos, kvh) / p.cache.head_dim
                                : paged_offset(p.cache, slot, pos, kvh) + ch * 8) : 0;
       }
@@ -285,8 +299,8 @@ attention_mma_kernel(AttnParams p) {
   int requested = 0;
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) {
-    if (requested == i && b_lo + i <= b_hi && (b_lo + i + 1) * BLOCK_N <= before) {
-      load_kv(b_lo + i, i);
+    if (requested == i && b_lo + i <= b_hi && (block_of(b_lo + i) + 1) * BLOCK_N <= before) {
+      load_kv(block_of(b_lo + i), i);
       cp_async_commit();
       ++requested;
     }
@@ -319,7 +333,7 @@ attention_mma_kernel(AttnParams p) {
   // The new token's key (rotated) and value: held in registers by the first threads of the CTA whose
   // key range ends at the new position, written to the cache now and into the shared-memory tile
   // once that block's copy from the cache (which holds nothing valid for this row yet) has landed.
-  const bool patch_cta = fused_rope && p.k_write != nullptr && b_lo <= b_hi && pos_last / BLOCK_N == b_hi;
+  const bool patch_cta = fused_rope && p.k_write != nullptr && b_lo <= b_hi && pos_last / BLOCK_N == block_of(b_hi);
   uint4 new_k0 = make_uint4(0, 0, 0, 0), new_k1 = new_k0, new_v = new_k0;
   int new_k_pieces = 0;
   if (patch_cta && tid < 2 * CHUNKS) {
@@ -339,14 +353,14 @@ attention_mma_kernel(AttnParams p) {
 #pragma unroll
   for (int i = 0; i < STAGES - 1; ++i) {
     if (i >= requested) {
-      if (b_lo + i <= b_hi) load_kv(b_lo + i, i);
+      if (b_lo + i <= b_hi) load_kv(block_of(b_lo + i), i);
       cp_async_commit();
     }
   }
 
   for (int b = b_lo; b <= b_hi; ++b) {
     int stage = (b - b_lo) % STAGES;
-    if (b + STAGES - 1 <= b_hi) load_kv(b + STAGES - 1, (b - b_lo + STAGES - 1) % STAGES);
+    if (b + STAGES - 1 <= b_hi) load_kv(block_of(b + STAGES - 1), (b - b_lo + STAGES - 1) % STAGES);
     cp_async_commit();
     cp_async_wait<STAGES - 1>();
     __syncthreads();
@@ -373,6 +387,7 @@ attention_mma_kernel(AttnParams p) {
       for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < HD / 16; ++ks) {
+      if (DIST && ks * 16 >= kdim) break;                 // tiles are as wide as the larger of the two sizes
       uint32_t a[4];
       ldmatrix_x4(a, q_s + (wrow + (lane & 15)) * PITCH + ks * 16 + (lane >> 4) * 8);
 #pragma unroll
@@ -386,7 +401,7 @@ attention_mma_kernel(AttnParams p) {
 
     // ---- mask (only in blocks that reach past a row's position or below its window), online
     // softmax on the raw scores: p = 2^(s*c - m*c) with c = scale*log2(e) folded into one FMA
-    const int key0 = b * BLOCK_N + wkey;                       // first key this warp visits in the block
+    const int key0 = block_of(b) * BLOCK_N + wkey;             // first key this warp visits in the block
     if constexpr (DIST) {
       if (p.dist_r1 != nullptr) {
 #pragma unroll
@@ -397,6 +412,13 @@ attention_mma_kernel(AttnParams p) {
             const float dist = (float)max(row_pos[h] - (key0 + nt * 8 + 2 * c + (j & 1)), 0);
             s[nt][j] = fmaf(s[nt][j], p.scale_log2, -row_r1[h] * __log2f(fmaf(row_r2[h], dist, 1.f)));
           }
+      } else if (p.cap_log2 > 0.f) {
+        // cap * tanh(x / cap) = cap - 2 cap / (e^(2x / cap) + 1): exact in both tails, some 1e-7 of the cap in between
+#pragma unroll
+        for (int nt = 0; nt < WKEYS / 8; ++nt)
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+            s[nt][j] = fmaf(-2.f * p.cap_log2, fast_reciprocal(fast_exp2(s[nt][j] * p.cap_in) + 1.f), p.cap_log2);
       } else {
 #pragma unroll
         for (int nt = 0; nt < WKEYS / 8; ++nt)
@@ -414,7 +436,7 @@ attention_mma_kernel(AttnParams p) {
         for (int j = 0; j < 4; ++j) {
           int h = j >> 1;
           int key = key0 + nt * 8 + 2 * c + (j & 1);
-          bool ok = key <= row_pos[h] && (p.window <= 0 || key > row_pos[h] - p.window);
+          bool ok = key <= row_pos[h] && (p.window <= 0 || key > row_pos[h] - p.window || (DIST && key < p.keep_first));
           if (!ok) s[nt][j] = -INFINITY;
         }
     }
@@ -463,6 +485,7 @@ attention_mma_kernel(AttnParams p) {
       a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
       for (int dp = 0; dp < HD / 16; ++dp) {
+        if (DIST && dp * 16 >= vdim) break;
         uint32_t vb[4];
         ldmatrix_x4_trans(vb, vt + (wkey + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + dp * 16 + (lane >> 4) * 8);
         mma_bf16(o_acc[2 * dp], a, vb[0], vb[1]);
@@ -658,6 +681,7 @@ struct RopeFusion {
 // A penalty on distance and sizes of their own for keys and values (head_dim of the call is then the tile size)
 struct DistanceOption {
   int key_dim, value_dim; const float* r1; const float* r2; float out_scale; const float* sink;
+  int keep_first; float softcap;
 };
 
 int attention_mma_impl(const void* q, int ld_q, const void* k_pool, const void* v_pool,
@@ -695,6 +719,9 @@ int attention_mma_impl(const void* q, int ld_q, const void* k_pool, const void* 
   make_paged_cache(&p.vcache, block_table, max_pages, page_size, kv_heads, dist ? dist->value_dim : head_dim);
   p.dist_r1 = dist ? dist->r1 : nullptr; p.dist_r2 = dist ? dist->r2 : nullptr; p.out_scale = dist ? dist->out_scale : 1.f;
   p.sink = dist ? dist->sink : nullptr;
+  p.keep_first = dist ? dist->keep_first : 0;
+  p.cap_log2 = dist && dist->softcap > 0.f ? dist->softcap * 1.4426950408889634f : 0.f;
+  p.cap_in = p.cap_log2 > 0.f ? 2.f * 1.4426950408889634f * scale / dist->softcap : 0.f;
   p.cu_tokens = cu_tokens; p.slots = slots; p.context_before = context_before;
   p.heads = heads; p.group = group;
   p.scale_log2 = scale * 1.4426950408889634f;
@@ -778,7 +805,7 @@ HFEE_API int hfee_attention_mma_distance(const void* q, int ld_q, const void* k_
   const int tile = hfee_attention_mma_distance_tile(key_dim, value_dim);
   HFEE_REQUIRE(tile > 0, "attention_mma_distance: key size %d and value size %d must be multiples of 8 up to 256", key_dim, value_dim);
   HFEE_REQUIRE(r1 != nullptr && r2 != nullptr, "attention_mma_distance: the penalty needs both of its arrays");
-  DistanceOption dist{key_dim, value_dim, r1, r2, out_scale, nullptr};
+  DistanceOption dist{key_dim, value_dim, r1, r2, out_scale, nullptr, 0, 0.f};
   return attention_mma_impl(q, ld_q, k_pool, v_pool, block_table, max_pages, page_size, cu_tokens, slots, context_before,
                             out, ld_o, n_tokens, requests, max_new, heads, kv_heads, tile, scale, window, num_splits,
                             scratch, nullptr, stream, &dist);
@@ -786,16 +813,20 @@ HFEE_API int hfee_attention_mma_distance(const void* q, int ld_q, const void* k_
 
 // hfee_attention_mma_distance with the penalty optional (r1 and r2 both null: none) and an optional sink: with
 // `sink` (float32 per query head) the softmax's denominator also holds exp(sink[h]), a term without key or value.
+// keep_first: that many positions from the start stay visible behind the window.  softcap > 0 (not with the penalty): the
+// scaled score becomes softcap * tanh(score / softcap).
 HFEE_API int hfee_attention_mma_general(const void* q, int ld_q, const void* k_pool, const void* v_pool,
                                         const int* block_table, int max_pages, int page_size, const int* cu_tokens,
                                         const int* slots, const int* context_before, void* out, int ld_o, int n_tokens,
                                         int requests, int max_new, int heads, int kv_heads, int key_dim, int value_dim,
                                         float scale, const float* r1, const float* r2, const float* sink, float out_scale,
-                                        int window, int num_splits, float* scratch, cudaStream_t stream) {
+                                        int window, int keep_first, float softcap, int num_splits, float* scratch,
+                                        cudaStream_t stream) {
   const int tile = hfee_attention_mma_distance_tile(key_dim, value_dim);
   HFEE_REQUIRE(tile > 0, "attention_mma_general: key size %d and value size %d must be multiples of 8 up to 256", key_dim, value_dim);
   HFEE_REQUIRE((r1 == nullptr) == (r2 == nullptr), "attention_mma_general: the penalty needs both of its arrays");
-  DistanceOption dist{key_dim, value_dim, r1, r2, out_scale, sink};
+  HFEE_REQUIRE(keep_first >= 0 && (softcap <= 0.f || r1 == nullptr), "attention_mma_general: bad mask, or a cap beside a penalty");
+  DistanceOption dist{key_dim, value_dim, r1, r2, out_scale, sink, keep_first, softcap};
   return attention_mma_impl(q, ld_q, k_pool, v_pool, block_table, max_pages, page_size, cu_tokens, slots, context_before,
                             out, ld_o, n_tokens, requests, max_new, heads, kv_heads, tile, scale, window, num_splits,
                             scratch, nullptr, stream, &dist);

@@ -35,7 +35,7 @@ attention_simt_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k
                       float scale, int window, int chunk, const float* __restrict__ head_scale,
                       const float* __restrict__ head_bias, const T* __restrict__ gate, long long ld_gate,
                       int gate_mode, const float* __restrict__ dist_r1, const float* __restrict__ dist_r2, float out_scale,
-                      const float* __restrict__ sink) {
+                      const float* __restrict__ sink, int keep_first, float softcap) {
   pdl_wait();
   pdl_launch_dependents();
   __shared__ float q_s[WARPS][MAX_HD];
@@ -63,29 +63,33 @@ attention_simt_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k
   // a sink is one more term exp(sink[h]) of the denominator that has no key and no value
   float m = (!SIGMOID && sink != nullptr) ? sink[h] : -INFINITY, l = (!SIGMOID && sink != nullptr) ? 1.f : 0.f;
 
-  for (int base = lo; base <= pos; base += 32) {
+  // the first keep_first positions stay visible behind the window: they are visited first, [0, kept), then [lo, pos]
+  const int kept = min(keep_first, lo);
+  for (int base = kept > 0 ? 0 : lo; base <= pos;) {
+    const int end = base < kept ? kept - 1 : pos;            // last key of the range this block of 32 lies in
     int key = base + lane;
     float s = -INFINITY;
-    if (key <= pos) {
+    if (key <= end) {
       const T* kr = k_pool + paged_offset(cache, slot, key, kvh);
       float acc = 0.f;
       for (int d = 0; d < hd; ++d) acc = fmaf(q_s[warp][d], to_f32<T>(kr[d]), acc);
       s = acc * scale;
+      if (softcap > 0.f) s = softcap * tanhf(s / softcap);
       if (dist_r1 != nullptr) s -= r1 * log1pf(r2 * (float)(pos - key));
     }
     float p;
     if constexpr (SIGMOID) {
-      p = key <= pos ? 1.f / (1.f + expf(-(s * h_scale + h_bias))) : 0.f;
+      p = key <= end ? 1.f / (1.f + expf(-(s * h_scale + h_bias))) : 0.f;
     } else {
       float m_new = fmaxf(m, warp_max(s));
-      p = key <= pos ? expf(s - m_new) : 0.f;
+      p = key <= end ? expf(s - m_new) : 0.f;
       float alpha = expf(m - m_new);          // exp(-inf) = 0 on the first block
       l = l * alpha + warp_sum(p);
 #pragma unroll
       for (int j = 0; j < DPL; ++j) o[j] *= alpha;
       m = m_new;
     }
-    int count = min(32, pos + 1 - base);
+    int count = min(32, end + 1 - base);
     for (int t = 0; t < count; ++t) {
       float pt = __shfl_sync(0xffffffffu, p, t);
       const T* vr = v_pool + paged_offset(vcache, slot, base + t, kvh);
@@ -95,6 +99,8 @@ attention_simt_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k
         if (d < vd) o[j] = fmaf(pt, to_f32<T>(vr[d]), o[j]);
       }
     }
+    base += 32;
+    if (base >= kept && base < lo) base = lo;
   }
   T* orow = out + (long long)i * ld_o + (long long)h * vd;
   float inv = (SIGMOID ? 1.f : 1.f / l) * out_scale;
@@ -119,17 +125,18 @@ void launch_simt(const void* q, int ld_q, const void* k_pool, const void* v_pool
                  int vd, const int* positions,
                  const int* slot_of_token, void* out, int ld_o, int n, int heads, float scale, int window, int chunk,
                  int sigmoid, const float* head_scale, const float* head_bias, const void* gate, long long ld_gate,
-                 int gate_mode, const float* dist_r1, const float* dist_r2, float out_scale, const float* sink, cudaStream_t stream) {
+                 int gate_mode, const float* dist_r1, const float* dist_r2, float out_scale, const float* sink, int keep_first,
+                 float softcap, cudaStream_t stream) {
   long long tasks = (long long)n * heads;
   unsigned blocks = (unsigned)((tasks + WARPS - 1) / WARPS);
   if (sigmoid)
     hfee_launch(attention_simt_kernel<T, true>, dim3(blocks), dim3(WARPS * 32), 0, stream, (const T*)q, ld_q, (const T*)k_pool,
                 (const T*)v_pool, c, vc, vd, positions, slot_of_token, (T*)out, ld_o, n, heads, scale, window, chunk, head_scale,
-                head_bias, (const T*)gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink);
+                head_bias, (const T*)gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink, keep_first, softcap);
   else
     hfee_launch(attention_simt_kernel<T, false>, dim3(blocks), dim3(WARPS * 32), 0, stream, (const T*)q, ld_q, (const T*)k_pool,
                 (const T*)v_pool, c, vc, vd, positions, slot_of_token, (T*)out, ld_o, n, heads, scale, window, chunk, head_scale,
-                head_bias, (const T*)gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink);
+                head_bias, (const T*)gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink, keep_first, softcap);
 }
 }  // namespace
 
@@ -139,15 +146,17 @@ void launch_simt(const void* q, int ld_q, const void* k_pool, const void* v_pool
 // element ([n, heads * value_dim]), 2 one number per head ([n, heads]); the output is multiplied by its sigmoid.
 // dist_r1, dist_r2 (per head, or both null): r1[h] * ln(1 + r2[h] * (query position - key position)) is taken off the
 // score before the softmax.  out_scale multiplies the output.  sink (per head, or null): the softmax's denominator also
-// holds exp(sink[h]).
-HFEE_API int hfee_attention_simt_sink(const void* q, int ld_q, const void* k_pool, const void* v_pool,
+// holds exp(sink[h]).  keep_first: that many positions from the start stay visible behind a window.  softcap > 0: the scaled
+// score becomes softcap * tanh(score / softcap).
+HFEE_API int hfee_attention_simt_capped(const void* q, int ld_q, const void* k_pool, const void* v_pool,
                                           const int* block_table, int max_pages, int page_size, const int* positions,
                                           const int* slot_of_token, void* out, int ld_o, int n, int heads, int kv_heads,
                                           int head_dim, int value_dim, int values_in_keys, float scale, int window,
                                           int chunk, int weights, const float* head_scale, const float* head_bias,
                                           const void* gate, long long ld_gate, int gate_mode, const float* dist_r1,
-                                          const float* dist_r2, float out_scale, const float* sink, int dtype,
-                                          cudaStream_t stream) {
+                                          const float* dist_r2, float out_scale, const float* sink, int keep_first,
+                                          float softcap, int dtype, cudaStream_t stream) {
+  HFEE_REQUIRE(keep_first >= 0 && (keep_first == 0 || chunk == 0), "attention_simt: kept first positions go with a window");
   HFEE_REQUIRE(sink == nullptr || weights == 0, "attention_simt: a sink goes with the softmax");
   HFEE_REQUIRE((dist_r1 == nullptr) == (dist_r2 == nullptr), "attention_simt: the distance penalty needs both of its arrays");
   HFEE_REQUIRE(dist_r1 == nullptr || weights == 0, "attention_simt: the distance penalty goes with the softmax");
@@ -174,14 +183,29 @@ HFEE_API int hfee_attention_simt_sink(const void* q, int ld_q, const void* k_poo
   }
   if (dtype == HFEE_F32)
     launch_simt<float>(q, ld_q, k_pool, v_pool, c, vc, value_dim, positions, slot_of_token, out, ld_o, n, heads, scale,
-                       window, chunk, weights, head_scale, head_bias, gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink, stream);
+                       window, chunk, weights, head_scale, head_bias, gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink, keep_first,
+                       softcap, stream);
   else if (dtype == HFEE_BF16)
     launch_simt<__nv_bfloat16>(q, ld_q, k_pool, v_pool, c, vc, value_dim, positions, slot_of_token, out, ld_o, n, heads,
                                scale, window, chunk, weights, head_scale, head_bias, gate, ld_gate, gate_mode, dist_r1, dist_r2,
-                               out_scale, sink, stream);
+                               out_scale, sink, keep_first, softcap, stream);
   else
     return hfee_fail(HFEE_ERR_ARG, "attention_simt: unknown dtype %d", dtype);
   return hfee_check_launch("attention_simt");
+}
+
+HFEE_API int hfee_attention_simt_sink(const void* q, int ld_q, const void* k_pool, const void* v_pool,
+                                      const int* block_table, int max_pages, int page_size, const int* positions,
+                                      const int* slot_of_token, void* out, int ld_o, int n, int heads, int kv_heads,
+                                      int head_dim, int value_dim, int values_in_keys, float scale, int window,
+                                      int chunk, int weights, const float* head_scale, const float* head_bias,
+                                      const void* gate, long long ld_gate, int gate_mode, const float* dist_r1,
+                                      const float* dist_r2, float out_scale, const float* sink, int dtype,
+                                      cudaStream_t stream) {
+  return hfee_attention_simt_capped(q, ld_q, k_pool, v_pool, block_table, max_pages, page_size, positions, slot_of_token, out,
+                                    ld_o, n, heads, kv_heads, head_dim, value_dim, values_in_keys, scale, window, chunk,
+                                    weights, head_scale, head_bias, gate, ld_gate, gate_mode, dist_r1, dist_r2, out_scale, sink,
+                                    0, 0.f, dtype, stream);
 }
 
 HFEE_API int hfee_attention_simt_distance(const void* q, int ld_q, const void* k_pool, const void* v_pool,

@@ -115,6 +115,20 @@ __device__ __forceinline__ float gelu_tanh_gate_fast(float z) {
   return __fdividef(z, 1.f + __expf(-2.f * u));
 }
 
+// The gate of a gated product: act(z) for the epilogue ids that every product shares (2: SiLU, 4: tanh-GELU, 7: relu).
+constexpr int GATE_SILU = 2, GATE_GELU_TANH = 4, GATE_RELU = 7;
+template <int EPI> __device__ __forceinline__ float gate_value(float z) {
+  if constexpr (EPI == GATE_GELU_TANH) return gelu_tanh_gate(z);
+  if constexpr (EPI == GATE_RELU) return fmaxf(z, 0.f);
+  return z / (1.f + expf(-z));
+}
+// for results that are rounded to bfloat16 right away
+template <int EPI> __device__ __forceinline__ float gate_value_fast(float z) {
+  if constexpr (EPI == GATE_GELU_TANH) return gelu_tanh_gate_fast(z);
+  if constexpr (EPI == GATE_RELU) return fmaxf(z, 0.f);
+  return __fdividef(z, 1.f + __expf(-z));
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

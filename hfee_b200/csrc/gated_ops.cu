@@ -2,7 +2,7 @@
 //
 //   hfee_rmsnorm_add      residual += y / sqrt(mean(y^2) + eps) * w          (a norm on a sublayer's output)
 //   hfee_norm_gate        out = [x / sqrt(mean(x^2) + eps) * w] * sigmoid(g)  (the norm is optional)
-//   hfee_gated_act        out = act(gate) * up, act = SiLU or tanh-GELU
+//   hfee_gated_act        out = act(gate) * up, act = SiLU, tanh-GELU or relu
 //   hfee_scale_f32        x *= alpha
 //   hfee_cast_rows        out = x rounded to the activations' type (what a matrix product reads of the residual stream)
 //   hfee_qk_norm_rope_cache   RMS norm over a token's whole query (and key) projection, rotary on the
@@ -177,9 +177,10 @@ norm_gate_vec_kernel(const float* __restrict__ x, long long ld_x, const float* _
   }
 }
 
-enum GateActivation { GA_SILU = 0, GA_GELU_TANH = 1 };
+enum GateActivation { GA_SILU = 0, GA_GELU_TANH = 1, GA_RELU = 2 };
 
 __device__ __forceinline__ float gate_activation(float z, int act) {
+  if (act == GA_RELU) return fmaxf(z, 0.f);
   if (act == GA_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
   return z / (1.f + expf(-z));
 }
@@ -392,7 +393,7 @@ HFEE_API int hfee_gated_act(const void* gu, long long ld_gu, void* h, long long 
   if (n == 0) return HFEE_OK;
   HFEE_REQUIRE(n > 0 && inter > 0 && ld_gu >= 2 * inter && ld_h >= inter, "gated_act: bad sizes");
   HFEE_REQUIRE(granule > 0 && inter % granule == 0, "gated_act: granule %d does not divide %d", granule, inter);
-  HFEE_REQUIRE(act == GA_SILU || act == GA_GELU_TANH, "gated_act: unknown activation %d", act);
+  HFEE_REQUIRE(act == GA_SILU || act == GA_GELU_TANH || act == GA_RELU, "gated_act: unknown activation %d", act);
   long long total = (long long)n * inter;
   unsigned blocks = (unsigned)((total + 255) / 256);
   if (dtype == HFEE_F32)
@@ -456,6 +457,8 @@ HFEE_API int hfee_qk_norm_rope_cache(const void* qk, long long ld_qk, const floa
 // ---------------------------------------------------------------------------------------------------------------
 //   hfee_head_norm_gate   per (token, head): out = x / sqrt(mean_head(x^2) + eps) * w[d] * act(gate) * out_scale, the weight
 //                         [head_dim] shared by the heads, or [heads * head_dim] (w_head_stride = head_dim); act = sigmoid or SiLU
+//   hfee_gate_parts_norm  g = x * silu(z), then every one of `parts` equal parts of the row divided by its own root mean
+//                         square, times w per column, times out_scale: the gate in front of the norm
 //   hfee_unary_act        out = act(x) element by element; act = relu(x)^2
 //   hfee_head_gate        x[i, h, :] *= sigmoid(gate[i, h]): one gate number per head
 namespace {
@@ -488,6 +491,86 @@ head_norm_gate_kernel(const float* __restrict__ x, long long ld_x, const float* 
   }
 }
 
+template <typename T> __device__ __forceinline__ float silu_gate(float z);
+template <> __device__ __forceinline__ float silu_gate<float>(float z) { return z / (1.f + expf(-z)); }
+template <> __device__ __forceinline__ float silu_gate<__nv_bfloat16>(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+
+// A block per (row, part).  VEC: columns per access (4: rows that 16- and 8-byte accesses can read); NCH accesses per thread
+// stay in registers between the passes (longer parts are computed twice).
+template <typename T, int VEC, int NCH>
+__global__ void __launch_bounds__(ROW_THREADS)
+gate_parts_norm_kernel(const float* __restrict__ x, long long ld_x, const T* __restrict__ z, long long ld_z,
+                       const float* __restrict__ w, float eps, T* __restrict__ out, long long ld_o, int part, float out_scale) {
+  __shared__ float partial[ROW_THREADS / 32];
+  const long long c0 = (long long)blockIdx.y * part;
+  const float* wr = w + c0;
+  pdl_wait();
+  pdl_launch_dependents();
+  const float* xr = x + (long long)blockIdx.x * ld_x + c0;
+  const T* zr = z + (long long)blockIdx.x * ld_z + c0;
+  T* orow = out + (long long)blockIdx.x * ld_o + c0;
+  auto gated = [&](int c, float (&g)[VEC]) {
+    if constexpr (VEC == 4) {
+      const float4 xv = load4(xr + c), zv = load4(zr + c);
+      g[0] = xv.x * silu_gate<T>(zv.x); g[1] = xv.y * silu_gate<T>(zv.y);
+      g[2] = xv.z * silu_gate<T>(zv.z); g[3] = xv.w * silu_gate<T>(zv.w);
+    } else {
+      g[0] = xr[c] * silu_gate<T>(to_f32<T>(zr[c]));
+    }
+  };
+  auto put = [&](int c, const float (&g)[VEC], float scale) {
+    if constexpr (VEC == 4) {
+      const float4 wv = load4(wr + c);
+      store4(orow + c, make_float4(g[0] * scale * wv.x, g[1] * scale * wv.y, g[2] * scale * wv.z, g[3] * scale * wv.w));
+    } else {
+      orow[c] = from_f32<T>(g[0] * scale * wr[c]);
+    }
+  };
+  constexpr int STRIDE = ROW_THREADS * VEC;
+  float kept[NCH][VEC];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NCH; ++j) {
+    const int c = threadIdx.x * VEC + j * STRIDE;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) kept[j][e] = 0.f;
+    if (c < part) gated(c, kept[j]);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(kept[j][e], kept[j][e], ss);
+  }
+  for (int c = threadIdx.x * VEC + NCH * STRIDE; c < part; c += STRIDE) {
+    float g[VEC];
+    gated(c, g);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(g[e], g[e], ss);
+  }
+  const float scale = out_scale / sqrtf(block_sum(ss, partial) / (float)part + eps);
+#pragma unroll
+  for (int j = 0; j < NCH; ++j) {
+    const int c = threadIdx.x * VEC + j * STRIDE;
+    if (c < part) put(c, kept[j], scale);
+  }
+  for (int c = threadIdx.x * VEC + NCH * STRIDE; c < part; c += STRIDE) {
+    float g[VEC];
+    gated(c, g);
+    put(c, g, scale);
+  }
+}
+
+template <typename T>
+void launch_gate_parts_norm(const float* x, long long ld_x, const void* z, long long ld_z, const float* w, float eps, void* out,
+                            long long ld_o, int n, int parts, int part, float out_scale, cudaStream_t stream) {
+  const bool vec = part % 4 == 0 && ld_x % 4 == 0 && ld_z % 4 == 0 && ld_o % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
+                   (uintptr_t)z % (4 * sizeof(T)) == 0 && (uintptr_t)out % (4 * sizeof(T)) == 0;
+  const dim3 grid((unsigned)n, (unsigned)parts), block(ROW_THREADS);
+  if (vec && part <= ROW_THREADS * 4)
+    hfee_launch(gate_parts_norm_kernel<T, 4, 1>, grid, block, 0, stream, x, ld_x, (const T*)z, ld_z, w, eps, (T*)out, ld_o, part, out_scale);
+  else if (vec)
+    hfee_launch(gate_parts_norm_kernel<T, 4, 4>, grid, block, 0, stream, x, ld_x, (const T*)z, ld_z, w, eps, (T*)out, ld_o, part, out_scale);
+  else
+    hfee_launch(gate_parts_norm_kernel<T, 1, 8>, grid, block, 0, stream, x, ld_x, (const T*)z, ld_z, w, eps, (T*)out, ld_o, part, out_scale);
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256)
 unary_act_kernel(const T* __restrict__ x, long long ld_x, T* __restrict__ out, long long ld_o, int cols, long long total, int act) {
@@ -517,6 +600,20 @@ head_gate_kernel(T* __restrict__ x, long long ld_x, const T* __restrict__ gate, 
 }
 
 }  // namespace
+
+HFEE_API int hfee_gate_parts_norm(const float* x, long long ld_x, const void* z, long long ld_z, const float* w, float eps, void* out,
+                                  long long ld_o, int n, int width, int parts, float out_scale, int dtype, cudaStream_t stream) {
+  if (n == 0) return HFEE_OK;
+  HFEE_REQUIRE(n > 0 && width > 0 && parts > 0 && width % parts == 0 && parts <= 65535, "gate_parts_norm: %d parts do not divide %d columns", parts, width);
+  HFEE_REQUIRE(ld_x >= width && ld_z >= width && ld_o >= width, "gate_parts_norm: a row stride is too small");
+  if (dtype == HFEE_F32)
+    launch_gate_parts_norm<float>(x, ld_x, z, ld_z, w, eps, out, ld_o, n, parts, width / parts, out_scale, stream);
+  else if (dtype == HFEE_BF16)
+    launch_gate_parts_norm<__nv_bfloat16>(x, ld_x, z, ld_z, w, eps, out, ld_o, n, parts, width / parts, out_scale, stream);
+  else
+    return hfee_fail(HFEE_ERR_ARG, "gate_parts_norm: unknown dtype %d", dtype);
+  return hfee_check_launch("gate_parts_norm");
+}
 
 HFEE_API int hfee_head_norm_gate_scaled(const float* x, long long ld_x, const float* w, int w_per_head, float eps, const void* gate,
                                         long long ld_g, void* out, long long ld_o, int n, int heads, int head_dim, int act,

@@ -7,6 +7,10 @@
 //                      S_t = e^(f_t + m_(t-1) - m_t) S_(t-1) + e^(i_t - m_t) k_t v_t^T          (n_t the same with k_t alone)
 //                      o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + 1e-6)
 //
+//   step sizes         S_t = exp(-exp(A_log_h) dt_t) S_(t-1) + dt_t k_t v_t^T           dt_t = softplus(x_dt + bias) per head
+//                      o_t = S_t^T q_t + D_h v_t                             (a state-space scan with one decay per head and
+//                      token; neighbouring heads may share one q and k)
+//
 // S: [dim][vdim], n: [dim], m: one number; all zero for a fresh request.  q (times q_scale), k and v are slices of one
 // projection buffer (type T); the gates' pre-activations z, x_i, x_f are float32, and so are the decays, their
 // logarithms and exponentials, the states, every product and o.
@@ -38,7 +42,7 @@ constexpr int GR_MAX_DIM = 256;
 constexpr int GC_T = 64;             // tokens of a run of the chunked path
 enum Pass { PASS_WHOLE = 0, PASS_LOCAL = 1, PASS_OUT = 2 };
 
-enum Mode { MODE_CHANNEL_DECAY = 0, MODE_EXP_GATES = 1 };
+enum Mode { MODE_CHANNEL_DECAY = 0, MODE_EXP_GATES = 1, MODE_STEP = 2 };
 
 __device__ __forceinline__ float log_sigmoid_f32(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
@@ -65,7 +69,15 @@ struct RecurrenceArgs {
   const float* gates;           // [3][n_tokens, heads]: a_t, b_t, e^(-m_t) (exponential gates)
   long long gate_stride;        // n_tokens * heads
   int decays_given;             // channel decay: `pre` holds the decays themselves (the chunked path computes them once)
+  // step sizes: x_dt [n, heads] in the activations' type, a decay rate and a skip weight per head, heads per q/k head
+  const void* step;
+  long long ld_step;
+  const float* a_log;
+  const float* d_skip;
+  int qk_share;
 };
+
+__device__ __forceinline__ float softplus_f32(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 __device__ __forceinline__ int runs_of(int count) { return (count + GC_T - 1) / GC_T; }
 
@@ -134,7 +146,7 @@ gated_recurrence_kernel(const T* __restrict__ q, const T* __restrict__ k, const 
   // A block has as many threads as a staged token has (padded) key channels: thread `tid` brings channel `tid` of every
   // token of a stage, and its share of the stage's values.
   const bool live_d = tid < dim;
-  const int chan = head * dim + tid;
+  const int chan = (MODE == MODE_STEP ? head / p.qk_share : head) * dim + tid;
   const float z_bias = (MODE == MODE_CHANNEL_DECAY && live_d && !p.decays_given && p.bias != nullptr) ? p.bias[chan] : 0.f;
   for (int t0 = 0; t0 < count; t0 += GR_STAGE) {
     const int nt = min(GR_STAGE, count - t0);
@@ -159,6 +171,21 @@ gated_recurrence_kernel(const T* __restrict__ q, const T* __restrict__ k, const 
     for (int e = tid; e < nt * GR_COLS; e += threads) {
       const int t = e / GR_COLS, c = blockIdx.z * GR_COLS + e % GR_COLS;
       vs[e] = c < vdim ? to_f32<T>(v[(long long)(begin + t0 + t) * p.ld + (long long)head * vdim + c]) : 0.f;
+    }
+    if constexpr (MODE == MODE_STEP && PASS == PASS_WHOLE) {
+      if (tid < nt) {
+        const float dt = softplus_f32(to_f32<T>(reinterpret_cast<const T*>(p.step)[(long long)(begin + t0 + tid) * p.ld_step + head]) +
+                                      p.bias[head]);
+        a_s[tid] = expf(-expf(p.a_log[head]) * dt);
+        b_s[tid] = dt;
+      }
+    }
+    if constexpr (MODE == MODE_STEP && PASS != PASS_WHOLE) {
+      if (tid < nt) {
+        const long long at = (long long)(begin + t0 + tid) * heads + head;
+        a_s[tid] = p.gates[at];
+        b_s[tid] = p.gates[p.gate_stride + at];
+      }
     }
     if constexpr (MODE == MODE_EXP_GATES && PASS != PASS_WHOLE) {
       if (tid < nt) {                                 // the gates were computed for every token beforehand
@@ -222,9 +249,9 @@ gated_recurrence_kernel(const T* __restrict__ q, const T* __restrict__ k, const 
           S[1][4 * i + 2] = fmaf(a, S[1][4 * i + 2], kk.z * bw);  acd = fmaf(S[1][4 * i + 2], qq.z, acd);
           S[1][4 * i + 3] = fmaf(a, S[1][4 * i + 3], kk.w * bw);  acd = fmaf(S[1][4 * i + 3], qq.w, acd);
         }
-        n_own = fmaf(a, n_own, b_s[t] * ks[t * dim_pad + own_row]);
+        if constexpr (MODE == MODE_EXP_GATES) n_own = fmaf(a, n_own, b_s[t] * ks[t * dim_pad + own_row]);
         if constexpr (PASS == PASS_LOCAL) decay_own *= a;
-        if constexpr (PASS != PASS_LOCAL) {
+        if constexpr (MODE == MODE_EXP_GATES && PASS != PASS_LOCAL) {
           const float nq = warp_sum(n_own * qs[t * dim_pad + own_row]);
           if (j == 0) part_n[t * groups + g] = nq;
         }
@@ -245,6 +272,7 @@ gated_recurrence_kernel(const T* __restrict__ q, const T* __restrict__ k, const 
         for (int gg = 0; gg < groups; ++gg) nq += part_n[t * groups + gg];
         sum /= fmaxf(fabsf(nq), em_s[t]) + 1e-6f;
       }
+      if constexpr (MODE == MODE_STEP) sum = fmaf(p.d_skip[head], vs[t * GR_COLS + jj], sum);
       if (c < vdim) p.out[(long long)(begin + t0 + t) * p.ld_o + (long long)head * vdim + c] = sum;
     }
   }
@@ -280,6 +308,22 @@ channel_decays_kernel(float* __restrict__ pre, long long ld_pre, const float* __
   const int c = (int)(e - r * cols);
   float* at = pre + r * ld_pre + c;
   *at = expf(log_sigmoid_f32(*at + (bias != nullptr ? bias[c] : 0.f)) * p0);
+}
+
+// Every token's decay and step size (step sizes): gates[t, h] = exp(-exp(A_log_h) dt), gates[stride + (t, h)] = dt.
+template <typename T>
+__global__ void __launch_bounds__(256)
+step_gates_kernel(const T* __restrict__ step, long long ld_step, const float* __restrict__ bias, const float* __restrict__ a_log,
+                  int heads, float* __restrict__ gates, long long total) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const long long e = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (e >= total) return;
+  const long long t = e / heads;
+  const int h = (int)(e - t * heads);
+  const float dt = softplus_f32(to_f32<T>(step[t * ld_step + h]) + bias[h]);
+  gates[e] = expf(-expf(a_log[h]) * dt);
+  gates[total + e] = dt;
 }
 
 // Every token's gates of the exponential recurrence, one warp per (request, head).  The running maximum is the map
@@ -404,6 +448,8 @@ int launch_recurrence(int mode, const void* q, const void* k, const void* v, con
   const size_t smem = floats * sizeof(float);
   if (mode == MODE_CHANNEL_DECAY)
     hfee_launch(gated_recurrence_kernel<T, MODE_CHANNEL_DECAY, PASS>, grid, block, smem, stream, (const T*)q, (const T*)k, (const T*)v, p);
+  else if (mode == MODE_STEP)
+    hfee_launch(gated_recurrence_kernel<T, MODE_STEP, PASS>, grid, block, smem, stream, (const T*)q, (const T*)k, (const T*)v, p);
   else
     hfee_launch(gated_recurrence_kernel<T, MODE_EXP_GATES, PASS>, grid, block, smem, stream, (const T*)q, (const T*)k, (const T*)v, p);
   return hfee_check_launch("gated_recurrence");
@@ -419,6 +465,12 @@ int launch_chunked(int mode, const void* q, const void* k, const void* v, Recurr
     int rc = hfee_check_launch("channel_decays");
     if (rc != HFEE_OK) return rc;
     p.decays_given = 1;
+  }
+  if (mode == MODE_STEP) {
+    hfee_launch(step_gates_kernel<T>, dim3((unsigned)((p.gate_stride + 255) / 256)), dim3(256), 0, stream, (const T*)p.step, p.ld_step, bias,
+                p.a_log, p.heads, (float*)p.gates, p.gate_stride);
+    int rc = hfee_check_launch("step_gates");
+    if (rc != HFEE_OK) return rc;
   }
   if (mode == MODE_EXP_GATES) {
     hfee_launch(memory_gates_kernel, dim3((p.requests * p.heads + 3) / 4), dim3(128), 0, stream, pre, ld_pre, bias, cap, p.max_state,
@@ -498,4 +550,38 @@ HFEE_API int hfee_gated_recurrence_chunked(int mode, const void* q, const void* 
   if (dtype == HFEE_F32) return launch_chunked<float>(mode, q, k, v, p, pre, ld_pre, bias, p0, n_tokens, (int)max_runs, stream);
   if (dtype == HFEE_BF16) return launch_chunked<__nv_bfloat16>(mode, q, k, v, p, pre, ld_pre, bias, p0, n_tokens, (int)max_runs, stream);
   return hfee_fail(HFEE_ERR_ARG, "gated_recurrence: unknown dtype %d", dtype);
+}
+
+// The scan with step sizes: x [n, heads * vdim] (the values), bmat and cmat: `groups` vectors of `state_dim` entries a token (head h
+// uses group h / (heads / groups)), all of rows with the stride ld; step: [n, heads] (stride ld_step, the same type), in front of
+// its bias and softplus; state [slots, heads, state_dim, vdim] float32, read and renewed; out [n, heads * vdim] float32.
+// With a workspace (hfee_gated_recurrence_workspace floats) runs of 64 tokens are walked side by side.
+HFEE_API int hfee_head_scan(const void* x, const void* bmat, const void* cmat, long long ld, const void* step, long long ld_step,
+                            int dtype, const float* dt_bias, const float* a_log, const float* d_skip, float* state,
+                            const int* cu_tokens, const int* slots, float* out, long long ld_o, int requests, int n_tokens,
+                            int heads, int groups, int state_dim, int vdim, int write_state, float* workspace,
+                            long long workspace_floats, cudaStream_t stream) {
+  if (requests == 0 || n_tokens == 0) return HFEE_OK;
+  HFEE_REQUIRE(heads > 0 && groups > 0 && heads % groups == 0 && vdim > 0, "head_scan: heads %d must be a multiple of groups %d", heads, groups);
+  HFEE_REQUIRE(state_dim > 0 && state_dim <= GR_MAX_DIM, "head_scan: state size %d is outside 1..%d", state_dim, GR_MAX_DIM);
+  HFEE_REQUIRE(requests <= 65535 && (vdim + GR_COLS - 1) / GR_COLS <= 65535, "head_scan: too many requests or columns for one grid");
+  HFEE_REQUIRE(ld_o >= (long long)heads * vdim && ld_step >= heads, "head_scan: a row stride is too small");
+  RecurrenceArgs p{ld, nullptr, 0, dt_bias, 1.f, 1.f, state, nullptr, nullptr, cu_tokens, slots, out, ld_o, heads, state_dim, vdim, write_state,
+                   requests, nullptr, nullptr, nullptr, nullptr, 0, 0, step, ld_step, a_log, d_skip, heads / groups};
+  if (workspace == nullptr) {
+    if (dtype == HFEE_F32) return launch_recurrence<float, PASS_WHOLE>(MODE_STEP, cmat, bmat, x, p, requests, stream);
+    if (dtype == HFEE_BF16) return launch_recurrence<__nv_bfloat16, PASS_WHOLE>(MODE_STEP, cmat, bmat, x, p, requests, stream);
+    return hfee_fail(HFEE_ERR_ARG, "head_scan: unknown dtype %d", dtype);
+  }
+  const long long max_runs = n_tokens / GC_T + requests;
+  HFEE_REQUIRE(max_runs <= 65535, "head_scan: too many runs for one grid");
+  HFEE_REQUIRE(workspace_floats >= hfee_gated_recurrence_workspace(requests, n_tokens, heads, state_dim, vdim), "head_scan: the workspace is too small");
+  p.run_state = workspace;
+  p.run_norm = p.run_state + max_runs * heads * state_dim * vdim;
+  p.run_decay = p.run_norm + max_runs * heads * state_dim;
+  p.gates = p.run_decay + max_runs * heads * state_dim;
+  p.gate_stride = (long long)n_tokens * heads;
+  if (dtype == HFEE_F32) return launch_chunked<float>(MODE_STEP, cmat, bmat, x, p, nullptr, 0, dt_bias, 1.f, n_tokens, (int)max_runs, stream);
+  if (dtype == HFEE_BF16) return launch_chunked<__nv_bfloat16>(MODE_STEP, cmat, bmat, x, p, nullptr, 0, dt_bias, 1.f, n_tokens, (int)max_runs, stream);
+  return hfee_fail(HFEE_ERR_ARG, "head_scan: unknown dtype %d", dtype);
 }

@@ -3,6 +3,7 @@
 //
 //   hfee_moe_route     scores = softmax(logits) over all experts (float32); the `top` largest per token (ties: the lower
 //                      expert), their weights = score * scale (not renormalised).
+//   hfee_moe_route_chosen  the same with weights that are a softmax over the chosen logits (plus a bias per expert).
 //   hfee_moe_plan      orders the (token, choice) pairs by expert: offsets[e] .. offsets[e + 1] are the places of expert
 //                      e's pairs, sorted[place] = token * top + choice; the places are cut into tiles of MOE_TILE rows
 //                      that never span two experts (tile_expert, tile_row; unused tiles carry expert -1).
@@ -131,6 +132,48 @@ __global__ void moe_route_grouped_kernel(const float* __restrict__ logits, int l
   }
   if (lane < top) weight[(long long)t * top + lane] = weight[(long long)t * top + lane] / (sum + 1e-20f) * scale;
   for (int k = 32 + lane; k < top; k += 32) weight[(long long)t * top + k] = weight[(long long)t * top + k] / (sum + 1e-20f) * scale;
+}
+
+// Router whose weights are a softmax over the chosen logits alone: z = logits + bias (bias may be null), the `top` largest z
+// (ties: the lower expert), weight_k = scale * exp(z_k) / sum over the chosen of exp(z).  One warp per token; rows have the
+// stride ld (columns behind `experts` are not the router's).
+__global__ void moe_route_chosen_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int experts, int top,
+                                        float scale, int* __restrict__ choice, float* __restrict__ weight, int n) {
+  extern __shared__ float score_s[];       // [warps][experts]
+  pdl_wait();
+  pdl_launch_dependents();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+  if (t >= n) return;
+  float* s = score_s + (long long)warp * experts;
+  const float* z = logits + (long long)t * ld;
+  for (int e = lane; e < experts; e += 32) s[e] = z[e] + (bias != nullptr ? bias[e] : 0.f);
+  __syncwarp();
+  float top_z = 0.f, sum = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float best = -INFINITY;
+    int at = experts;
+    for (int e = lane; e < experts; e += 32)
+      if (s[e] > best) { best = s[e]; at = e; }            // ascending e: the lowest index wins a tie within the lane
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+      if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+    }
+    if (at >= experts) at = 0;               // no finite logit is left: still an expert that exists, with no weight
+    if (k == 0) top_z = best;
+    const float e = best == -INFINITY ? 0.f : expf(best - top_z);
+    sum += e;
+    if (lane == 0) {
+      choice[(long long)t * top + k] = at;
+      weight[(long long)t * top + k] = e;
+      s[at] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  const float norm = sum > 0.f ? scale / sum : 0.f;
+  for (int k = lane; k < top; k += 32) weight[(long long)t * top + k] *= norm;
 }
 
 __global__ void __launch_bounds__(PLAN_THREADS)
@@ -347,6 +390,18 @@ HFEE_API int hfee_moe_route(const float* logits, int n, int experts, int top, fl
   hfee_launch(moe_route_kernel, dim3((n + warps - 1) / warps), dim3(32 * warps), (size_t)warps * experts * sizeof(float), stream,
               logits, experts, top, scale, choice, weight, n);
   return hfee_check_launch("moe_route");
+}
+
+// logits: [n, ld] float32 of which the first `experts` columns are the router's; bias: [experts] or null.
+HFEE_API int hfee_moe_route_chosen(const float* logits, long long ld, const float* bias, int n, int experts, int top, float scale,
+                                   int* choice, float* weight, cudaStream_t stream) {
+  if (n == 0) return HFEE_OK;
+  HFEE_REQUIRE(n > 0 && experts >= 1 && experts <= MAX_EXPERTS, "moe_route_chosen: %d experts are outside 1..%d", experts, MAX_EXPERTS);
+  HFEE_REQUIRE(top >= 1 && top <= experts && ld >= experts, "moe_route_chosen: top %d is outside 1..%d, or ld is too small", top, experts);
+  const int warps = 4;
+  hfee_launch(moe_route_chosen_kernel, dim3((n + warps - 1) / warps), dim3(32 * warps), (size_t)warps * experts * sizeof(float), stream,
+              logits, (int)ld, bias, experts, top, scale, choice, weight, n);
+  return hfee_check_launch("moe_route_chosen");
 }
 
 // offsets: [experts + 1]; sorted: [pairs]; tile_expert, tile_row: [max_tiles], max_tiles >= pairs / MOE_TILE + experts.

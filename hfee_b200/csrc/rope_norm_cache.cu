@@ -187,6 +187,7 @@ latent_attend_prepare_kernel(const T* __restrict__ proj, long long ld, int kv_of
 }
 
 constexpr int AP_THREADS = 128;
+constexpr int MIX_NONE = 0, MIX_STORE = 1, MIX_MIX = 2;
 
 __device__ __forceinline__ float block_sum_ap(float v, float* partial) {
   v = warp_sum(v);
@@ -221,7 +222,8 @@ attention_prepare_kernel(const T* __restrict__ src, long long ld_src, int q_off,
                          const float* __restrict__ cs, int rope_dim, int interleaved,
                          const int* __restrict__ positions, const int* __restrict__ slot_of_token,
                          T* __restrict__ q_out, long long ld_q, T* __restrict__ k_pool, PagedCache kc,
-                         T* __restrict__ v_pool, PagedCache vc, int heads, int key_dim) {
+                         T* __restrict__ v_pool, PagedCache vc, int heads, int key_dim, T* __restrict__ first_values,
+                         long long ld_first, int mix_mode, float share) {
   extern __shared__ float row_s[];            // [q_cols | k_cols | v_cols]
   __shared__ float partial[AP_THREADS / 32];
   const int i = blockIdx.x;
@@ -269,7 +271,11 @@ attention_prepare_kernel(const T* __restrict__ src, long long ld_src, int q_off,
   const int vd = vc.head_dim;
   for (int c = threadIdx.x; c < v_cols; c += AP_THREADS) {
     const int g = c / vd, d = c - g * vd;
-    v_pool[paged_offset(vc, slot, pos, g) + d] = from_f32<T>(vs[c]);
+    float v = vs[c];
+    if (mix_mode == MIX_MIX) v = fmaf(share, to_f32<T>(first_values[(long long)i * ld_first + c]), (1.f - share) * v);
+    const T vt = from_f32<T>(v);
+    if (mix_mode == MIX_STORE) first_values[(long long)i * ld_first + c] = vt;
+    v_pool[paged_offset(vc, slot, pos, g) + d] = vt;
   }
 }
 
@@ -341,15 +347,20 @@ HFEE_API int hfee_rope_norm_cache(const void* src, long long ld_src, int dtype, 
 // key_dim) and the value projection at v_off (kv_heads * value_dim).  bq, bk, bv: a bias per column (float32, each may
 // be null); wq, wk: weights of an RMS norm over the whole query / key projection (null: no norm); cs: [n, rope_dim/2,
 // 2] cosines and sines (null: no rotation); interleaved: pairs (2i, 2i+1) instead of (i, i + rope_dim/2).  k_pool null:
-// queries only (a run that reads a cache another run filled).
+// queries only (a run that reads a cache another run filled).  mix_mode 1: the values also go to first_values ([n,
+// kv_heads * value_dim], stride ld_first); 2: the value becomes (1 - share) * value + share * first_values.
 HFEE_API int hfee_attention_prepare(const void* src, long long ld_src, int dtype, int n, int q_off, int k_off, int v_off,
                                     const float* bq, const float* bk, const float* bv, const float* wq, const float* wk,
                                     float eps, const float* cs, int rope_dim, int interleaved, const int* positions,
                                     const int* slot_of_token, void* q_out, long long ld_q, void* k_pool, void* v_pool,
                                     const int* block_table, int max_pages, int page_size, int heads, int kv_heads,
-                                    int key_dim, int value_dim, cudaStream_t stream) {
+                                    int key_dim, int value_dim, void* first_values, long long ld_first, int mix_mode,
+                                    float share, cudaStream_t stream) {
   if (n == 0) return HFEE_OK;
   HFEE_REQUIRE(heads > 0 && kv_heads > 0 && key_dim > 0 && value_dim > 0, "attention_prepare: bad sizes");
+  HFEE_REQUIRE(mix_mode >= MIX_NONE && mix_mode <= MIX_MIX && (mix_mode == MIX_NONE) == (first_values == nullptr) &&
+               (mix_mode == MIX_NONE || (k_pool != nullptr && ld_first >= (long long)kv_heads * value_dim)),
+               "attention_prepare: mixed values need the cache and a buffer of the first ones");
   HFEE_REQUIRE(rope_dim >= 0 && rope_dim % 2 == 0 && rope_dim <= key_dim,
                "attention_prepare: rope_dim %d must be even and at most the key size %d", rope_dim, key_dim);
   HFEE_REQUIRE((k_pool == nullptr) == (v_pool == nullptr), "attention_prepare: keys and values are cached together");
@@ -363,11 +374,12 @@ HFEE_API int hfee_attention_prepare(const void* src, long long ld_src, int dtype
   if (dtype == HFEE_F32)
     hfee_launch(attention_prepare_kernel<float>, dim3(n), dim3(AP_THREADS), smem, stream, (const float*)src, ld_src, q_off, k_off, v_off,
                 bq, bk, bv, wq, wk, eps, cs, rope_dim, interleaved, positions, slot_of_token, (float*)q_out, ld_q, (float*)k_pool, kc,
-                (float*)v_pool, vc, heads, key_dim);
+                (float*)v_pool, vc, heads, key_dim, (float*)first_values, ld_first, mix_mode, share);
   else if (dtype == HFEE_BF16)
     hfee_launch(attention_prepare_kernel<__nv_bfloat16>, dim3(n), dim3(AP_THREADS), smem, stream, (const __nv_bfloat16*)src, ld_src,
                 q_off, k_off, v_off, bq, bk, bv, wq, wk, eps, cs, rope_dim, interleaved, positions, slot_of_token,
-                (__nv_bfloat16*)q_out, ld_q, (__nv_bfloat16*)k_pool, kc, (__nv_bfloat16*)v_pool, vc, heads, key_dim);
+                (__nv_bfloat16*)q_out, ld_q, (__nv_bfloat16*)k_pool, kc, (__nv_bfloat16*)v_pool, vc, heads, key_dim,
+                (__nv_bfloat16*)first_values, ld_first, mix_mode, share);
   else
     return hfee_fail(HFEE_ERR_ARG, "attention_prepare: unknown dtype %d", dtype);
   return hfee_check_launch("attention_prepare");

@@ -10,6 +10,8 @@
 //                         `residual_add` (optional, float32 [n, width], not with `rows`) is added to x first and the
 //                         sum stored back to x: a sublayer's residual update and the next norm in one pass.
 //   hfee_add_bias         x[r, c] += bias[c].
+//   hfee_embed_norm       out[i,:] = table[token_i,:] / sqrt(mean(its squares) + eps) * w (float32): the embedding and the
+//                         RMS norm on it in one pass.
 #include "common.cuh"
 
 namespace {
@@ -221,6 +223,41 @@ __global__ void add_bias_kernel(float* __restrict__ x, long long ld, const float
   x[r * ld + c] += bias[c];
 }
 
+// A block per token; NCH values of the row per thread stay in registers between the passes, wider rows are read twice.
+template <typename T, int NCH>
+__global__ void __launch_bounds__(ROW_THREADS)
+embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ tokens, const int* __restrict__ slot_of_token,
+                  const int* __restrict__ feedback, const float* __restrict__ w, float eps, float* __restrict__ out, int width,
+                  int vocab) {
+  __shared__ float partial[ROW_THREADS / 32];
+  pdl_wait();
+  pdl_launch_dependents();
+  const int i = blockIdx.x;
+  const int tok = token_at(tokens, slot_of_token, feedback, i);
+  const bool ok = tok >= 0 && tok < vocab;
+  const T* row = table + (long long)(ok ? tok : 0) * width;
+  float v[NCH];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NCH; ++j) {
+    const int c = threadIdx.x + j * ROW_THREADS;
+    v[j] = ok && c < width ? to_f32<T>(row[c]) : 0.f;
+    ss = fmaf(v[j], v[j], ss);
+  }
+  for (int c = threadIdx.x + NCH * ROW_THREADS; c < width; c += ROW_THREADS) {
+    const float x = ok ? to_f32<T>(row[c]) : 0.f;
+    ss = fmaf(x, x, ss);
+  }
+  const float scale = 1.0f / sqrtf(block_total<ROW_THREADS>(ss, partial) / (float)width + eps);
+  float* dst = out + (long long)i * width;
+#pragma unroll
+  for (int j = 0; j < NCH; ++j) {
+    const int c = threadIdx.x + j * ROW_THREADS;
+    if (c < width) dst[c] = v[j] * scale * w[c];
+  }
+  for (int c = threadIdx.x + NCH * ROW_THREADS; c < width; c += ROW_THREADS) dst[c] = (ok ? to_f32<T>(row[c]) : 0.f) * scale * w[c];
+}
+
 template <typename TOut>
 void launch_layernorm(float* x, const float* residual_add, const float* w, const int* rows, void* out, long long ld_o, int n,
                       int width, float eps, cudaStream_t stream) {
@@ -255,6 +292,21 @@ HFEE_API int hfee_embed_bigram(const void* table, const void* pairs, int dtype, 
   else
     return hfee_fail(HFEE_ERR_ARG, "embed_bigram: unknown dtype %d", dtype);
   return hfee_check_launch("embed_bigram");
+}
+
+HFEE_API int hfee_embed_norm(const void* table, int dtype, const int* tokens, const int* slot_of_token, const int* feedback,
+                             const float* w, float eps, float* out, int n, int width, int vocab, cudaStream_t stream) {
+  if (n == 0) return HFEE_OK;
+  HFEE_REQUIRE(n > 0 && width > 0 && vocab > 0 && w != nullptr, "embed_norm: bad sizes");
+  if (dtype == HFEE_F32)
+    hfee_launch(embed_norm_kernel<float, 8>, dim3(n), dim3(ROW_THREADS), 0, stream, (const float*)table, tokens, slot_of_token, feedback,
+                w, eps, out, width, vocab);
+  else if (dtype == HFEE_BF16)
+    hfee_launch(embed_norm_kernel<__nv_bfloat16, 8>, dim3(n), dim3(ROW_THREADS), 0, stream, (const __nv_bfloat16*)table, tokens,
+                slot_of_token, feedback, w, eps, out, width, vocab);
+  else
+    return hfee_fail(HFEE_ERR_ARG, "embed_norm: unknown dtype %d", dtype);
+  return hfee_check_launch("embed_norm");
 }
 
 HFEE_API int hfee_remember_tokens(const int* tokens, const int* slot_of_token, const int* feedback, const int* cu_tokens,

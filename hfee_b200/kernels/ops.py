@@ -94,18 +94,24 @@ _SIGNATURES = {
     "hfee_moe_combine": [_P, _P, _P, _I, _I, _P, _I, _I, _P],
     "hfee_moe_plan_tiles": [_P, _I, _I, _I, _P, _P, _P, _I, _P],
     "hfee_moe_gather_rows": [_P, _L, _I, _P, _P, _I, _P, _L, _I, _I, _P],
+    "hfee_moe_route_chosen": [_P, _L, _P, _I, _I, _I, _F, _P, _P, _P],
     "hfee_gemm_tcgen05_grouped": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _P, _I, _F, _F, _F, _P, _P],
     "hfee_gemm_tcgen05_pair_clamped": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _F, _F, _F, _P, _P],
     "hfee_embed_bigram": [_P, _P, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _L, _L, _P],
     "hfee_remember_tokens": [_P, _P, _P, _P, _P, _I, _P, _P],
     "hfee_layernorm": [_P, _P, _P, _P, _P, _L, _I, _I, _I, _F, _P],
     "hfee_add_bias": [_P, _L, _P, _I, _I, _P],
+    "hfee_embed_norm": [_P, _I, _P, _P, _P, _P, _F, _P, _I, _I, _I, _P],
+    "hfee_gate_parts_norm": [_P, _L, _P, _L, _P, _F, _P, _L, _I, _I, _I, _F, _I, _P],
+    "hfee_head_scan": [_P, _P, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _L, _P],
     "hfee_attention_prepare": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _F, _P, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I,
-                               _I, _I, _I, _I, _P],
+                               _I, _I, _I, _I, _P, _L, _I, _F, _P],
+    "hfee_attention_simt_capped": [_P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _L, _I,
+                                   _P, _P, _F, _P, _I, _F, _I, _P],
     "hfee_attention_simt_sink": [_P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _I, _P, _P, _P, _L, _I,
                                  _P, _P, _F, _P, _I, _P],
     "hfee_attention_mma_general": [_P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _P, _P, _P, _F, _I,
-                                   _I, _P, _P],
+                                   _I, _F, _I, _P, _P],
     "hfee_gated_recurrence": [_I, _P, _P, _P, _L, _I, _P, _L, _P, _F, _F, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _P],
     "hfee_gated_recurrence_chunked": [_I, _P, _P, _P, _L, _I, _P, _L, _P, _F, _F, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _P, _L, _P],
     "hfee_head_norm_gate_scaled": [_P, _L, _P, _I, _F, _P, _L, _P, _L, _I, _I, _I, _I, _F, _I, _P],
@@ -414,8 +420,8 @@ def gemm_simt(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: b
 
 STREAM_MAX_TOKENS = 64
 USE_TCGEN05 = True
-EPI_STORE, EPI_ACCUM, EPI_SWIGLU, EPI_GEGLU, EPI_RELU2 = 0, 1, 2, 4, 5      # 5 (tcgen05 kernels only): store relu(x)^2
-EPI_GATED = (EPI_SWIGLU, EPI_GEGLU)         # out = act(gate) * up over rows of w interleaved as [4 gate | 4 up]
+EPI_STORE, EPI_ACCUM, EPI_SWIGLU, EPI_GEGLU, EPI_RELU2, EPI_REGLU = 0, 1, 2, 4, 5, 7      # 5 (tcgen05 kernels only): store relu(x)^2
+EPI_GATED = (EPI_SWIGLU, EPI_GEGLU, EPI_REGLU)         # out = act(gate) * up over rows of w interleaved as [4 gate | 4 up]
 
 
 def _streamable(a: torch.Tensor, w: torch.Tensor) -> bool:
@@ -683,11 +689,11 @@ SWIGLU_GRANULE = 4
 
 def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, granule: int,
                   scratch: torch.Tensor, activation: str = "silu") -> None:
-    """out = act(a @ w_gate^T) * (a @ w_up^T) (``activation``: ``"silu"`` or ``"gelu_tanh"``) where ``w_gate_up`` holds the rows of both in groups
+    """out = act(a @ w_gate^T) * (a @ w_up^T) (``activation``: ``"silu"``, ``"gelu_tanh"`` or ``"relu"``) where ``w_gate_up`` holds the rows of both in groups
     of ``granule`` gate rows followed by ``granule`` up rows; ``scratch`` [m, 2*inner] holds the
     projection when it is not fused."""
     fusable = granule == SWIGLU_GRANULE and w_gate_up.shape[0] % 8 == 0
-    epilogue = EPI_SWIGLU if activation == "silu" else EPI_GEGLU
+    epilogue = GATED_EPILOGUES[activation]
     if fusable and _streamable(a, w_gate_up):
         _small_gemm(a, w_gate_up, out, epilogue)
     elif fusable and USE_TCGEN05 and _tensor_core_ok(a, w_gate_up) and out.dtype == torch.bfloat16:
@@ -697,9 +703,12 @@ def linear_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, g
         gated_act(scratch, out, activation, granule)
 
 
+GATED_EPILOGUES = {"silu": EPI_SWIGLU, "gelu_tanh": EPI_GEGLU, "relu": EPI_REGLU}
+
+
 def linear_gated_normed(inp, w_gate_up: torch.Tensor, out: torch.Tensor, granule: int, scratch: torch.Tensor,
                         activation: str) -> None:
-    """:func:`linear_swiglu` with another gate activation (``"gelu_tanh"``): in the product's epilogue where a
+    """:func:`linear_swiglu` with another gate activation (``"gelu_tanh"``, ``"relu"``): in the product's epilogue where a
     kernel with gated epilogues takes the shape, else through ``scratch`` [m, 2*inner] and :func:`gated_act`."""
     a = inp if isinstance(inp, torch.Tensor) else inp.tensor()
     linear_swiglu(a, w_gate_up, out, granule, scratch, activation)
@@ -870,7 +879,7 @@ def paged_attention_rope(qkv, cs, rope_dim, interleaved, write_cache, k_pool, v_
 # ---------------------------------------------------------------------------- mechanisms beside softmax attention
 WEIGHTS_SOFTMAX, WEIGHTS_SIGMOID = 0, 1
 ACTIVATIONS = {"none": 0, "silu": 1}
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu": 2}
 
 
 def attention_simt_masked(q, k_pool, v_pool, block_table, page_size, positions, slot_of_token, out, heads, kv_heads,
@@ -1500,7 +1509,7 @@ def norm_gate(x: torch.Tensor, weight: Optional[torch.Tensor], eps: float, gate:
 
 
 def gated_act(gate_up: torch.Tensor, out: torch.Tensor, activation: str, granule: Optional[int] = None) -> None:
-    """out[i, c] = act(gate) * up with the column layout of :func:`swiglu`; ``activation`` is ``"silu"`` or
+    """out[i, c] = act(gate) * up with the column layout of :func:`swiglu`; ``activation`` is ``"silu"``, ``"relu"`` or
     ``"gelu_tanh"`` (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))))."""
     lib = library()
     n, inter = out.shape
@@ -1654,6 +1663,21 @@ def moe_route_grouped(logits: torch.Tensor, experts: int, top: int, groups: int,
     assert tuple(choice.shape) == (n, top) and tuple(weight.shape) == (n, top) and weight.is_contiguous()
     _check(lib.hfee_moe_route_grouped(logits.data_ptr(), logits.stride(0), n, experts, top, groups, keep, float(scale),
                                       choice.data_ptr(), weight.data_ptr(), _stream()), lib)
+
+
+def moe_route_chosen(logits: torch.Tensor, experts: int, top: int, scale: float, choice: torch.Tensor, weight: torch.Tensor,
+                     bias: Optional[torch.Tensor] = None) -> None:
+    """Per row of ``logits`` (float32; the first ``experts`` columns) plus ``bias`` (float32 per expert, optional): the ``top``
+    largest (ties: the lower expert) into ``choice`` [n, top] int32, and ``scale`` times the softmax over just those into
+    ``weight`` [n, top] float32."""
+    lib = library()
+    n = logits.shape[0]
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1 and logits.shape[1] >= experts and weight.dtype == torch.float32
+    assert bias is None or (bias.dtype == torch.float32 and bias.is_contiguous() and bias.numel() == experts)
+    _i32(choice, "choice")
+    assert tuple(choice.shape) == (n, top) and tuple(weight.shape) == (n, top) and weight.is_contiguous()
+    _check(lib.hfee_moe_route_chosen(logits.data_ptr(), logits.stride(0), _ptr(bias), n, experts, top, float(scale), choice.data_ptr(),
+                                     weight.data_ptr(), _stream()), lib)
 
 
 def moe_plan(choice: torch.Tensor, experts: int, offsets: torch.Tensor, order: torch.Tensor, tile_expert: torch.Tensor,
@@ -1883,15 +1907,32 @@ def add_bias(x: torch.Tensor, bias: torch.Tensor) -> None:
     _check(lib.hfee_add_bias(x.data_ptr(), _rows(x, "x"), bias.data_ptr(), x.shape[0], x.shape[1], _stream()), lib)
 
 
+def embed_norm(table: torch.Tensor, tokens: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+               slot_of_token: Optional[torch.Tensor] = None, feedback: Optional[torch.Tensor] = None) -> None:
+    """out[i] = table[tokens[i]] / sqrt(mean of its squares + eps) * weight in float32; ``feedback`` as in :func:`embed`."""
+    lib = library()
+    _i32(tokens, "embed tokens"); _i32(slot_of_token, "slot_of_token"); _i32(feedback, "feedback")
+    n, width = out.shape
+    assert out.dtype == weight.dtype == torch.float32 and out.is_contiguous() and table.is_contiguous()
+    assert weight.is_contiguous() and weight.numel() == width == table.shape[1] and (feedback is None or slot_of_token is not None)
+    _check(lib.hfee_embed_norm(table.data_ptr(), _dt(table), tokens.data_ptr(), _ptr(slot_of_token), _ptr(feedback), weight.data_ptr(),
+                               float(eps), out.data_ptr(), n, width, table.shape[0], _stream()), lib)
+
+
+VALUES_AS_THEY_ARE, VALUES_STORE_FIRST, VALUES_MIX = 0, 1, 2
+
+
 def attention_prepare(src: torch.Tensor, q_off: int, k_off: int, v_off: int, heads: int, kv_heads: int, key_dim: int,
                       value_dim: int, step, q_out: torch.Tensor, k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor],
                       block_table: torch.Tensor, page_size: int, cs: Optional[torch.Tensor] = None, rope_dim: int = 0,
-                      interleaved: bool = False, biases=(None, None, None), norm_weights=(None, None), eps: float = 0.0) -> None:
+                      interleaved: bool = False, biases=(None, None, None), norm_weights=(None, None), eps: float = 0.0,
+                      first_values: Optional[torch.Tensor] = None, value_mix: int = VALUES_AS_THEY_ARE, share: float = 0.0) -> None:
     """One token's [q | k | v] projection on its way to the score kernel: ``biases`` = (q, k, v) float32 per column (each may
     be None), ``norm_weights`` = (q, k) weights of an RMS norm over the whole query / key projection (None: no norm),
     then the rotation of the first ``rope_dim`` dimensions of every head by the step's (cos, sin) table ``cs``, pairing
     (i, i + rope_dim/2) or, ``interleaved``, (2i, 2i + 1).  Queries to ``q_out``, keys and values to their pages (pools None:
-    queries only)."""
+    queries only).  ``value_mix``: VALUES_STORE_FIRST also leaves the values in ``first_values`` [n, kv_heads * value_dim],
+    VALUES_MIX caches (1 - share) * value + share * first_values in place of the value."""
     lib = library()
     n = src.shape[0]
     _i32(block_table, "block_table")
@@ -1902,22 +1943,26 @@ def attention_prepare(src: torch.Tensor, q_off: int, k_off: int, v_off: int, hea
     if k_pool is not None:
         assert k_pool.dtype == v_pool.dtype == src.dtype and k_pool.is_contiguous() and v_pool.is_contiguous()
         assert tuple(k_pool.shape[1:]) == (kv_heads, page_size, key_dim) and tuple(v_pool.shape[1:]) == (kv_heads, page_size, value_dim)
+    assert (value_mix == VALUES_AS_THEY_ARE) == (first_values is None)
+    assert first_values is None or (first_values.dtype == src.dtype and tuple(first_values.shape) == (n, kv_heads * value_dim))
     _check(lib.hfee_attention_prepare(src.data_ptr(), _rows(src, "src"), _dt(src), n, q_off, k_off, v_off, _ptr(biases[0]),
                                       _ptr(biases[1]), _ptr(biases[2]), _ptr(norm_weights[0]), _ptr(norm_weights[1]), float(eps),
                                       _ptr(cs), int(rope_dim) if cs is not None else 0, int(interleaved), step.positions.data_ptr(),
                                       step.slot_of_token.data_ptr(), q_out.data_ptr(), _rows(q_out, "q_out"), _ptr(k_pool),
                                       _ptr(v_pool), block_table.data_ptr(), block_table.shape[1], page_size, heads, kv_heads,
-                                      key_dim, value_dim, _stream()), lib)
+                                      key_dim, value_dim, _ptr(first_values), _rows(first_values, "first values") if value_mix else 0,
+                                      int(value_mix), float(share), _stream()), lib)
 
 
 SOFTMAX_ATTENTION_ON_TENSOR_CORES = True
 
 
 def softmax_attention(q, k_pool, v_pool, block_table, page_size, step, out, heads, kv_heads, head_dim, value_dim, scale,
-                      window=0, sink=None, out_scale=1.0, scratch=None) -> None:
+                      window=0, sink=None, out_scale=1.0, scratch=None, keep_first=0, softcap=None) -> None:
     """Causal grouped-query softmax attention over the paged cache with key and value sizes of their own, an optional
     window, an optional ``sink`` (float32 per query head: the denominator also holds exp(sink[h]), a term without key or
-    value) and the output times ``out_scale``.  bfloat16 with key and value sizes that are multiples of 8 (up to 256) runs
+    value) and the output times ``out_scale``.  ``keep_first``: that many positions from the start stay visible behind the
+    window; ``softcap`` c: a scaled score s becomes c * tanh(s / c).  bfloat16 with key and value sizes that are multiples of 8 (up to 256) runs
     on the tensor cores (prompt portions, decode steps with their keys split among CTAs when ``scratch`` is given, and
     mixtures), everything else on the CUDA cores in float32 arithmetic."""
     lib = library()
@@ -1927,26 +1972,30 @@ def softmax_attention(q, k_pool, v_pool, block_table, page_size, step, out, head
     assert k_pool.is_contiguous() and v_pool.is_contiguous() and v_pool.dtype == q.dtype
     assert tuple(k_pool.shape[1:]) == (kv_heads, page_size, head_dim) and tuple(v_pool.shape[1:]) == (kv_heads, page_size, value_dim)
     _i32(block_table, "block_table")
+    cap = 0.0 if softcap is None else float(softcap)
     tile = distance_attention_tile(head_dim, value_dim) if (SOFTMAX_ATTENTION_ON_TENSOR_CORES and q.dtype == torch.bfloat16) else 0
     if not (tile and group <= 64 and _rows(q, "q") % 8 == 0 and q.data_ptr() % 16 == 0 and _rows(out, "out") % 4 == 0
             and out.data_ptr() % 8 == 0):
-        _check(lib.hfee_attention_simt_sink(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), v_pool.data_ptr(), block_table.data_ptr(),
-                                            block_table.shape[1], page_size, step.positions.data_ptr(), step.slot_of_token.data_ptr(),
-                                            out.data_ptr(), _rows(out, "attention out"), step.n, heads, kv_heads, head_dim,
-                                            value_dim, 0, float(scale), int(window or 0), 0, WEIGHTS_SOFTMAX, None, None, None, 0,
-                                            GATE_NONE, None, None, float(out_scale), _ptr(sink), _dt(q), _stream()), lib)
+        _check(lib.hfee_attention_simt_capped(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), v_pool.data_ptr(), block_table.data_ptr(),
+                                              block_table.shape[1], page_size, step.positions.data_ptr(), step.slot_of_token.data_ptr(),
+                                              out.data_ptr(), _rows(out, "attention out"), step.n, heads, kv_heads, head_dim,
+                                              value_dim, 0, float(scale), int(window or 0), 0, WEIGHTS_SOFTMAX, None, None, None, 0,
+                                              GATE_NONE, None, None, float(out_scale), _ptr(sink), int(keep_first), cap, _dt(q),
+                                              _stream()), lib)
         return
     splits = 1
     if step.max_new * group <= 16 and scratch is not None:
-        splits = getattr(step, "attention_splits", None) or attention_splits(
-            step.r, kv_heads, getattr(step, "planning_context", step.max_context))
+        keys = getattr(step, "planning_context", step.max_context)
+        if window:                              # no more keys than these are ever visited
+            keys = min(keys, int(window) + int(keep_first) + 128)
+        splits = getattr(step, "attention_splits", None) or attention_splits(step.r, kv_heads, keys)
         if step.n * heads * splits * (tile + 2) > scratch.numel():
             splits = 1
     _check(lib.hfee_attention_mma_general(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), v_pool.data_ptr(), block_table.data_ptr(),
                                           block_table.shape[1], page_size, step.cu_tokens.data_ptr(), step.slots.data_ptr(),
                                           step.context_before.data_ptr(), out.data_ptr(), _rows(out, "attention out"), step.n,
                                           step.r, step.max_new, heads, kv_heads, head_dim, value_dim, float(scale), None, None,
-                                          _ptr(sink), float(out_scale), int(window or 0), splits,
+                                          _ptr(sink), float(out_scale), int(window or 0), int(keep_first), cap, splits,
                                           _ptr(scratch) if splits > 1 else None, _stream()), lib)
     if splits > 1:
         count_launches(1)
@@ -1997,6 +2046,59 @@ def gated_recurrence(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tenso
                                      _ptr(bias), float(p0), float(q_scale), state.data_ptr(), _ptr(norm_state), _ptr(max_state),
                                      step.cu_tokens.data_ptr(), step.slots.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r,
                                      heads, dim, vdim, int(write_state), _stream()), lib)
+
+
+HEAD_SCAN_RUNS_MIN = 65            # from this many new tokens of one request on, runs of 64 tokens work side by side
+
+
+def head_scan(x: torch.Tensor, bmat: torch.Tensor, cmat: torch.Tensor, step_size: torch.Tensor, dt_bias: torch.Tensor,
+              a_log: torch.Tensor, d_skip: torch.Tensor, state: torch.Tensor, step, out: torch.Tensor, heads: int, groups: int,
+              state_dim: int, vdim: int, write_state: bool = True, workspace: Optional[torch.Tensor] = None) -> None:
+    """A state-space scan with one decay per head and token: dt = softplus(step_size + dt_bias); S = exp(-exp(a_log) dt) S +
+    dt B x^T; out = S^T C + d_skip x per head, S [state_dim, vdim] float32 from ``state`` [slots, heads, state_dim, vdim],
+    which is renewed.  ``x`` [n, heads * vdim], ``bmat`` and ``cmat`` [n, groups * state_dim] are column slices of one buffer
+    (head h uses group h / (heads / groups)), ``step_size`` [n, heads] has a row stride of its own; ``out`` [n, heads * vdim]
+    float32.  Portions of HEAD_SCAN_RUNS_MIN tokens and more take runs of 64 tokens side by side when ``workspace`` (float32,
+    :func:`head_scan_workspace`) is given."""
+    lib = library()
+    ld = _rows(x, "x")
+    n = x.shape[0]
+    assert _rows(bmat, "B") == ld and _rows(cmat, "C") == ld and x.dtype == bmat.dtype == cmat.dtype == step_size.dtype
+    assert x.shape[1] == heads * vdim and bmat.shape[1] == cmat.shape[1] == groups * state_dim and tuple(step_size.shape) == (n, heads)
+    assert out.dtype == torch.float32 and tuple(out.shape) == (n, heads * vdim)
+    for t in (dt_bias, a_log, d_skip):
+        assert t.dtype == torch.float32 and t.is_contiguous() and t.numel() == heads
+    assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, state_dim, vdim)
+    runs = workspace is not None and step.max_new >= HEAD_SCAN_RUNS_MIN
+    assert workspace is None or (workspace.dtype == torch.float32 and workspace.is_contiguous())
+    _check(lib.hfee_head_scan(x.data_ptr(), bmat.data_ptr(), cmat.data_ptr(), ld, step_size.data_ptr(), _rows(step_size, "step"), _dt(x),
+                              dt_bias.data_ptr(), a_log.data_ptr(), d_skip.data_ptr(), state.data_ptr(), step.cu_tokens.data_ptr(),
+                              step.slots.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r, n, heads, groups, state_dim, vdim,
+                              int(write_state), _ptr(workspace) if runs else None, workspace.numel() if runs else 0, _stream()), lib)
+    if runs:
+        count_launches(3)
+
+
+def head_scan_takes_workspace(step) -> bool:
+    """Whether a step has a portion long enough for the paths of :func:`head_scan` that need a workspace."""
+    return step.max_new >= HEAD_SCAN_RUNS_MIN
+
+
+def head_scan_workspace(requests: int, tokens: int, heads: int, state_dim: int, vdim: int) -> int:
+    """Floats of workspace :func:`head_scan` wants for steps of at most ``tokens`` tokens of ``requests`` requests."""
+    return gated_recurrence_workspace(requests, tokens, heads, state_dim, vdim)
+
+
+def gate_parts_norm(x: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, parts: int, out: torch.Tensor,
+                    out_scale: float = 1.0) -> None:
+    """g = x * silu(z); every one of ``parts`` equal parts of a row of g divided by its own root mean square (eps inside the
+    root), times ``weight`` per column and ``out_scale``.  ``x`` and ``weight`` float32; ``z`` and ``out`` share a dtype."""
+    lib = library()
+    n, width = x.shape
+    assert x.dtype == weight.dtype == torch.float32 and weight.is_contiguous() and weight.numel() == width
+    assert z.dtype == out.dtype and z.shape == x.shape == out.shape
+    _check(lib.hfee_gate_parts_norm(x.data_ptr(), _rows(x, "x"), z.data_ptr(), _rows(z, "z"), weight.data_ptr(), float(eps), out.data_ptr(),
+                                    _rows(out, "out"), n, width, int(parts), float(out_scale), _dt(out), _stream()), lib)
 
 
 def head_norm_gate_scaled(x: torch.Tensor, weight: torch.Tensor, eps: float, gate: torch.Tensor, out: torch.Tensor, heads: int,
@@ -2100,6 +2202,7 @@ for _name in ("rmsnorm_add_norm", "latent_attention", "linear_act", "attention_s
               "linear_swiglu_normed", "paged_attention", "paged_attention_rope", "sample", "argmax", "sample_chain",
               "mingru", "selective_scan", "distance_attention", "moe_route", "moe_plan", "moe_experts", "moe_experts_grouped", "moe_combine",
               "clamped_glu", "linear_clamped_glu", "depth_average", "scaled_add_norm", "scaled_add", "add_sinusoid", "softcap_",
-              "channel_delta", "stream_step", "latent_attend_prepare"):
+              "channel_delta", "stream_step", "latent_attend_prepare", "softmax_attention", "attention_prepare", "gated_recurrence",
+              "head_norm_gate_scaled", "moe_route_grouped", "moe_route_chosen", "head_scan", "gate_parts_norm", "embed_norm"):
     globals()[_name] = _measurable(globals()[_name])
 del _name

@@ -1,2 +1,2 @@
 """Architectures: each module registers itself in ``hfee_b200.config.registry``."""
-from . import bamipel, dobelix, fokalorn, llama, muvetar, pupinex  # noqa: F401
+from . import bamipel, bumisun, dobelix, fokalorn, llama, muvetar, pupinex  # noqa: F401

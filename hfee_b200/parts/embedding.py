@@ -13,14 +13,18 @@ from .base import Part, register_part
 
 class TokenEmbedding(Part):
     """``x[i,:] = table[token_i,:] * scale`` (hostfog/hfee internal/llm/forward.go:75-77 has no scale).
-    spec: ``vocab``, ``width``, ``scale`` (default 1), ``sinusoid_base`` (default None; a base b adds the token's
+    spec: ``vocab``, ``width``, ``scale`` (default 1), ``norm_eps`` (default None; else the row is RMS-normed with the weight
+    ``"norm"``, in the same kernel), ``sinusoid_base`` (default None; a base b adds the token's
     position p as ``sin(p * b^(-2i/width))`` to entry 2i and the cosine of the same angle to entry 2i + 1)."""
     category = "embedding"
     graph_safe = True
 
     @staticmethod
     def tensor_needs(spec: PartSpec) -> Dict[str, TensorNeed]:
-        return {"table": TensorNeed((spec.vocab, spec.width), role="table")}
+        needs = {"table": TensorNeed((spec.vocab, spec.width), role="table")}
+        if spec.get("norm_eps") is not None:
+            needs["norm"] = TensorNeed((spec.width,), role="scale")
+        return needs
 
     def __init__(self, spec, tensors, rt):
         super().__init__(spec, tensors, rt)
@@ -28,11 +32,20 @@ class TokenEmbedding(Part):
         self.scale = float(spec.get("scale", 1.0))
         base = spec.get("sinusoid_base")
         self.sinusoid_base = None if base is None else float(base)
+        eps = spec.get("norm_eps")
+        self.norm_eps = None if eps is None else float(eps)
+        self.norm_weight = tensors.get("norm")
+        if self.norm_eps is not None and self.scale != 1.0:
+            raise ValueError("a normed embedding has no scale")
 
     def forward(self, step: Any, residual: torch.Tensor) -> None:
         ops.tag("embed")
-        ops.embed(self.table, step.token_ids, residual, step.slot_of_token, getattr(step, "feedback", None),
-                  scale=self.scale)
+        if self.norm_eps is not None:
+            ops.embed_norm(self.table, step.token_ids, self.norm_weight, self.norm_eps, residual, step.slot_of_token,
+                           getattr(step, "feedback", None))
+        else:
+            ops.embed(self.table, step.token_ids, residual, step.slot_of_token, getattr(step, "feedback", None),
+                      scale=self.scale)
         if self.sinusoid_base is not None:
             ops.add_sinusoid(residual, step.positions, self.sinusoid_base)
 

@@ -1,6 +1,6 @@
 """Dense gated feed-forward: ``down(act(gate(x)) * up(x))`` added to the residual
 stream; ``act`` is SiLU (hostfog/hfee internal/llm/forward.go:110-114, internal/ggml/ops.go:160-165)
-or the tanh form of GELU."""
+the tanh form of GELU, or relu."""
 from __future__ import annotations
 
 from typing import Any, Dict
@@ -14,8 +14,8 @@ from .base import Part, register_part
 
 
 class SwiGLUFeedForward(Part):
-    """spec: ``width``, ``inner`` (intermediate size), ``activation`` (``"silu"``, the default, or
-    ``"gelu_tanh"``).  ``forward(..., accumulate=False)`` stores the output instead of adding it."""
+    """spec: ``width``, ``inner`` (intermediate size), ``activation`` (``"silu"``, the default,
+    ``"gelu_tanh"`` or ``"relu"``).  ``forward(..., accumulate=False)`` stores the output instead of adding it."""
     can_overwrite = True
     category = "feed_forward"
     graph_safe = True

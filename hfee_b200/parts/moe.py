@@ -6,7 +6,9 @@
 
 The chosen weights are not renormalised.  ``router`` = ``"sigmoid_groups"`` is another router: s = sigmoid(W_router h);
 the experts form ``groups`` equal groups of neighbours, a group's score is the sum of its two largest s, only experts of the
-``keep`` best groups can be chosen, and the chosen s are divided by their sum (+ 1e-20) before the scale.  ``limit`` None
+``keep`` best groups can be chosen, and the chosen s are divided by their sum (+ 1e-20) before the scale.  ``"softmax_chosen"``: the
+``top`` largest logits W_router h + b are chosen (``b``, tensor ``router.b``, with ``router_bias``), and their weights are the
+softmax over the chosen logits only, times the scale.  ``limit`` None
 means no clamp (with alpha = 1 and shift = 0 the expert is silu(gate) * up), and ``shared_gate`` multiplies the shared
 expert's output by sigmoid(W_sg h), one number per token.  The experts' tensors are stacked at load time (``[experts, 2 * inner, width]``,
 each expert's gate rows and then its up rows, and ``[experts, width, inner]``); the (token, choice) pairs are ordered by
@@ -32,7 +34,7 @@ from .gated_attention import pad8
 class RoutedExperts(Part):
     """spec: ``width``, ``experts``, ``top``, ``router_scale``, ``inner``, ``limit``, ``alpha``, ``shared_inner`` and
     ``shared_limit`` (``shared_inner`` None: no shared expert); optional: ``shift`` (default 1), ``router`` (``"softmax"``,
-    the default, or ``"sigmoid_groups"`` with ``groups`` and ``keep``), ``shared_gate`` (default False; tensor
+    the default, ``"softmax_chosen"`` with ``router_bias``, or ``"sigmoid_groups"`` with ``groups`` and ``keep``), ``shared_gate`` (default False; tensor
     ``shared.sg`` [1, width]).  ``forward(..., accumulate=False)`` stores the output."""
     category = "feed_forward"
     graph_safe = True
@@ -42,6 +44,8 @@ class RoutedExperts(Part):
     def tensor_needs(spec: PartSpec) -> Dict[str, TensorNeed]:
         w, f = spec.width, spec.inner
         needs = {"router": TensorNeed((spec.experts, w))}
+        if spec.get("router_bias"):
+            needs["router.b"] = TensorNeed((spec.experts,), role="vector")
         for e in range(spec.experts):
             needs[f"e{e}.gate"] = TensorNeed((f, w))
             needs[f"e{e}.up"] = TensorNeed((f, w))
@@ -69,15 +73,18 @@ class RoutedExperts(Part):
                 raise ValueError(f"{self.experts} experts do not form {self.groups} equal groups of which {self.keep} are kept")
             if self.top > self.keep * (self.experts // self.groups):
                 raise ValueError(f"top {self.top} exceeds the {self.keep * (self.experts // self.groups)} experts of the kept groups")
-        elif self.router != "softmax":
-            raise ValueError(f"unknown router {self.router!r} (known: softmax, sigmoid_groups)")
+        elif self.router not in ("softmax", "softmax_chosen"):
+            raise ValueError(f"unknown router {self.router!r} (known: softmax, softmax_chosen, sigmoid_groups)")
+        self.router_bias = tensors.get("router.b")
+        if self.router_bias is not None and self.router != "softmax_chosen":
+            raise ValueError("a router bias goes with the softmax_chosen router")
         self.w_router = tensors["router"]
         self.shared_gate = spec.get("shared_inner") is not None and bool(spec.get("shared_gate", False))
         if self.shared_gate:
-            # the shared expert's gate rides in the router's product as one more row; the grouped router reads its rows
-            # with a stride, the softmax router does not
-            if self.router != "sigmoid_groups":
-                raise ValueError("a gated shared expert goes with the sigmoid_groups router")
+            # the shared expert's gate rides in the router's product as one more row; the other routers read their rows
+            # with a stride, the softmax router over all experts does not
+            if self.router == "softmax":
+                raise ValueError("a gated shared expert goes with the sigmoid_groups or the softmax_chosen router")
             self.w_router = torch.cat([tensors["router"], tensors["shared.sg"]], dim=0).contiguous()
         pairs = rt.max_tokens * self.top
         self.grouped = ops.moe_experts_grouped_ok(rt.dtype, self.width, self.inner)
@@ -116,6 +123,8 @@ class RoutedExperts(Part):
         ops.linear(xn, self.w_router, logits)
         if self.router == "sigmoid_groups":
             ops.moe_route_grouped(logits, self.experts, top, self.groups, self.keep, self.router_scale, choice, weight)
+        elif self.router == "softmax_chosen":
+            ops.moe_route_chosen(logits, self.experts, top, self.router_scale, choice, weight, self.router_bias)
         else:
             ops.moe_route(logits, top, self.router_scale, choice, weight)
         gate_col = logits[:, self.experts:] if self.shared_gate else None

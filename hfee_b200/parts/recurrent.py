@@ -1,4 +1,4 @@
-"""Mixers built on an elementwise linear recurrence S_t = a_t S_(t-1) + b_t with a float32 state per request.
+"""Mixers built on a linear recurrence S_t = a_t S_(t-1) + b_t with a float32 state per request.
 
 ``mingru``: the gates read only the current token.  With h the mixer's input::
 
@@ -13,10 +13,17 @@ short causal convolution::
     S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n              y_c = sum_n S[c, n] C_n + D_c x_c
     out = W_o (y * silu(z))
 
+``head_scan``: a state-space scan with one decay per head and token, whose input and read-out vectors are shared by groups of
+heads (state-space duality, as in Mamba-2)::
+
+    [z | x | B | C | dt] = W_in h                        (x, B, C) = silu(conv(x, B, C) + b_conv)
+    dt = softplus(dt + b_dt)                             S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T   (per head)
+    y_t = S_t^T C_t + D x_t                              out = W_o (norm_in_parts(y * silu(z)) * w)
+
 States start at zero and belong to the request (as do the convolution's last ``taps - 1`` inputs), so a prompt may be
 cut anywhere.  Gates, step sizes, decays and states are float32; the projections are the activations' dtype.
 
-Both are *split mixers*: ``in_weight`` (the rows of their input projection), ``inner_cols`` and ``w_o`` are public and
+All are *split mixers*: ``in_weight`` (the rows of their input projection), ``inner_cols`` and ``w_o`` are public and
 ``mix(proj, step, cache, writes_cache, into, out_scale)`` leaves what W_o reads, times ``out_scale``, in ``into``, so
 that a mixer that runs several of them side by side can project once in and once out.  A split mixer may also carry
 ``out_bias`` (added after W_o) and set ``needs_input`` (its ``mix`` then gets the mixer's input as ``h=`` for a small
@@ -139,5 +146,72 @@ class SelectiveScan(SplitMixer):
                            self.dt_bias, cache.states["recurrent"], step, into, out_scale, writes_cache)
 
 
+class HeadScan(SplitMixer):
+    """spec: ``width``, ``heads``, ``head_dim`` (size of a head's x), ``state`` (entries of B and C), ``groups`` (of heads that
+    share B and C), ``taps``, ``norm_parts``, ``eps``.  Tensors: ``in`` [2 * heads * head_dim + 2 * groups * state + heads, width]
+    (rows z, x, B, C, dt), ``conv`` [channels, taps] and ``conv_bias`` over x, B and C together, ``dt_bias``, ``A_log``, ``D``
+    [heads], ``norm`` [heads * head_dim], ``o``."""
+
+    @staticmethod
+    def tensor_needs(spec: PartSpec) -> Dict[str, TensorNeed]:
+        inner, bc, h, w = spec.heads * spec.head_dim, spec.groups * spec.state, spec.heads, spec.width
+        vector = lambda *shape: TensorNeed(shape, role="vector")
+        return {"in": TensorNeed((2 * inner + 2 * bc + h, w)), "conv": vector(inner + 2 * bc, spec.taps), "conv_bias": vector(inner + 2 * bc),
+                "dt_bias": vector(h), "A_log": vector(h), "D": vector(h), "norm": TensorNeed((inner,), role="scale"),
+                "o": TensorNeed((w, inner))}
+
+    def __init__(self, spec, tensors, rt):
+        super().__init__(spec, tensors, rt)
+        self.heads, self.head_dim, self.n_state, self.groups = int(spec.heads), int(spec.head_dim), int(spec.state), int(spec.groups)
+        self.taps, self.norm_parts, self.eps = int(spec.taps), int(spec.norm_parts), float(spec.eps)
+        if self.heads % self.groups:
+            raise ValueError(f"heads {self.heads} must be a multiple of groups {self.groups}")
+        if self.taps < 1:
+            raise ValueError(f"a convolution needs at least one tap, got {self.taps}")
+        self.inner, self.bc = self.heads * self.head_dim, self.groups * self.n_state
+        if self.inner % self.norm_parts:
+            raise ValueError(f"{self.norm_parts} parts do not divide {self.inner} columns")
+        self.conv_cols = self.inner + 2 * self.bc
+        # rows x, B, C, then z, then dt, each from a multiple of eight on, so that every piece starts on 16 bytes
+        self.z_at = pad8(self.conv_cols)
+        self.dt_at = pad8(self.z_at + self.inner)
+        w = tensors["in"]
+        self.in_weight = torch.zeros((self.dt_at + self.heads, w.shape[1]), dtype=w.dtype, device=w.device)
+        self.in_weight[:self.conv_cols] = w[self.inner:self.inner + self.conv_cols]
+        self.in_weight[self.z_at:self.z_at + self.inner] = w[:self.inner]
+        self.in_weight[self.dt_at:] = w[self.inner + self.conv_cols:]
+        self.conv_weight, self.conv_bias = tensors["conv"], tensors["conv_bias"]
+        self.dt_bias, self.a_log, self.d_skip, self.norm_weight = tensors["dt_bias"], tensors["A_log"], tensors["D"], tensors["norm"]
+        self.w_o = tensors["o"]
+        self.inner_cols, self.in_rows = self.inner, self.in_weight.shape[0]
+
+    def cache_need(self) -> CacheBundle:
+        return CacheBundle.of(None, conv=FixedState((self.taps - 1, self.conv_cols), "float32"),
+                              recurrent=FixedState((self.heads, self.n_state, self.head_dim), "float32"))
+
+    def mix(self, proj, step, cache, writes_cache, into, out_scale: float = 1.0) -> None:
+        n, rt = step.n, self.rt
+        xbc = rt.scratch("scan_conv", (rt.max_tokens, pad8(self.conv_cols)))[:n, :self.conv_cols]
+        ops.tag("conv")
+        ops.conv_act(proj[:, :self.conv_cols], self.conv_weight, cache.states["conv"], step, xbc, "silu", writes_cache, bias=self.conv_bias)
+        y = rt.scratch("head_scan_out", (rt.max_tokens, self.inner), torch.float32)[:n]
+        ops.tag("scan")
+        b, c = self.inner, self.inner + self.bc
+        ops.head_scan(xbc[:, :b], xbc[:, b:c], xbc[:, c:c + self.bc], proj[:, self.dt_at:self.dt_at + self.heads], self.dt_bias,
+                      self.a_log, self.d_skip, cache.states["recurrent"], step, y, self.heads, self.groups, self.n_state, self.head_dim,
+                      writes_cache, self._workspace(step))
+        ops.tag("gate")
+        ops.gate_parts_norm(y, proj[:, self.z_at:self.z_at + self.inner], self.norm_weight, self.eps, self.norm_parts, into, out_scale)
+
+    def _workspace(self, step):
+        """The prompt path's workspace, sized once for the engine's limits, for steps that take that path."""
+        rt = self.rt
+        if not ops.head_scan_takes_workspace(step):
+            return None
+        return rt.scratch("head_scan_work", (ops.head_scan_workspace(rt.max_requests, rt.max_tokens, self.heads, self.n_state, self.head_dim),),
+                          torch.float32)
+
+
 register_part("mixer", "mingru", MinGRU)
+register_part("mixer", "head_scan", HeadScan)
 register_part("mixer", "selective_scan", SelectiveScan)
