@@ -99,8 +99,9 @@ attention_simt_kernel(const T* __restrict__ q, int ld_q, const T* __restrict__ k
         if (d < vd) o[j] = fmaf(pt, to_f32<T>(vr[d]), o[j]);
       }
     }
+    const bool front = base < kept;
     base += 32;
-    if (base >= kept && base < lo) base = lo;
+    if (front && base >= kept) base = lo;
   }
   T* orow = out + (long long)i * ld_o + (long long)h * vd;
   float inv = (SIGMOID ? 1.f : 1.f / l) * out_scale;
