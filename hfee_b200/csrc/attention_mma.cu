@@ -387,7 +387,6 @@ attention_mma_kernel(AttnParams p) {
       for (int j = 0; j < 4; ++j) s[i][j] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < HD / 16; ++ks) {
-      if (DIST && ks * 16 >= kdim) break;                 // tiles are as wide as the larger of the two sizes
       uint32_t a[4];
       ldmatrix_x4(a, q_s + (wrow + (lane & 15)) * PITCH + ks * 16 + (lane >> 4) * 8);
 #pragma unroll
@@ -485,7 +484,6 @@ attention_mma_kernel(AttnParams p) {
       a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
       for (int dp = 0; dp < HD / 16; ++dp) {
-        if (DIST && dp * 16 >= vdim) break;
         uint32_t vb[4];
         ldmatrix_x4_trans(vb, vt + (wkey + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PITCH + dp * 16 + (lane >> 4) * 8);
         mma_bf16(o_acc[2 * dp], a, vb[0], vb[1]);

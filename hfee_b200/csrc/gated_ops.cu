@@ -557,12 +557,61 @@ gate_parts_norm_kernel(const float* __restrict__ x, long long ld_x, const T* __r
   }
 }
 
+// Short parts (at most 128 * NV columns, vector accesses): a warp per (row, part), the part in registers.
+template <typename T, int NV>
+__global__ void __launch_bounds__(ROW_THREADS)
+gate_parts_norm_warp_kernel(const float* __restrict__ x, long long ld_x, const T* __restrict__ z, long long ld_z,
+                            const float* __restrict__ w, float eps, T* __restrict__ out, long long ld_o, int parts, int part,
+                            float out_scale, unsigned tasks) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const unsigned task = blockIdx.x * (ROW_THREADS / 32) + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (task >= tasks) return;
+  const unsigned row = task / (unsigned)parts;
+  const int c0 = (int)(task - row * (unsigned)parts) * part;
+  const float* xr = x + (long long)row * ld_x + c0;
+  const T* zr = z + (long long)row * ld_z + c0;
+  T* orow = out + (long long)row * ld_o + c0;
+  float4 xv[NV], zv[NV];
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int c = (lane + j * 32) * 4;
+    xv[j] = c < part ? load4(xr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    zv[j] = c < part ? load4(zr + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    xv[j].x *= silu_gate<T>(zv[j].x); xv[j].y *= silu_gate<T>(zv[j].y);
+    xv[j].z *= silu_gate<T>(zv[j].z); xv[j].w *= silu_gate<T>(zv[j].w);
+    ss = fmaf(xv[j].x, xv[j].x, fmaf(xv[j].y, xv[j].y, fmaf(xv[j].z, xv[j].z, fmaf(xv[j].w, xv[j].w, ss))));
+  }
+  const float scale = out_scale / sqrtf(warp_sum(ss) / (float)part + eps);
+#pragma unroll
+  for (int j = 0; j < NV; ++j) {
+    const int c = (lane + j * 32) * 4;
+    if (c >= part) continue;
+    const float4 wv = load4(w + c0 + c);
+    store4(orow + c, make_float4(xv[j].x * scale * wv.x, xv[j].y * scale * wv.y, xv[j].z * scale * wv.z, xv[j].w * scale * wv.w));
+  }
+}
+
 template <typename T>
 void launch_gate_parts_norm(const float* x, long long ld_x, const void* z, long long ld_z, const float* w, float eps, void* out,
                             long long ld_o, int n, int parts, int part, float out_scale, cudaStream_t stream) {
   const bool vec = part % 4 == 0 && ld_x % 4 == 0 && ld_z % 4 == 0 && ld_o % 4 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)w % 16 == 0 &&
                    (uintptr_t)z % (4 * sizeof(T)) == 0 && (uintptr_t)out % (4 * sizeof(T)) == 0;
   const dim3 grid((unsigned)n, (unsigned)parts), block(ROW_THREADS);
+  const long long tasks = (long long)n * parts;
+  if (vec && part <= 512 && tasks < (1ll << 31)) {
+    const dim3 blocks((unsigned)((tasks + ROW_THREADS / 32 - 1) / (ROW_THREADS / 32)));
+    if (part <= 128)
+      hfee_launch(gate_parts_norm_warp_kernel<T, 1>, blocks, block, 0, stream, x, ld_x, (const T*)z, ld_z, w, eps, (T*)out, ld_o, parts, part, out_scale, (unsigned)tasks);
+    else
+      hfee_launch(gate_parts_norm_warp_kernel<T, 4>, blocks, block, 0, stream, x, ld_x, (const T*)z, ld_z, w, eps, (T*)out, ld_o, parts, part, out_scale, (unsigned)tasks);
+    return;
+  }
   if (vec && part <= ROW_THREADS * 4)
     hfee_launch(gate_parts_norm_kernel<T, 4, 1>, grid, block, 0, stream, x, ld_x, (const T*)z, ld_z, w, eps, (T*)out, ld_o, part, out_scale);
   else if (vec)

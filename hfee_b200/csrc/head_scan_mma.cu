@@ -1,0 +1,505 @@
+// The state-space scan with one decay per head and token (see gated_recurrence.cu, "step sizes") for prompt portions, on
+// mma.sync tiles: bfloat16 x, B and C, float32 step sizes, decays and states.
+//
+//   S_t = e^(a_t) S_(t-1) + dt_t B_t x_t^T,   y_t = S_t^T C_t + D x_t,   dt_t = softplus(step_t + bias), a_t = -exp(A_log) dt_t
+//
+// A request's tokens go in runs of HS_T.  With s_t the sum of a over the run's tokens up to t, a run of n tokens is
+//
+//   y_t   = e^(s_t) S_in^T C_t + sum_(u <= t) e^(s_t - s_u) dt_u (C_t . B_u) x_u + D x_t
+//   S_out = e^(s_n) S_in + sum_u e^(s_n - s_u) dt_u B_u x_u^T
+//
+// which is the recurrence written out; every exponent is at most zero, so nothing overflows and a strong decay becomes zero.
+// Three kernels: (1) head_scan_gates: dt_t and s_t (in log2 units) of every token and head; (2) head_scan_states: per
+// (request, head, 32 columns of x) the walk over the runs with the state in the MMA accumulators; the state in front of
+// every run goes to the workspace, the state behind the last one to the request's slot; (3) head_scan_outputs: all runs at
+// once.  C . B is shared by the heads of a group, so a block of (3) takes several heads of one.
+//
+// x, B and C enter the products as they are.  What is float32 (the weighted x, the weights times C . B, the state) enters as
+// the sum of two bfloat16 numbers, the value rounded and what the rounding left, each with a product of its own; sums are
+// float32.  (2) computes S transposed, so that its accumulators, packed in pairs, are the very B fragments that (3) wants:
+// the workspace holds them in that order, one 16-byte piece (two halves, high and low) per lane.
+#include "common.cuh"
+#include "mma_tiles.cuh"
+
+namespace {
+
+constexpr int HS_T = 64;            // tokens of a run
+constexpr int HS_WARPS = 4;
+constexpr int HS_THREADS = HS_WARPS * 32;
+constexpr int HS_COLS_STATES = 32;  // columns of x per block of the walk
+constexpr int HS_COLS_OUT = 64;     // and of the outputs
+constexpr int HS_PAD = 8;
+constexpr float HS_LOG2E = 1.4426950408889634f;
+
+struct HeadScanArgs {
+  const bf16* x; const bf16* b; const bf16* c;
+  long long ld;
+  const bf16* step;
+  long long ld_step;
+  const float* dt_bias; const float* a_log; const float* d_skip;
+  float* state;                 // [slots, heads, n_state, vdim]
+  const int* cu_tokens; const int* slots;
+  float* out;
+  long long ld_o;
+  float* gate_s; float* gate_dt;          // [heads][n_tokens]
+  uint4* carried;                         // [runs][heads][tiles of 16 state entries][tiles of 8 columns][32 lanes]
+  int requests, n_tokens, heads, groups, n_state, vdim, ctiles, write_state, heads_per_block;
+};
+
+__device__ __forceinline__ int hs_runs(int count) { return (count + HS_T - 1) / HS_T; }
+
+__device__ __forceinline__ bool hs_find_run(const int* __restrict__ cu_tokens, int requests, int number, int* req, int* run) {
+  int base = 0;
+  for (int r = 0; r < requests; ++r) {
+    const int c = hs_runs(cu_tokens[r + 1] - cu_tokens[r]);
+    if (number < base + c) { *req = r; *run = number - base; return true; }
+    base += c;
+  }
+  return false;
+}
+
+__device__ __forceinline__ float hs_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void hs_copy16(void* smem, const void* gmem, bool valid) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(s), "l"(gmem), "r"(valid ? 16 : 0));
+}
+__device__ __forceinline__ void hs_copy4(void* smem, const void* gmem, bool valid) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;\n" ::"r"(s), "l"(gmem), "r"(valid ? 4 : 0));
+}
+__device__ __forceinline__ void hs_commit() { asm volatile("cp.async.commit_group;\n" ::); }
+__device__ __forceinline__ void hs_wait_all() { asm volatile("cp.async.wait_group 0;\n" ::); }
+
+// a pair of float32 numbers as two packed pairs of bfloat16: rounded, and what the rounding left
+__device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint32_t& lo) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  const __nv_bfloat162 l = __floats2bfloat162_rn(a - __bfloat162float(h.x), b - __bfloat162float(h.y));
+  hi = *reinterpret_cast<const uint32_t*>(&h);
+  lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+
+// ------------------------------------------------------------------------------------------ (1) gates
+__global__ void __launch_bounds__(256)
+head_scan_gates_kernel(HeadScanArgs p) {
+  __shared__ float dt_s[HS_T][33];
+  int req = 0, run = 0;
+  const bool mine = hs_find_run(p.cu_tokens, p.requests, blockIdx.y, &req, &run);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (!mine) return;
+  const int begin = p.cu_tokens[req] + run * HS_T, n = min(HS_T, p.cu_tokens[req + 1] - begin);
+  const int h0 = blockIdx.x * 32, lane = threadIdx.x & 31;
+  for (int e = threadIdx.x; e < HS_T * 32; e += 256) {
+    const int t = e >> 5, h = h0 + (e & 31);
+    float dt = 0.f;
+    if (t < n && h < p.heads) {
+      const float z = __bfloat162float(p.step[(long long)(begin + t) * p.ld_step + h]) + p.dt_bias[h];
+      dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
+    }
+    dt_s[t][e & 31] = dt;
+  }
+  __syncthreads();
+  for (int j = threadIdx.x >> 5; j < 32; j += 8) {
+    const int h = h0 + j;
+    if (h >= p.heads) break;                             // the same for the whole warp
+    const float rate = -expf(p.a_log[h]) * HS_LOG2E;
+    const float d0 = dt_s[2 * lane][j], d1 = dt_s[2 * lane + 1][j];
+    const float a0 = rate * d0, a1 = rate * d1;
+    float sum = a0 + a1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float before = __shfl_up_sync(0xffffffffu, sum, o);
+      if (lane >= o) sum += before;
+    }
+    float front = __shfl_up_sync(0xffffffffu, sum, 1);
+    if (lane == 0) front = 0.f;
+    const long long at = (long long)h * p.n_tokens + begin + 2 * lane;
+    if (2 * lane < n) { p.gate_s[at] = front + a0; p.gate_dt[at] = d0; }
+    if (2 * lane + 1 < n) { p.gate_s[at + 1] = front + a0 + a1; p.gate_dt[at + 1] = d1; }
+  }
+}
+
+// ------------------------------------------------------------------------------------------ (2) states
+template <int NP> struct StatesCfg {
+  static constexpr int TILES = NP / 16;                    // tiles of 16 state entries
+  static constexpr int MINE = TILES >= HS_WARPS ? TILES / HS_WARPS : 1;   // per warp
+  static constexpr int LDB = NP + HS_PAD, LDX = HS_COLS_STATES + HS_PAD;
+  static constexpr int STAGE = HS_T * (LDB + LDX) * 2 + 2 * HS_T * 4;     // bytes: B, x, s, dt of one run
+  static constexpr int SMEM = 2 * STAGE + 2 * HS_T * LDX * 2;             // + the weighted x, high and low
+};
+
+template <int NP>
+__global__ void __launch_bounds__(HS_THREADS)
+head_scan_states_kernel(HeadScanArgs p) {
+  using C = StatesCfg<NP>;
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int head = blockIdx.x, req = blockIdx.y, c0 = blockIdx.z * HS_COLS_STATES;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int begin = p.cu_tokens[req], count = p.cu_tokens[req + 1] - begin;
+  const int slot = p.slots[req];
+  int first_run = 0;
+  for (int r = 0; r < req; ++r) first_run += hs_runs(p.cu_tokens[r + 1] - p.cu_tokens[r]);
+  const int group = head / (p.heads / p.groups);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (count <= 0) return;
+  bf16* wx_hi = reinterpret_cast<bf16*>(smem_raw + 2 * C::STAGE);        // [HS_T][LDX]
+  bf16* wx_lo = wx_hi + HS_T * C::LDX;
+  auto b_of = [&](int st) { return reinterpret_cast<bf16*>(smem_raw + st * C::STAGE); };
+  auto x_of = [&](int st) { return b_of(st) + HS_T * C::LDB; };
+  auto s_of = [&](int st) { return reinterpret_cast<float*>(x_of(st) + HS_T * C::LDX); };
+  auto load = [&](int run, int st) {
+    const int row0 = begin + run * HS_T, n = min(HS_T, count - run * HS_T);
+    bf16* bd = b_of(st);
+    bf16* xd = x_of(st);
+    float* sd = s_of(st);
+#pragma unroll
+    for (int e = tid; e < HS_T * (NP / 8); e += HS_THREADS) {
+      const int s = e / (NP / 8), k = (e % (NP / 8)) * 8;
+      const bool ok = s < n && k < p.n_state;
+      hs_copy16(bd + s * C::LDB + k, ok ? p.b + (long long)(row0 + s) * p.ld + group * p.n_state + k : p.b, ok);
+    }
+#pragma unroll
+    for (int e = tid; e < HS_T * (HS_COLS_STATES / 8); e += HS_THREADS) {
+      const int s = e / (HS_COLS_STATES / 8), c = (e % (HS_COLS_STATES / 8)) * 8;
+      const bool ok = s < n && c0 + c < p.vdim;
+      hs_copy16(xd + s * C::LDX + c, ok ? p.x + (long long)(row0 + s) * p.ld + (long long)head * p.vdim + c0 + c : p.x, ok);
+    }
+    const int s = tid % HS_T;
+    const float* src = (tid < HS_T ? p.gate_s : p.gate_dt) + (long long)head * p.n_tokens + row0;
+    hs_copy4(sd + tid, s < n ? src + s : p.gate_s, s < n);                // s first, dt behind it
+    hs_commit();
+  };
+  load(0, 0);
+
+  float acc[2][2 * C::MINE][4];                            // [16 columns][8 state entries]: S transposed
+  float* S_g = p.state + ((long long)slot * p.heads + head) * p.n_state * p.vdim;
+  const bool active = warp < C::TILES;
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int j = 0; j < 2 * C::MINE; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int c = c0 + m * 16 + g + (i >= 2 ? 8 : 0), k = warp * C::MINE * 16 + j * 8 + 2 * t + (i & 1);
+        acc[m][j][i] = active && c < p.vdim && k < p.n_state ? S_g[(long long)k * p.vdim + c] : 0.f;
+      }
+  const int runs = hs_runs(count);
+  for (int run = 0; run < runs; ++run) {
+    const int st = run & 1, n = min(HS_T, count - run * HS_T);
+    hs_wait_all();
+    __syncthreads();                                       // the run's rows are here, the run before is used up
+    if (run + 1 < runs) load(run + 1, st ^ 1);
+    // the state in front of the run, as B fragments
+    if (active) {
+      uint4* dst = p.carried + ((long long)(first_run + run) * p.heads + head) * (C::TILES * p.ctiles * 32) + lane;
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int ct = c0 / 8 + m * 2 + half;
+          if (ct >= p.ctiles) continue;
+#pragma unroll
+          for (int j = 0; j < C::MINE; ++j) {
+            uint4 f;
+            split_pair(acc[m][2 * j][2 * half], acc[m][2 * j][2 * half + 1], f.x, f.z);
+            split_pair(acc[m][2 * j + 1][2 * half], acc[m][2 * j + 1][2 * half + 1], f.y, f.w);
+            dst[((warp * C::MINE + j) * p.ctiles + ct) * 32] = f;
+          }
+        }
+    }
+    const float* ss = s_of(st);
+    const float* sdt = ss + HS_T;
+    const float s_last = ss[n - 1];
+    const bf16* xs = x_of(st);
+#pragma unroll
+    for (int e = tid; e < HS_T * (HS_COLS_STATES / 8); e += HS_THREADS) {
+      const int s = e / (HS_COLS_STATES / 8), c = (e % (HS_COLS_STATES / 8)) * 8;
+      const float w = s < n ? hs_exp2(s_last - ss[s]) * sdt[s] : 0.f;
+      const uint4 raw = *reinterpret_cast<const uint4*>(xs + s * C::LDX + c);
+      const uint32_t in[4] = {raw.x, raw.y, raw.z, raw.w};
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        split_pair(__uint_as_float(in[i] << 16) * w, __uint_as_float(in[i] & 0xffff0000u) * w, hi[i], lo[i]);
+      *reinterpret_cast<uint4*>(wx_hi + s * C::LDX + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(wx_lo + s * C::LDX + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    }
+    __syncthreads();
+    const float decay = hs_exp2(s_last);
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int j = 0; j < 2 * C::MINE; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[m][j][i] *= decay;
+    if (active) {
+      const bf16* bs = b_of(st);
+#pragma unroll
+      for (int ks = 0; ks < HS_T / 16; ++ks) {
+        uint32_t ah[2][4], al[2][4];
+#pragma unroll
+        for (int m = 0; m < 2; ++m) {
+          load_a_trans(ah[m], wx_hi, C::LDX, m * 16, ks * 16, lane);
+          load_a_trans(al[m], wx_lo, C::LDX, m * 16, ks * 16, lane);
+        }
+#pragma unroll
+        for (int j = 0; j < C::MINE; ++j) {
+          uint32_t b[4];
+          load_b_pair_trans(b, bs, C::LDB, (warp * C::MINE + j) * 16, ks * 16, lane);
+#pragma unroll
+          for (int m = 0; m < 2; ++m) {
+            mma_bf16(acc[m][2 * j], ah[m], b[0], b[1]);
+            mma_bf16(acc[m][2 * j + 1], ah[m], b[2], b[3]);
+            mma_bf16(acc[m][2 * j], al[m], b[0], b[1]);
+            mma_bf16(acc[m][2 * j + 1], al[m], b[2], b[3]);
+          }
+        }
+      }
+    }
+  }
+  if (!p.write_state) return;
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int j = 0; j < 2 * C::MINE; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int c = c0 + m * 16 + g + (i >= 2 ? 8 : 0), k = warp * C::MINE * 16 + j * 8 + 2 * t + (i & 1);
+        if (active && c < p.vdim && k < p.n_state) S_g[(long long)k * p.vdim + c] = acc[m][j][i];
+      }
+}
+
+// ------------------------------------------------------------------------------------------ (3) outputs
+template <int NP> struct OutCfg {
+  static constexpr int TILES = NP / 16;
+  static constexpr int LDB = NP + HS_PAD, LDX = HS_COLS_OUT + HS_PAD;
+  static constexpr int X_STAGE = HS_T * LDX * 2 + 2 * HS_T * 4;           // bytes: x, s, dt of one head
+  static constexpr int SMEM = 2 * HS_T * LDB * 2 + 2 * X_STAGE;
+};
+
+template <int NP>
+__global__ void __launch_bounds__(HS_THREADS, NP <= 128 ? 3 : 2)
+head_scan_outputs_kernel(HeadScanArgs p) {
+  using C = OutCfg<NP>;
+  extern __shared__ __align__(16) unsigned char smem_raw[];
+  const int head0 = blockIdx.y * p.heads_per_block, c0 = blockIdx.z * HS_COLS_OUT;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  int req = 0, run = 0;
+  const bool mine = hs_find_run(p.cu_tokens, p.requests, blockIdx.x, &req, &run);
+  pdl_wait();
+  pdl_launch_dependents();
+  if (!mine) return;
+  const int begin = p.cu_tokens[req] + run * HS_T, n = min(HS_T, p.cu_tokens[req + 1] - begin);
+  const int group = head0 / (p.heads / p.groups);
+  bf16* cs = reinterpret_cast<bf16*>(smem_raw);            // [HS_T][LDB]
+  bf16* bs = cs + HS_T * C::LDB;                           // [HS_T][LDB]
+  unsigned char* stages = smem_raw + 2 * HS_T * C::LDB * 2;
+  auto x_of = [&](int st) { return reinterpret_cast<bf16*>(stages + st * C::X_STAGE); };
+  auto s_of = [&](int st) { return reinterpret_cast<float*>(x_of(st) + HS_T * C::LDX); };
+  auto load_head = [&](int head, int st) {
+    bf16* xd = x_of(st);
+    float* sd = s_of(st);
+#pragma unroll
+    for (int e = tid; e < HS_T * (HS_COLS_OUT / 8); e += HS_THREADS) {
+      const int s = e / (HS_COLS_OUT / 8), c = (e % (HS_COLS_OUT / 8)) * 8;
+      const bool ok = s < n && c0 + c < p.vdim;
+      hs_copy16(xd + s * C::LDX + c, ok ? p.x + (long long)(begin + s) * p.ld + (long long)head * p.vdim + c0 + c : p.x, ok);
+    }
+    const int s = tid % HS_T;
+    const float* src = (tid < HS_T ? p.gate_s : p.gate_dt) + (long long)head * p.n_tokens + begin;
+    hs_copy4(sd + tid, s < n ? src + s : p.gate_s, s < n);
+    hs_commit();
+  };
+#pragma unroll
+  for (int e = tid; e < HS_T * (NP / 8); e += HS_THREADS) {
+    const int s = e / (NP / 8), k = (e % (NP / 8)) * 8;
+    const bool ok = s < n && k < p.n_state;
+    const long long at = (long long)(begin + s) * p.ld + group * p.n_state + k;
+    hs_copy16(cs + s * C::LDB + k, ok ? p.c + at : p.c, ok);
+    hs_copy16(bs + s * C::LDB + k, ok ? p.b + at : p.b, ok);
+  }
+  load_head(head0, 0);
+  hs_wait_all();
+  __syncthreads();
+
+  const int r0 = warp * 16;
+  // C . B of the warp's 16 tokens with the tokens up to the diagonal, for all heads of the block
+  float cb[HS_T / 8][4];
+#pragma unroll
+  for (int j = 0; j < HS_T / 8; ++j) cb[j][0] = cb[j][1] = cb[j][2] = cb[j][3] = 0.f;
+#pragma unroll
+  for (int kk = 0; kk < C::TILES; ++kk) {
+    uint32_t a[4];
+    load_a(a, cs, C::LDB, r0, kk * 16, lane);
+#pragma unroll
+    for (int kt = 0; kt < HS_T / 16; ++kt) {
+      if (kt <= warp) {
+        uint32_t b[4];
+        load_b_pair(b, bs, C::LDB, kt * 16, kk * 16, lane);
+        mma_bf16(cb[2 * kt], a, b[0], b[1]);
+        mma_bf16(cb[2 * kt + 1], a, b[2], b[3]);
+      }
+    }
+  }
+  const int ct0 = c0 / 8, cts = min(HS_COLS_OUT / 8, p.ctiles - ct0);
+  for (int hh = 0; hh < p.heads_per_block; ++hh) {
+    const int head = head0 + hh, st = hh & 1;
+    if (hh + 1 < p.heads_per_block) load_head(head + 1, st ^ 1);
+    float acc[HS_COLS_OUT / 8][4];
+#pragma unroll
+    for (int j = 0; j < HS_COLS_OUT / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+    if (r0 < n) {
+      const float* ss = s_of(st);
+      const float* sdt = ss + HS_T;
+      const bf16* xs = x_of(st);
+      // what the state in front of the run gives
+      const uint4* S = p.carried + ((long long)(blockIdx.x) * p.heads + head) * (C::TILES * p.ctiles * 32) + ct0 * 32 + lane;
+      uint4 f[2][HS_COLS_OUT / 8];
+#pragma unroll
+      for (int j = 0; j < HS_COLS_OUT / 8; ++j)
+        if (j < cts) f[0][j] = S[j * 32];
+#pragma unroll
+      for (int kk = 0; kk < C::TILES; ++kk) {
+        if (kk + 1 < C::TILES) {
+#pragma unroll
+          for (int j = 0; j < HS_COLS_OUT / 8; ++j)
+            if (j < cts) f[(kk + 1) & 1][j] = S[((kk + 1) * p.ctiles + j) * 32];
+        }
+        uint32_t a[4];
+        load_a(a, cs, C::LDB, r0, kk * 16, lane);
+#pragma unroll
+        for (int j = 0; j < HS_COLS_OUT / 8; ++j)
+          if (j < cts) {
+            mma_bf16(acc[j], a, f[kk & 1][j].x, f[kk & 1][j].y);
+            mma_bf16(acc[j], a, f[kk & 1][j].z, f[kk & 1][j].w);
+          }
+      }
+      const float s_lo = ss[r0 + g], s_hi = ss[r0 + g + 8];
+      const float e_lo = hs_exp2(s_lo), e_hi = hs_exp2(s_hi);
+#pragma unroll
+      for (int j = 0; j < HS_COLS_OUT / 8; ++j) { acc[j][0] *= e_lo; acc[j][1] *= e_lo; acc[j][2] *= e_hi; acc[j][3] *= e_hi; }
+      // what the run's own tokens give: weights e^(s_t - s_u) dt_u (C_t . B_u), straight from the accumulators
+#pragma unroll
+      for (int kt = 0; kt < HS_T / 16; ++kt) {
+        if (kt <= warp) {
+          uint32_t ah[4], al[4];
+#pragma unroll
+          for (int q = 0; q < 2; ++q) {
+            const int u = kt * 16 + q * 8 + 2 * t;
+            const float su0 = ss[u], su1 = ss[u + 1], du0 = sdt[u], du1 = sdt[u + 1];
+            const int lo_row = r0 + g, hi_row = r0 + g + 8;
+            const float* v = cb[2 * kt + q];
+            const float w0 = u <= lo_row ? v[0] * (hs_exp2(s_lo - su0) * du0) : 0.f;
+            const float w1 = u + 1 <= lo_row ? v[1] * (hs_exp2(s_lo - su1) * du1) : 0.f;
+            const float w2 = u <= hi_row ? v[2] * (hs_exp2(s_hi - su0) * du0) : 0.f;
+            const float w3 = u + 1 <= hi_row ? v[3] * (hs_exp2(s_hi - su1) * du1) : 0.f;
+            split_pair(w0, w1, ah[2 * q], al[2 * q]);
+            split_pair(w2, w3, ah[2 * q + 1], al[2 * q + 1]);
+          }
+#pragma unroll
+          for (int j = 0; j < HS_COLS_OUT / 8; j += 2)
+            if (j < cts) {
+              uint32_t b[4];
+              load_b_pair_trans(b, xs, C::LDX, j * 8, kt * 16, lane);
+              mma_bf16(acc[j], ah, b[0], b[1]);
+              mma_bf16(acc[j + 1], ah, b[2], b[3]);
+              mma_bf16(acc[j], al, b[0], b[1]);
+              mma_bf16(acc[j + 1], al, b[2], b[3]);
+            }
+        }
+      }
+      const float skip = p.d_skip[head];
+#pragma unroll
+      for (int j = 0; j < HS_COLS_OUT / 8; ++j) {
+        const int c = c0 + j * 8 + 2 * t;
+        if (c >= p.vdim) continue;
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int row = r0 + g + 8 * half;
+          if (row >= n) continue;
+          const __nv_bfloat162 xv = *reinterpret_cast<const __nv_bfloat162*>(xs + row * C::LDX + j * 8 + 2 * t);
+          *reinterpret_cast<float2*>(p.out + (long long)(begin + row) * p.ld_o + (long long)head * p.vdim + c) =
+              make_float2(fmaf(skip, __bfloat162float(xv.x), acc[j][2 * half]), fmaf(skip, __bfloat162float(xv.y), acc[j][2 * half + 1]));
+        }
+      }
+    }
+    hs_wait_all();
+    __syncthreads();
+  }
+}
+
+int padded_state(int n_state) { return n_state <= 32 ? 32 : n_state <= 64 ? 64 : n_state <= 128 ? 128 : 256; }
+
+template <int NP>
+int launch_head_scan(HeadScanArgs p, int max_runs, cudaStream_t stream) {
+  static bool configured = false;
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(head_scan_states_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, StatesCfg<NP>::SMEM);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(head_scan_outputs_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, OutCfg<NP>::SMEM);
+    if (e != cudaSuccess) return hfee_fail(HFEE_ERR_CUDA, "head_scan_mma: cannot get its shared memory: %s", cudaGetErrorString(e));
+    configured = true;
+  }
+  hfee_launch(head_scan_gates_kernel, dim3((p.heads + 31) / 32, max_runs), dim3(256), 0, stream, p);
+  int rc = hfee_check_launch("head_scan_gates");
+  if (rc != HFEE_OK) return rc;
+  hfee_launch(head_scan_states_kernel<NP>, dim3(p.heads, p.requests, (p.vdim + HS_COLS_STATES - 1) / HS_COLS_STATES), dim3(HS_THREADS),
+              StatesCfg<NP>::SMEM, stream, p);
+  rc = hfee_check_launch("head_scan_states");
+  if (rc != HFEE_OK) return rc;
+  const int tiles = (p.vdim + HS_COLS_OUT - 1) / HS_COLS_OUT;
+  // several heads of a group per block share its C . B, as long as the blocks still fill the GPU
+  p.heads_per_block = 1;
+  for (int h : {4, 2})
+    if ((p.heads / p.groups) % h == 0 && (long long)max_runs * (p.heads / h) * tiles >= 2 * hfee_sm_count()) { p.heads_per_block = h; break; }
+  hfee_launch(head_scan_outputs_kernel<NP>, dim3(max_runs, p.heads / p.heads_per_block, tiles), dim3(HS_THREADS), OutCfg<NP>::SMEM, stream, p);
+  return hfee_check_launch("head_scan_outputs");
+}
+
+}  // namespace
+
+// 1 if hfee_head_scan_mma takes these sizes (bfloat16 is implied).
+HFEE_API int hfee_head_scan_mma_supports(int state_dim, int vdim) {
+  return state_dim > 0 && state_dim <= 256 && state_dim % 8 == 0 && vdim > 0 && vdim % 8 == 0 ? 1 : 0;
+}
+
+// Floats of workspace for steps of at most n_tokens tokens of at most `requests` requests.
+HFEE_API long long hfee_head_scan_mma_workspace(int requests, int n_tokens, int heads, int state_dim, int vdim) {
+  const long long runs = n_tokens / HS_T + requests;
+  return runs * heads * (padded_state(state_dim) / 16) * ((vdim + 7) / 8) * 128 + 2ll * heads * n_tokens;
+}
+
+// Arguments as hfee_head_scan (all activations bfloat16); the workspace must start on 16 bytes.
+HFEE_API int hfee_head_scan_mma(const void* x, const void* bmat, const void* cmat, long long ld, const void* step, long long ld_step,
+                                const float* dt_bias, const float* a_log, const float* d_skip, float* state, const int* cu_tokens,
+                                const int* slots, float* out, long long ld_o, int requests, int n_tokens, int heads, int groups,
+                                int state_dim, int vdim, int write_state, float* workspace, long long workspace_floats,
+                                cudaStream_t stream) {
+  if (requests == 0 || n_tokens == 0) return HFEE_OK;
+  HFEE_REQUIRE(hfee_head_scan_mma_supports(state_dim, vdim), "head_scan_mma: state size %d and vdim %d must be multiples of 8, the former at most 256",
+               state_dim, vdim);
+  HFEE_REQUIRE(heads > 0 && groups > 0 && heads % groups == 0, "head_scan_mma: heads %d must be a multiple of groups %d", heads, groups);
+  HFEE_REQUIRE(ld % 8 == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)bmat % 16 == 0 && (uintptr_t)cmat % 16 == 0 && ld_o % 2 == 0 &&
+               (uintptr_t)out % 8 == 0, "head_scan_mma: rows must start on 16 bytes (the output's on 8)");
+  HFEE_REQUIRE(ld_o >= (long long)heads * vdim && ld_step >= heads, "head_scan_mma: a row stride is too small");
+  HFEE_REQUIRE(workspace != nullptr && (uintptr_t)workspace % 16 == 0 &&
+               workspace_floats >= hfee_head_scan_mma_workspace(requests, n_tokens, heads, state_dim, vdim), "head_scan_mma: the workspace is too small");
+  const int max_runs = n_tokens / HS_T + requests;
+  HFEE_REQUIRE(max_runs <= 65535 && requests <= 65535 && heads <= 65535, "head_scan_mma: too many runs or heads for one grid");
+  const int np = padded_state(state_dim), ctiles = (vdim + 7) / 8;
+  HeadScanArgs p{(const bf16*)x, (const bf16*)bmat, (const bf16*)cmat, ld, (const bf16*)step, ld_step, dt_bias, a_log, d_skip, state,
+                 cu_tokens, slots, out, ld_o, nullptr, nullptr, (uint4*)workspace, requests, n_tokens, heads, groups, state_dim, vdim, ctiles,
+                 write_state, 1};
+  p.gate_s = workspace + (long long)max_runs * heads * (np / 16) * ctiles * 128;
+  p.gate_dt = p.gate_s + (long long)heads * n_tokens;
+  switch (np) {
+    case 32: return launch_head_scan<32>(p, max_runs, stream);
+    case 64: return launch_head_scan<64>(p, max_runs, stream);
+    case 128: return launch_head_scan<128>(p, max_runs, stream);
+    default: return launch_head_scan<256>(p, max_runs, stream);
+  }
+}

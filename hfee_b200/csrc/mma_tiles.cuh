@@ -35,6 +35,21 @@ __device__ __forceinline__ void load_b(uint32_t& b0, uint32_t& b1, const bf16* B
   b0 = *reinterpret_cast<const uint32_t*>(p);
   b1 = *reinterpret_cast<const uint32_t*>(p + 8);
 }
+__device__ __forceinline__ void ldmatrix_x4_trans(uint32_t (&r)[4], const bf16* row) {
+  const uint32_t addr = (uint32_t)__cvta_generic_to_shared(row);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+// the A operand of load_a and the B operands of load_b_pair from matrices that are stored the other way round, the summed
+// index outermost: At[k][m], B[k][n]
+__device__ __forceinline__ void load_a_trans(uint32_t (&a)[4], const bf16* At, int ld, int m0, int k0, int lane) {
+  const int piece = lane >> 3, r = lane & 7;
+  ldmatrix_x4_trans(a, At + (k0 + r + (piece >> 1) * 8) * ld + m0 + (piece & 1) * 8);
+}
+__device__ __forceinline__ void load_b_pair_trans(uint32_t (&b)[4], const bf16* B, int ld, int n0, int k0, int lane) {
+  const int piece = lane >> 3, r = lane & 7;
+  ldmatrix_x4_trans(b, B + (k0 + r + (piece & 1) * 8) * ld + n0 + (piece >> 1) * 8);
+}
 __device__ __forceinline__ void split_bf16(float x, bf16* hi, bf16* lo) {
   *hi = __float2bfloat16_rn(x);
   *lo = __float2bfloat16_rn(x - __bfloat162float(*hi));

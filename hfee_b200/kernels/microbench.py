@@ -22,6 +22,9 @@ where that matters, and prints what it achieved against the roofline that bounds
     python -m hfee_b200.kernels.microbench selective_scan    --tokens 2048 --channels 2048 --state 16 [--decode --batch 8]
     python -m hfee_b200.kernels.microbench distance_attention --tokens 2048 --heads 32 --kv-heads 8 --head-dim 64 [--value-dim 128] [--decode --batch 8]
     python -m hfee_b200.kernels.microbench moe_experts       --tokens 2048 --k 2048 --inner 2048 --experts 16 --top 2
+    python -m hfee_b200.kernels.microbench softmax_attention --tokens 2048 --window 1024 [--keep-first 4 --softcap 30] [--decode --batch 8]
+    python -m hfee_b200.kernels.microbench head_scan         --tokens 2048 --heads 64 --kv-heads 1 --head-dim 64 --state 128 [--decode --batch 8]
+    python -m hfee_b200.kernels.microbench bumisun_rows      --tokens 2048 --k 2048 --inner 4096
     python -m hfee_b200.kernels.microbench row_ops           --tokens 2048 --k 2048 --inner 4096 --depth 6
 
 ``--iters`` timed launches follow ``--warmup`` untimed ones; ``--rotate`` distinct weight
@@ -408,7 +411,7 @@ def _row_ops(args) -> dict:
 
 
 def _softmax_attention(args) -> dict:
-    """Windowed softmax attention with a sink (``--window``, 0: none): one prompt portion, or a decode step of ``--batch``."""
+    """Windowed softmax attention with a sink (``--window``, 0: none; ``--keep-first``, ``--softcap``): one prompt portion, or a decode step of ``--batch``."""
     heads, kv, hd, vd, page = args.heads, args.kv_heads, args.head_dim, args.value_dim or args.head_dim, args.page_size
     before, new = ([args.context] * args.batch, [1] * args.batch) if args.decode else ([args.context_before], [args.tokens])
     b = _batch_of(before, new)
@@ -422,14 +425,15 @@ def _softmax_attention(args) -> dict:
     sink = torch.linspace(-1.0, 2.0, heads, device=DEV)
     tile = ops.distance_attention_tile(hd, vd)
     scratch = torch.empty(b.r * heads * ops.MAX_SPLITS * (tile + 2), dtype=torch.float32, device=DEV) if args.decode and tile else None
-    fn = lambda i: ops.softmax_attention(q, kp, vp, table, page, b, out, heads, kv, hd, vd, hd ** -0.5, args.window, sink, 1.0, scratch)
+    fn = lambda i: ops.softmax_attention(q, kp, vp, table, page, b, out, heads, kv, hd, vd, hd ** -0.5, args.window, sink, 1.0, scratch,
+                                         args.keep_first, args.softcap or None)
     sec = _time(fn, args.warmup, args.iters)
     w = args.window or (1 << 30)
     seen = lambda s, c: sum(min(w, s + j + 1) for j in range(c))          # keys each new token reads
     kv_bytes = sum(min(s + c, w + c) for s, c in zip(before, new)) * kv * (hd + vd) * 2
     flops = sum(2.0 * heads * (hd + vd) * seen(s, c) for s, c in zip(before, new))
     return {"kernel": "softmax_attention", "heads": heads, "kv_heads": kv, "head_dim": hd, "value_dim": vd, "requests": b.r,
-            "context": b.max_context, "window": args.window, "us": round(sec * 1e6, 2), "kv_gbs": round(kv_bytes / sec / 1e9, 1),
+            "context": b.max_context, "window": args.window, "keep_first": args.keep_first, "softcap": args.softcap, "us": round(sec * 1e6, 2), "kv_gbs": round(kv_bytes / sec / 1e9, 1),
             "tflops": round(flops / sec / 1e12, 1)}
 
 
@@ -462,6 +466,51 @@ def _gated_recurrence(args, mode: int) -> dict:
     return {"kernel": "gla" if mode == 0 else "matrix_memory", "heads": heads, "key_dim": d, "value_dim": vd, "tokens": b.n,
             "requests": b.r, "chunked": chunked, "us": round(sec * 1e6, 2), "fp32_tflops": round(flops / sec / 1e12, 2),
             "io_gbs": round(io / sec / 1e9, 1)}
+
+
+def _head_scan(args) -> dict:
+    """The state-space scan with one decay per head and token: ``--heads`` heads of ``--head-dim`` columns, ``--state`` entries,
+    ``--kv-heads`` groups: one prompt portion of ``--tokens`` tokens, or a decode step of ``--batch`` requests."""
+    heads, groups, vd, ns = args.heads, args.kv_heads, args.head_dim, args.state
+    before, new = ([args.context] * args.batch, [1] * args.batch) if args.decode else ([0] * args.requests, [args.tokens // args.requests] * args.requests)
+    b = _batch_of(before, new)
+    inner, bc = heads * vd, groups * ns
+    xbc = (torch.randn(b.n, inner + 2 * bc, device=DEV) * 0.5).to(torch.bfloat16)
+    dt = torch.randn(b.n, heads, device=DEV).to(torch.bfloat16)
+    bias, a_log, d = torch.full((heads,), -2.0, device=DEV), torch.linspace(-3.0, 1.0, heads, device=DEV), torch.ones(heads, device=DEV)
+    S = torch.zeros(b.r, heads, ns, vd, device=DEV)
+    out = torch.empty(b.n, inner, device=DEV)
+    ws = torch.empty(ops.head_scan_workspace(b.r, b.n, heads, ns, vd), device=DEV)
+    fn = lambda i: ops.head_scan(xbc[:, :inner], xbc[:, inner:inner + bc], xbc[:, inner + bc:], dt, bias, a_log, d, S, b, out, heads, groups, ns, vd,
+                                 True, ws)
+    sec = _time(fn, args.warmup, args.iters)
+    io = b.n * ((inner + 2 * bc + heads) * 2 + inner * 4) + 2 * S.numel() * 4
+    flops = 4.0 * b.n * heads * ns * vd
+    return {"kernel": "head_scan", "heads": heads, "groups": groups, "vdim": vd, "state": ns, "tokens": b.n, "requests": b.r,
+            "us": round(sec * 1e6, 2), "io_gbs": round(io / sec / 1e9, 1), "io_mb": round(io / 1e6, 1), "tflops": round(flops / sec / 1e12, 2)}
+
+
+def _bumisun_rows(args) -> dict:
+    """The normed embedding (``--k`` columns), the gate in front of a norm in parts (``--inner`` columns) and the router."""
+    n, k, inner = args.tokens, args.k, args.inner
+    table = torch.randn(32768, k, device=DEV).to(torch.bfloat16)
+    tok = torch.randint(0, 32768, (n,), dtype=torch.int32, device=DEV)
+    x, w, wi = torch.empty(n, k, device=DEV), torch.ones(k, device=DEV), torch.ones(inner, device=DEV)
+    y, z = torch.randn(n, inner, device=DEV), torch.randn(n, inner, device=DEV).to(torch.bfloat16)
+    o = torch.empty(n, inner, dtype=torch.bfloat16, device=DEV)
+    logits, bias = torch.randn(n, args.experts + 1, device=DEV), torch.randn(args.experts, device=DEV)
+    choice, weight = torch.empty(n, args.top, dtype=torch.int32, device=DEV), torch.empty(n, args.top, device=DEV)
+    cases = {
+        "embed_norm": (lambda i: ops.embed_norm(table, tok, w, 1e-5, x), n * k * 6),
+        "gate_parts_norm": (lambda i: ops.gate_parts_norm(y, z, wi, 1e-5, 1, o), n * inner * 8),
+        "gate_parts_norm_8": (lambda i: ops.gate_parts_norm(y, z, wi, 1e-5, 8, o), n * inner * 8),
+        "moe_route_chosen": (lambda i: ops.moe_route_chosen(logits, args.experts, args.top, 1.0, choice, weight, bias), n * args.experts * 4),
+    }
+    res = {"kernel": "bumisun_rows", "tokens": n, "width": k, "inner": inner}
+    for name, (fn, nbytes) in cases.items():
+        sec = _time(fn, args.warmup, args.iters)
+        res[name] = {"us": round(sec * 1e6, 2), "gbs": round(nbytes / sec / 1e9, 1)}
+    return res
 
 
 def _channel_delta(args) -> dict:
@@ -568,7 +617,7 @@ def main(argv=None) -> int:
                                        "gemm_tcgen05", "gemm_stream", "gemm_skinny", "gemm_ring", "gemm_pair", "attention_decode", "attention_prefill",
                                       "sigmoid_attention", "linear_attention", "mingru", "selective_scan",
                                        "distance_attention", "moe_experts", "row_ops", "softmax_attention", "gla", "matrix_memory",
-                                       "pupinex_rows", "channel_delta", "stream_step", "latent_prepare"])
+                                       "pupinex_rows", "channel_delta", "stream_step", "latent_prepare", "head_scan", "bumisun_rows"])
     ap.add_argument("--m", type=int, default=2048)
     ap.add_argument("--n", type=int, default=16384)
     ap.add_argument("--k", type=int, default=2048)
@@ -591,6 +640,8 @@ def main(argv=None) -> int:
     ap.add_argument("--channels", type=int, default=2048, help="mingru / selective_scan: channels of the recurrence")
     ap.add_argument("--state", type=int, default=16, help="selective_scan: state entries per channel")
     ap.add_argument("--value-dim", type=int, default=0, help="distance_attention: value size per head (0: the key size)")
+    ap.add_argument("--keep-first", type=int, default=0, help="softmax_attention: first positions that stay visible behind the window")
+    ap.add_argument("--softcap", type=float, default=0.0, help="softmax_attention: cap on the scores (0: none)")
     ap.add_argument("--streams", type=int, default=4, help="stream_step: residual streams")
     ap.add_argument("--requests", type=int, default=1, help="channel_delta: equal portions that --tokens is divided into")
     ap.add_argument("--experts", type=int, default=16)
@@ -626,6 +677,8 @@ def main(argv=None) -> int:
         res = _gated_recurrence(args, 0 if args.kernel == "gla" else 1)
     elif args.kernel in ("channel_delta", "stream_step", "latent_prepare"):
         res = {"channel_delta": _channel_delta, "stream_step": _stream_step, "latent_prepare": _latent_prepare}[args.kernel](args)
+    elif args.kernel in ("head_scan", "bumisun_rows"):
+        res = {"head_scan": _head_scan, "bumisun_rows": _bumisun_rows}[args.kernel](args)
     elif args.kernel == "pupinex_rows":
         res = _pupinex_rows(args)
     else:

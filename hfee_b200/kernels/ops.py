@@ -103,6 +103,8 @@ _SIGNATURES = {
     "hfee_add_bias": [_P, _L, _P, _I, _I, _P],
     "hfee_embed_norm": [_P, _I, _P, _P, _P, _P, _F, _P, _I, _I, _I, _P],
     "hfee_gate_parts_norm": [_P, _L, _P, _L, _P, _F, _P, _L, _I, _I, _I, _F, _I, _P],
+    "hfee_head_scan_mma": [_P, _P, _P, _L, _P, _L, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _L, _P],
+    "hfee_head_scan_mma_supports": [_I, _I],
     "hfee_head_scan": [_P, _P, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _P, _L, _I, _I, _I, _I, _I, _I, _I, _P, _L, _P],
     "hfee_attention_prepare": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _P, _P, _P, _F, _P, _I, _I, _P, _P, _P, _L, _P, _P, _P, _I, _I,
                                _I, _I, _I, _I, _P, _L, _I, _F, _P],
@@ -155,6 +157,8 @@ def library() -> ctypes.CDLL:
     lib.hfee_channel_delta_workspace.argtypes = [_I, _I, _I, _I, _I]
     lib.hfee_gated_recurrence_workspace.restype = _L
     lib.hfee_gated_recurrence_workspace.argtypes = [_I, _I, _I, _I, _I]
+    lib.hfee_head_scan_mma_workspace.restype = _L
+    lib.hfee_head_scan_mma_workspace.argtypes = [_I, _I, _I, _I, _I]
     lib.hfee_moe_tile_rows.restype = _I
     lib.hfee_moe_tile_rows.argtypes = []
     for name, sig in _SIGNATURES.items():
@@ -2049,6 +2053,16 @@ def gated_recurrence(mode: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tenso
 
 
 HEAD_SCAN_RUNS_MIN = 65            # from this many new tokens of one request on, runs of 64 tokens work side by side
+HEAD_SCAN_MMA_MIN = 24             # from here on the tensor-core kernels beat the walk token by token
+USE_HEAD_SCAN_MMA = True
+_HEAD_SCAN_MMA_TAKES: dict = {}
+
+
+def head_scan_mma_supports(state_dim: int, vdim: int) -> bool:
+    key = (state_dim, vdim)
+    if key not in _HEAD_SCAN_MMA_TAKES:
+        _HEAD_SCAN_MMA_TAKES[key] = bool(library().hfee_head_scan_mma_supports(*key))
+    return _HEAD_SCAN_MMA_TAKES[key]
 
 
 def head_scan(x: torch.Tensor, bmat: torch.Tensor, cmat: torch.Tensor, step_size: torch.Tensor, dt_bias: torch.Tensor,
@@ -2058,8 +2072,9 @@ def head_scan(x: torch.Tensor, bmat: torch.Tensor, cmat: torch.Tensor, step_size
     dt B x^T; out = S^T C + d_skip x per head, S [state_dim, vdim] float32 from ``state`` [slots, heads, state_dim, vdim],
     which is renewed.  ``x`` [n, heads * vdim], ``bmat`` and ``cmat`` [n, groups * state_dim] are column slices of one buffer
     (head h uses group h / (heads / groups)), ``step_size`` [n, heads] has a row stride of its own; ``out`` [n, heads * vdim]
-    float32.  Portions of HEAD_SCAN_RUNS_MIN tokens and more take runs of 64 tokens side by side when ``workspace`` (float32,
-    :func:`head_scan_workspace`) is given."""
+    float32.  With ``workspace`` (float32, :func:`head_scan_workspace`) bfloat16 portions of HEAD_SCAN_MMA_MIN tokens and more
+    run on the tensor cores (sizes in steps of 8, rows that start on 16 bytes), and others of HEAD_SCAN_RUNS_MIN tokens and more
+    take runs of 64 tokens side by side; without it tokens are walked one by one."""
     lib = library()
     ld = _rows(x, "x")
     n = x.shape[0]
@@ -2071,6 +2086,15 @@ def head_scan(x: torch.Tensor, bmat: torch.Tensor, cmat: torch.Tensor, step_size
     assert state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (heads, state_dim, vdim)
     runs = workspace is not None and step.max_new >= HEAD_SCAN_RUNS_MIN
     assert workspace is None or (workspace.dtype == torch.float32 and workspace.is_contiguous())
+    if (workspace is not None and USE_HEAD_SCAN_MMA and x.dtype == torch.bfloat16 and step.max_new >= HEAD_SCAN_MMA_MIN
+            and head_scan_mma_supports(state_dim, vdim) and ld % 8 == 0 and _rows(out, "out") % 2 == 0
+            and all(t.data_ptr() % 16 == 0 for t in (x, bmat, cmat, out))):
+        _check(lib.hfee_head_scan_mma(x.data_ptr(), bmat.data_ptr(), cmat.data_ptr(), ld, step_size.data_ptr(), _rows(step_size, "step"),
+                                      dt_bias.data_ptr(), a_log.data_ptr(), d_skip.data_ptr(), state.data_ptr(), step.cu_tokens.data_ptr(),
+                                      step.slots.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r, n, heads, groups, state_dim, vdim,
+                                      int(write_state), workspace.data_ptr(), workspace.numel(), _stream()), lib)
+        count_launches(2)
+        return
     _check(lib.hfee_head_scan(x.data_ptr(), bmat.data_ptr(), cmat.data_ptr(), ld, step_size.data_ptr(), _rows(step_size, "step"), _dt(x),
                               dt_bias.data_ptr(), a_log.data_ptr(), d_skip.data_ptr(), state.data_ptr(), step.cu_tokens.data_ptr(),
                               step.slots.data_ptr(), out.data_ptr(), _rows(out, "out"), step.r, n, heads, groups, state_dim, vdim,
@@ -2081,12 +2105,15 @@ def head_scan(x: torch.Tensor, bmat: torch.Tensor, cmat: torch.Tensor, step_size
 
 def head_scan_takes_workspace(step) -> bool:
     """Whether a step has a portion long enough for the paths of :func:`head_scan` that need a workspace."""
-    return step.max_new >= HEAD_SCAN_RUNS_MIN
+    return step.max_new >= min(HEAD_SCAN_RUNS_MIN, HEAD_SCAN_MMA_MIN)
 
 
 def head_scan_workspace(requests: int, tokens: int, heads: int, state_dim: int, vdim: int) -> int:
     """Floats of workspace :func:`head_scan` wants for steps of at most ``tokens`` tokens of ``requests`` requests."""
-    return gated_recurrence_workspace(requests, tokens, heads, state_dim, vdim)
+    walk = gated_recurrence_workspace(requests, tokens, heads, state_dim, vdim)
+    if not head_scan_mma_supports(state_dim, vdim):
+        return walk
+    return max(walk, int(library().hfee_head_scan_mma_workspace(requests, tokens, heads, state_dim, vdim)))
 
 
 def gate_parts_norm(x: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, parts: int, out: torch.Tensor,
