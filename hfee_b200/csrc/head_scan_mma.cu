@@ -24,7 +24,7 @@
 namespace {
 
 constexpr int HS_T = 64;            // tokens of a run
-constexpr int HS_WARPS = 4;
+constexpr int HS_WARPS = 4;         // of a block of outputs
 constexpr int HS_THREADS = HS_WARPS * 32;
 constexpr int HS_COLS_STATES = 32;  // columns of x per block of the walk
 constexpr int HS_COLS_OUT = 64;     // and of the outputs
@@ -83,62 +83,70 @@ __device__ __forceinline__ void split_pair(float a, float b, uint32_t& hi, uint3
 }
 
 // ------------------------------------------------------------------------------------------ (1) gates
-__global__ void __launch_bounds__(256)
+constexpr int HS_GATE_HEADS = 8;    // heads per block, one per warp
+
+__global__ void __launch_bounds__(HS_GATE_HEADS * 32)
 head_scan_gates_kernel(HeadScanArgs p) {
-  __shared__ float dt_s[HS_T][33];
+  __shared__ float dt_s[HS_T][HS_GATE_HEADS + 1];
   int req = 0, run = 0;
   const bool mine = hs_find_run(p.cu_tokens, p.requests, blockIdx.y, &req, &run);
+  const int h0 = blockIdx.x * HS_GATE_HEADS, lane = threadIdx.x & 31, j = threadIdx.x >> 5;
+  const int own = h0 + (threadIdx.x % HS_GATE_HEADS);
+  const float bias = own < p.heads ? p.dt_bias[own] : 0.f;
+  const float rate = h0 + j < p.heads ? -expf(p.a_log[h0 + j]) * HS_LOG2E : 0.f;
   pdl_wait();
   pdl_launch_dependents();
   if (!mine) return;
   const int begin = p.cu_tokens[req] + run * HS_T, n = min(HS_T, p.cu_tokens[req + 1] - begin);
-  const int h0 = blockIdx.x * 32, lane = threadIdx.x & 31;
-  for (int e = threadIdx.x; e < HS_T * 32; e += 256) {
-    const int t = e >> 5, h = h0 + (e & 31);
+#pragma unroll
+  for (int i = 0; i < HS_T / 32; ++i) {
+    const int t = threadIdx.x / HS_GATE_HEADS + i * 32;
     float dt = 0.f;
-    if (t < n && h < p.heads) {
-      const float z = __bfloat162float(p.step[(long long)(begin + t) * p.ld_step + h]) + p.dt_bias[h];
+    if (t < n && own < p.heads) {
+      const float z = __bfloat162float(p.step[(long long)(begin + t) * p.ld_step + own]) + bias;
       dt = fmaxf(z, 0.f) + log1pf(expf(-fabsf(z)));
     }
-    dt_s[t][e & 31] = dt;
+    dt_s[t][threadIdx.x % HS_GATE_HEADS] = dt;
   }
   __syncthreads();
-  for (int j = threadIdx.x >> 5; j < 32; j += 8) {
-    const int h = h0 + j;
-    if (h >= p.heads) break;                             // the same for the whole warp
-    const float rate = -expf(p.a_log[h]) * HS_LOG2E;
-    const float d0 = dt_s[2 * lane][j], d1 = dt_s[2 * lane + 1][j];
-    const float a0 = rate * d0, a1 = rate * d1;
-    float sum = a0 + a1;
+  if (h0 + j >= p.heads) return;
+  const float d0 = dt_s[2 * lane][j], d1 = dt_s[2 * lane + 1][j];
+  const float a0 = rate * d0, a1 = rate * d1;
+  float sum = a0 + a1;
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const float before = __shfl_up_sync(0xffffffffu, sum, o);
-      if (lane >= o) sum += before;
-    }
-    float front = __shfl_up_sync(0xffffffffu, sum, 1);
-    if (lane == 0) front = 0.f;
-    const long long at = (long long)h * p.n_tokens + begin + 2 * lane;
-    if (2 * lane < n) { p.gate_s[at] = front + a0; p.gate_dt[at] = d0; }
-    if (2 * lane + 1 < n) { p.gate_s[at + 1] = front + a0 + a1; p.gate_dt[at + 1] = d1; }
+  for (int o = 1; o < 32; o <<= 1) {
+    const float before = __shfl_up_sync(0xffffffffu, sum, o);
+    if (lane >= o) sum += before;
   }
+  float front = __shfl_up_sync(0xffffffffu, sum, 1);
+  if (lane == 0) front = 0.f;
+  const long long at = (long long)(h0 + j) * p.n_tokens + begin + 2 * lane;
+  if (2 * lane < n) { p.gate_s[at] = front + a0; p.gate_dt[at] = d0; }
+  if (2 * lane + 1 < n) { p.gate_s[at + 1] = front + a0 + a1; p.gate_dt[at + 1] = d1; }
 }
 
 // ------------------------------------------------------------------------------------------ (2) states
+// Warps 0..7 keep the state (transposed) and multiply: warp w has the columns 16 (w & 1) .. + 15 of the block's 32 and a
+// quarter of the state entries.  Warps 8..11 bring the runs in (three in flight) and weigh the next run's x while this
+// run is multiplied; one barrier a run.
+constexpr int HS_MUL_WARPS = 8, HS_IN_WARPS = 4, HS_IN = HS_IN_WARPS * 32;
+constexpr int HS_STATES_THREADS = (HS_MUL_WARPS + HS_IN_WARPS) * 32;
+
 template <int NP> struct StatesCfg {
   static constexpr int TILES = NP / 16;                    // tiles of 16 state entries
-  static constexpr int MINE = TILES >= HS_WARPS ? TILES / HS_WARPS : 1;   // per warp
+  static constexpr int MINE = TILES >= 4 ? TILES / 4 : 1;  // per warp
   static constexpr int LDB = NP + HS_PAD, LDX = HS_COLS_STATES + HS_PAD;
   static constexpr int STAGE = HS_T * (LDB + LDX) * 2 + 2 * HS_T * 4;     // bytes: B, x, s, dt of one run
-  static constexpr int SMEM = 2 * STAGE + 2 * HS_T * LDX * 2;             // + the weighted x, high and low
+  static constexpr int SMEM = 3 * STAGE + 4 * HS_T * LDX * 2;             // + the weighted x of two runs, high and low
 };
 
 template <int NP>
-__global__ void __launch_bounds__(HS_THREADS)
+__global__ void __launch_bounds__(HS_STATES_THREADS)
 head_scan_states_kernel(HeadScanArgs p) {
   using C = StatesCfg<NP>;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int head = blockIdx.x, req = blockIdx.y, c0 = blockIdx.z * HS_COLS_STATES;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int begin = p.cu_tokens[req], count = p.cu_tokens[req + 1] - begin;
   const int slot = p.slots[req];
   int first_run = 0;
@@ -147,77 +155,47 @@ head_scan_states_kernel(HeadScanArgs p) {
   pdl_wait();
   pdl_launch_dependents();
   if (count <= 0) return;
-  bf16* wx_hi = reinterpret_cast<bf16*>(smem_raw + 2 * C::STAGE);        // [HS_T][LDX]
-  bf16* wx_lo = wx_hi + HS_T * C::LDX;
-  auto b_of = [&](int st) { return reinterpret_cast<bf16*>(smem_raw + st * C::STAGE); };
-  auto x_of = [&](int st) { return b_of(st) + HS_T * C::LDB; };
-  auto s_of = [&](int st) { return reinterpret_cast<float*>(x_of(st) + HS_T * C::LDX); };
-  auto load = [&](int run, int st) {
-    const int row0 = begin + run * HS_T, n = min(HS_T, count - run * HS_T);
-    bf16* bd = b_of(st);
-    bf16* xd = x_of(st);
-    float* sd = s_of(st);
+  bf16* wx = reinterpret_cast<bf16*>(smem_raw + 3 * C::STAGE);            // [2 runs][high, low][HS_T][LDX]
+  auto b_of = [&](int run) { return reinterpret_cast<bf16*>(smem_raw + (run % 3) * C::STAGE); };
+  auto x_of = [&](int run) { return b_of(run) + HS_T * C::LDB; };
+  auto s_of = [&](int run) { return reinterpret_cast<float*>(x_of(run) + HS_T * C::LDX); };
+  auto wx_of = [&](int run, int low) { return wx + ((run & 1) * 2 + low) * HS_T * C::LDX; };
+  const int runs = hs_runs(count);
+  const int tid = threadIdx.x - HS_MUL_WARPS * 32;         // among the warps that bring the runs in
+
+  auto load = [&](int run) {                               // always a group, also when there is no such run
+    if (run < runs) {
+      const int row0 = begin + run * HS_T, n = min(HS_T, count - run * HS_T);
+      bf16* bd = b_of(run);
+      bf16* xd = x_of(run);
+      float* sd = s_of(run);
 #pragma unroll
-    for (int e = tid; e < HS_T * (NP / 8); e += HS_THREADS) {
-      const int s = e / (NP / 8), k = (e % (NP / 8)) * 8;
-      const bool ok = s < n && k < p.n_state;
-      hs_copy16(bd + s * C::LDB + k, ok ? p.b + (long long)(row0 + s) * p.ld + group * p.n_state + k : p.b, ok);
-    }
+      for (int e = tid; e < HS_T * (NP / 8); e += HS_IN) {
+        const int s = e / (NP / 8), k = (e % (NP / 8)) * 8;
+        const bool ok = s < n && k < p.n_state;
+        hs_copy16(bd + s * C::LDB + k, ok ? p.b + (long long)(row0 + s) * p.ld + group * p.n_state + k : p.b, ok);
+      }
 #pragma unroll
-    for (int e = tid; e < HS_T * (HS_COLS_STATES / 8); e += HS_THREADS) {
-      const int s = e / (HS_COLS_STATES / 8), c = (e % (HS_COLS_STATES / 8)) * 8;
-      const bool ok = s < n && c0 + c < p.vdim;
-      hs_copy16(xd + s * C::LDX + c, ok ? p.x + (long long)(row0 + s) * p.ld + (long long)head * p.vdim + c0 + c : p.x, ok);
+      for (int e = tid; e < HS_T * (HS_COLS_STATES / 8); e += HS_IN) {
+        const int s = e / (HS_COLS_STATES / 8), c = (e % (HS_COLS_STATES / 8)) * 8;
+        const bool ok = s < n && c0 + c < p.vdim;
+        hs_copy16(xd + s * C::LDX + c, ok ? p.x + (long long)(row0 + s) * p.ld + (long long)head * p.vdim + c0 + c : p.x, ok);
+      }
+      const int s = tid % HS_T;
+      const float* src = (tid < HS_T ? p.gate_s : p.gate_dt) + (long long)head * p.n_tokens + row0;
+      hs_copy4(sd + tid, s < n ? src + s : p.gate_s, s < n);              // s first, dt behind it
     }
-    const int s = tid % HS_T;
-    const float* src = (tid < HS_T ? p.gate_s : p.gate_dt) + (long long)head * p.n_tokens + row0;
-    hs_copy4(sd + tid, s < n ? src + s : p.gate_s, s < n);                // s first, dt behind it
     hs_commit();
   };
-  load(0, 0);
-
-  float acc[2][2 * C::MINE][4];                            // [16 columns][8 state entries]: S transposed
-  float* S_g = p.state + ((long long)slot * p.heads + head) * p.n_state * p.vdim;
-  const bool active = warp < C::TILES;
-#pragma unroll
-  for (int m = 0; m < 2; ++m)
-#pragma unroll
-    for (int j = 0; j < 2 * C::MINE; ++j)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int c = c0 + m * 16 + g + (i >= 2 ? 8 : 0), k = warp * C::MINE * 16 + j * 8 + 2 * t + (i & 1);
-        acc[m][j][i] = active && c < p.vdim && k < p.n_state ? S_g[(long long)k * p.vdim + c] : 0.f;
-      }
-  const int runs = hs_runs(count);
-  for (int run = 0; run < runs; ++run) {
-    const int st = run & 1, n = min(HS_T, count - run * HS_T);
-    hs_wait_all();
-    __syncthreads();                                       // the run's rows are here, the run before is used up
-    if (run + 1 < runs) load(run + 1, st ^ 1);
-    // the state in front of the run, as B fragments
-    if (active) {
-      uint4* dst = p.carried + ((long long)(first_run + run) * p.heads + head) * (C::TILES * p.ctiles * 32) + lane;
-#pragma unroll
-      for (int m = 0; m < 2; ++m)
-#pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int ct = c0 / 8 + m * 2 + half;
-          if (ct >= p.ctiles) continue;
-#pragma unroll
-          for (int j = 0; j < C::MINE; ++j) {
-            uint4 f;
-            split_pair(acc[m][2 * j][2 * half], acc[m][2 * j][2 * half + 1], f.x, f.z);
-            split_pair(acc[m][2 * j + 1][2 * half], acc[m][2 * j + 1][2 * half + 1], f.y, f.w);
-            dst[((warp * C::MINE + j) * p.ctiles + ct) * 32] = f;
-          }
-        }
-    }
-    const float* ss = s_of(st);
+  auto weigh = [&](int run) {
+    if (run >= runs) return;
+    const int n = min(HS_T, count - run * HS_T);
+    const float* ss = s_of(run);
     const float* sdt = ss + HS_T;
+    const bf16* xs = x_of(run);
     const float s_last = ss[n - 1];
-    const bf16* xs = x_of(st);
 #pragma unroll
-    for (int e = tid; e < HS_T * (HS_COLS_STATES / 8); e += HS_THREADS) {
+    for (int e = tid; e < HS_T * (HS_COLS_STATES / 8); e += HS_IN) {
       const int s = e / (HS_COLS_STATES / 8), c = (e % (HS_COLS_STATES / 8)) * 8;
       const float w = s < n ? hs_exp2(s_last - ss[s]) * sdt[s] : 0.f;
       const uint4 raw = *reinterpret_cast<const uint4*>(xs + s * C::LDX + c);
@@ -226,60 +204,104 @@ head_scan_states_kernel(HeadScanArgs p) {
 #pragma unroll
       for (int i = 0; i < 4; ++i)
         split_pair(__uint_as_float(in[i] << 16) * w, __uint_as_float(in[i] & 0xffff0000u) * w, hi[i], lo[i]);
-      *reinterpret_cast<uint4*>(wx_hi + s * C::LDX + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(wx_lo + s * C::LDX + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      *reinterpret_cast<uint4*>(wx_of(run, 0) + s * C::LDX + c) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      *reinterpret_cast<uint4*>(wx_of(run, 1) + s * C::LDX + c) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
     }
+  };
+  auto landed = [&]() {                                    // all copies but the newest run's, of every thread that copies
+    asm volatile("cp.async.wait_group 1;\n" ::);
+    asm volatile("bar.sync 1, %0;" ::"n"(HS_IN) : "memory");
+  };
+
+  if (warp >= HS_MUL_WARPS) {
+    load(0);
+    load(1);
+    landed();
+    weigh(0);
     __syncthreads();
-    const float decay = hs_exp2(s_last);
+    for (int run = 0; run < runs; ++run) {
+      load(run + 2);                                       // its place was used up before the last barrier
+      landed();
+      weigh(run + 1);
+      __syncthreads();
+    }
+    hs_wait_all();
+    return;
+  }
+
+  const int m0 = (warp & 1) * 16, tile0 = (warp >> 1) * C::MINE;
+  const bool active = tile0 < C::TILES;
+  float acc[2 * C::MINE][4];                               // [8 state entries]: S transposed, 16 columns
+  float* S_g = p.state + ((long long)slot * p.heads + head) * p.n_state * p.vdim;
 #pragma unroll
-    for (int m = 0; m < 2; ++m)
+  for (int j = 0; j < 2 * C::MINE; ++j)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = c0 + m0 + g + (i >= 2 ? 8 : 0), k = tile0 * 16 + j * 8 + 2 * t + (i & 1);
+      acc[j][i] = active && c < p.vdim && k < p.n_state ? S_g[(long long)k * p.vdim + c] : 0.f;
+    }
+  __syncthreads();
+  for (int run = 0; run < runs; ++run) {
+    if (active) {
+      const int n = min(HS_T, count - run * HS_T);
+      const float decay = hs_exp2(s_of(run)[n - 1]);
+      // the state in front of the run, as B fragments
+      uint4* dst = p.carried + ((long long)(first_run + run) * p.heads + head) * (C::TILES * p.ctiles * 32) + lane;
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const int ct = (c0 + m0) / 8 + half;
+        if (ct >= p.ctiles) continue;
+#pragma unroll
+        for (int j = 0; j < C::MINE; ++j) {
+          uint4 f;
+          split_pair(acc[2 * j][2 * half], acc[2 * j][2 * half + 1], f.x, f.z);
+          split_pair(acc[2 * j + 1][2 * half], acc[2 * j + 1][2 * half + 1], f.y, f.w);
+          dst[((tile0 + j) * p.ctiles + ct) * 32] = f;
+        }
+      }
 #pragma unroll
       for (int j = 0; j < 2 * C::MINE; ++j)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) acc[m][j][i] *= decay;
-    if (active) {
-      const bf16* bs = b_of(st);
+        for (int i = 0; i < 4; ++i) acc[j][i] *= decay;
+      const bf16* bs = b_of(run);
 #pragma unroll
       for (int ks = 0; ks < HS_T / 16; ++ks) {
-        uint32_t ah[2][4], al[2][4];
-#pragma unroll
-        for (int m = 0; m < 2; ++m) {
-          load_a_trans(ah[m], wx_hi, C::LDX, m * 16, ks * 16, lane);
-          load_a_trans(al[m], wx_lo, C::LDX, m * 16, ks * 16, lane);
-        }
+        uint32_t ah[4], al[4];
+        load_a_trans(ah, wx_of(run, 0), C::LDX, m0, ks * 16, lane);
+        load_a_trans(al, wx_of(run, 1), C::LDX, m0, ks * 16, lane);
 #pragma unroll
         for (int j = 0; j < C::MINE; ++j) {
           uint32_t b[4];
-          load_b_pair_trans(b, bs, C::LDB, (warp * C::MINE + j) * 16, ks * 16, lane);
-#pragma unroll
-          for (int m = 0; m < 2; ++m) {
-            mma_bf16(acc[m][2 * j], ah[m], b[0], b[1]);
-            mma_bf16(acc[m][2 * j + 1], ah[m], b[2], b[3]);
-            mma_bf16(acc[m][2 * j], al[m], b[0], b[1]);
-            mma_bf16(acc[m][2 * j + 1], al[m], b[2], b[3]);
-          }
+          load_b_pair_trans(b, bs, C::LDB, (tile0 + j) * 16, ks * 16, lane);
+          mma_bf16(acc[2 * j], ah, b[0], b[1]);
+          mma_bf16(acc[2 * j + 1], ah, b[2], b[3]);
+          mma_bf16(acc[2 * j], al, b[0], b[1]);
+          mma_bf16(acc[2 * j + 1], al, b[2], b[3]);
         }
       }
     }
+    __syncthreads();
   }
-  if (!p.write_state) return;
+  if (!p.write_state || !active) return;
 #pragma unroll
-  for (int m = 0; m < 2; ++m)
+  for (int j = 0; j < 2 * C::MINE; ++j)
 #pragma unroll
-    for (int j = 0; j < 2 * C::MINE; ++j)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int c = c0 + m * 16 + g + (i >= 2 ? 8 : 0), k = warp * C::MINE * 16 + j * 8 + 2 * t + (i & 1);
-        if (active && c < p.vdim && k < p.n_state) S_g[(long long)k * p.vdim + c] = acc[m][j][i];
-      }
+    for (int i = 0; i < 4; ++i) {
+      const int c = c0 + m0 + g + (i >= 2 ? 8 : 0), k = tile0 * 16 + j * 8 + 2 * t + (i & 1);
+      if (c < p.vdim && k < p.n_state) S_g[(long long)k * p.vdim + c] = acc[j][i];
+    }
 }
 
 // ------------------------------------------------------------------------------------------ (3) outputs
+// Warp w owns the run's tokens 16 w .. + 15 for C . B and the weights made of it, which meet in shared memory, and the
+// columns 16 w .. + 15 of the outputs of all of the run's tokens, so that a fragment of the state is read once per block.
 template <int NP> struct OutCfg {
   static constexpr int TILES = NP / 16;
-  static constexpr int LDB = NP + HS_PAD, LDX = HS_COLS_OUT + HS_PAD;
+  static constexpr int LDB = NP + HS_PAD, LDX = HS_COLS_OUT + HS_PAD, LDP = HS_T + HS_PAD;
   static constexpr int X_STAGE = HS_T * LDX * 2 + 2 * HS_T * 4;           // bytes: x, s, dt of one head
-  static constexpr int SMEM = 2 * HS_T * LDB * 2 + 2 * X_STAGE;
+  static constexpr int B_BYTES = HS_T * LDB * 2, P_BYTES = 2 * HS_T * LDP * 2;
+  static constexpr int SHARED = B_BYTES > P_BYTES ? B_BYTES : P_BYTES;    // B, later the weights (high and low)
+  static constexpr int SMEM = HS_T * LDB * 2 + SHARED + 2 * X_STAGE;
 };
 
 template <int NP>
@@ -298,7 +320,9 @@ head_scan_outputs_kernel(HeadScanArgs p) {
   const int group = head0 / (p.heads / p.groups);
   bf16* cs = reinterpret_cast<bf16*>(smem_raw);            // [HS_T][LDB]
   bf16* bs = cs + HS_T * C::LDB;                           // [HS_T][LDB]
-  unsigned char* stages = smem_raw + 2 * HS_T * C::LDB * 2;
+  bf16* w_hi = bs;                                         // [HS_T][LDP], once C . B is known
+  bf16* w_lo = w_hi + HS_T * C::LDP;
+  unsigned char* stages = smem_raw + HS_T * C::LDB * 2 + C::SHARED;
   auto x_of = [&](int st) { return reinterpret_cast<bf16*>(stages + st * C::X_STAGE); };
   auto s_of = [&](int st) { return reinterpret_cast<float*>(x_of(st) + HS_T * C::LDX); };
   auto load_head = [&](int head, int st) {
@@ -327,8 +351,8 @@ head_scan_outputs_kernel(HeadScanArgs p) {
   hs_wait_all();
   __syncthreads();
 
-  const int r0 = warp * 16;
   // C . B of the warp's 16 tokens with the tokens up to the diagonal, for all heads of the block
+  const int r0 = warp * 16;
   float cb[HS_T / 8][4];
 #pragma unroll
   for (int j = 0; j < HS_T / 8; ++j) cb[j][0] = cb[j][1] = cb[j][2] = cb[j][3] = 0.f;
@@ -346,85 +370,110 @@ head_scan_outputs_kernel(HeadScanArgs p) {
       }
     }
   }
-  const int ct0 = c0 / 8, cts = min(HS_COLS_OUT / 8, p.ctiles - ct0);
+  __syncthreads();                                         // B is used up: its place takes the weights
+  const int ct0 = c0 / 8 + 2 * warp;                       // the warp's two tiles of 8 columns
+  const int cts = min(2, p.ctiles - ct0);                  // 0 or less: none of them exists
+  const int row_tiles = (n + 15) / 16;
   for (int hh = 0; hh < p.heads_per_block; ++hh) {
     const int head = head0 + hh, st = hh & 1;
     if (hh + 1 < p.heads_per_block) load_head(head + 1, st ^ 1);
-    float acc[HS_COLS_OUT / 8][4];
+    // the state in front of the run: requested before the weights are computed
+    const uint4* S = p.carried + ((long long)(blockIdx.x) * p.heads + head) * (C::TILES * p.ctiles * 32) + ct0 * 32 + lane;
+    constexpr int AHEAD = C::TILES < 8 ? C::TILES : 8;
+    uint4 f[AHEAD][2];
 #pragma unroll
-    for (int j = 0; j < HS_COLS_OUT / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-    if (r0 < n) {
-      const float* ss = s_of(st);
-      const float* sdt = ss + HS_T;
-      const bf16* xs = x_of(st);
+    for (int kk = 0; kk < AHEAD; ++kk)
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+        if (j < cts) f[kk][j] = S[(kk * p.ctiles + j) * 32];
+    const float* ss = s_of(st);
+    const float* sdt = ss + HS_T;
+    const bf16* xs = x_of(st);
+    // weights e^(s_t - s_u) dt_u (C_t . B_u)
+    const float s_lo = ss[r0 + g], s_hi = ss[r0 + g + 8];
+#pragma unroll
+    for (int q = 0; q < HS_T / 8; ++q) {
+      if (q < 2 * (warp + 1)) {
+        const int u = q * 8 + 2 * t;
+        const float2 su = *reinterpret_cast<const float2*>(ss + u), du = *reinterpret_cast<const float2*>(sdt + u);
+        const int lo_row = r0 + g, hi_row = r0 + g + 8;
+        const float w0 = u <= lo_row ? cb[q][0] * (hs_exp2(s_lo - su.x) * du.x) : 0.f;
+        const float w1 = u + 1 <= lo_row ? cb[q][1] * (hs_exp2(s_lo - su.y) * du.y) : 0.f;
+        const float w2 = u <= hi_row ? cb[q][2] * (hs_exp2(s_hi - su.x) * du.x) : 0.f;
+        const float w3 = u + 1 <= hi_row ? cb[q][3] * (hs_exp2(s_hi - su.y) * du.y) : 0.f;
+        uint32_t hi, lo;
+        split_pair(w0, w1, hi, lo);
+        *reinterpret_cast<uint32_t*>(w_hi + lo_row * C::LDP + u) = hi;
+        *reinterpret_cast<uint32_t*>(w_lo + lo_row * C::LDP + u) = lo;
+        split_pair(w2, w3, hi, lo);
+        *reinterpret_cast<uint32_t*>(w_hi + hi_row * C::LDP + u) = hi;
+        *reinterpret_cast<uint32_t*>(w_lo + hi_row * C::LDP + u) = lo;
+      }
+    }
+    __syncthreads();
+    if (cts > 0) {
+      float acc[HS_T / 16][2][4];
+#pragma unroll
+      for (int r = 0; r < HS_T / 16; ++r)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) acc[r][j][0] = acc[r][j][1] = acc[r][j][2] = acc[r][j][3] = 0.f;
       // what the state in front of the run gives
-      const uint4* S = p.carried + ((long long)(blockIdx.x) * p.heads + head) * (C::TILES * p.ctiles * 32) + ct0 * 32 + lane;
-      uint4 f[2][HS_COLS_OUT / 8];
-#pragma unroll
-      for (int j = 0; j < HS_COLS_OUT / 8; ++j)
-        if (j < cts) f[0][j] = S[j * 32];
 #pragma unroll
       for (int kk = 0; kk < C::TILES; ++kk) {
-        if (kk + 1 < C::TILES) {
 #pragma unroll
-          for (int j = 0; j < HS_COLS_OUT / 8; ++j)
-            if (j < cts) f[(kk + 1) & 1][j] = S[((kk + 1) * p.ctiles + j) * 32];
-        }
-        uint32_t a[4];
-        load_a(a, cs, C::LDB, r0, kk * 16, lane);
+        for (int r = 0; r < HS_T / 16; ++r) {
+          uint32_t a[4];
+          load_a(a, cs, C::LDB, r * 16, kk * 16, lane);
 #pragma unroll
-        for (int j = 0; j < HS_COLS_OUT / 8; ++j)
-          if (j < cts) {
-            mma_bf16(acc[j], a, f[kk & 1][j].x, f[kk & 1][j].y);
-            mma_bf16(acc[j], a, f[kk & 1][j].z, f[kk & 1][j].w);
+          for (int j = 0; j < 2; ++j) {
+            mma_bf16(acc[r][j], a, f[kk % AHEAD][j].x, f[kk % AHEAD][j].y);
+            mma_bf16(acc[r][j], a, f[kk % AHEAD][j].z, f[kk % AHEAD][j].w);
           }
-      }
-      const float s_lo = ss[r0 + g], s_hi = ss[r0 + g + 8];
-      const float e_lo = hs_exp2(s_lo), e_hi = hs_exp2(s_hi);
+        }
+        if (kk + AHEAD < C::TILES) {
 #pragma unroll
-      for (int j = 0; j < HS_COLS_OUT / 8; ++j) { acc[j][0] *= e_lo; acc[j][1] *= e_lo; acc[j][2] *= e_hi; acc[j][3] *= e_hi; }
-      // what the run's own tokens give: weights e^(s_t - s_u) dt_u (C_t . B_u), straight from the accumulators
+          for (int j = 0; j < 2; ++j)
+            if (j < cts) f[kk % AHEAD][j] = S[((kk + AHEAD) * p.ctiles + j) * 32];
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < HS_T / 16; ++r) {
+        const float e_lo = hs_exp2(ss[r * 16 + g]), e_hi = hs_exp2(ss[r * 16 + g + 8]);
+#pragma unroll
+        for (int j = 0; j < 2; ++j) { acc[r][j][0] *= e_lo; acc[r][j][1] *= e_lo; acc[r][j][2] *= e_hi; acc[r][j][3] *= e_hi; }
+      }
+      // what the run's own tokens give
 #pragma unroll
       for (int kt = 0; kt < HS_T / 16; ++kt) {
-        if (kt <= warp) {
+        uint32_t b[4];
+        load_b_pair_trans(b, xs, C::LDX, warp * 16, kt * 16, lane);
+#pragma unroll
+        for (int r = kt; r < HS_T / 16; ++r) {
           uint32_t ah[4], al[4];
-#pragma unroll
-          for (int q = 0; q < 2; ++q) {
-            const int u = kt * 16 + q * 8 + 2 * t;
-            const float su0 = ss[u], su1 = ss[u + 1], du0 = sdt[u], du1 = sdt[u + 1];
-            const int lo_row = r0 + g, hi_row = r0 + g + 8;
-            const float* v = cb[2 * kt + q];
-            const float w0 = u <= lo_row ? v[0] * (hs_exp2(s_lo - su0) * du0) : 0.f;
-            const float w1 = u + 1 <= lo_row ? v[1] * (hs_exp2(s_lo - su1) * du1) : 0.f;
-            const float w2 = u <= hi_row ? v[2] * (hs_exp2(s_hi - su0) * du0) : 0.f;
-            const float w3 = u + 1 <= hi_row ? v[3] * (hs_exp2(s_hi - su1) * du1) : 0.f;
-            split_pair(w0, w1, ah[2 * q], al[2 * q]);
-            split_pair(w2, w3, ah[2 * q + 1], al[2 * q + 1]);
-          }
-#pragma unroll
-          for (int j = 0; j < HS_COLS_OUT / 8; j += 2)
-            if (j < cts) {
-              uint32_t b[4];
-              load_b_pair_trans(b, xs, C::LDX, j * 8, kt * 16, lane);
-              mma_bf16(acc[j], ah, b[0], b[1]);
-              mma_bf16(acc[j + 1], ah, b[2], b[3]);
-              mma_bf16(acc[j], al, b[0], b[1]);
-              mma_bf16(acc[j + 1], al, b[2], b[3]);
-            }
+          load_a(ah, w_hi, C::LDP, r * 16, kt * 16, lane);
+          load_a(al, w_lo, C::LDP, r * 16, kt * 16, lane);
+          mma_bf16(acc[r][0], ah, b[0], b[1]);
+          mma_bf16(acc[r][1], ah, b[2], b[3]);
+          mma_bf16(acc[r][0], al, b[0], b[1]);
+          mma_bf16(acc[r][1], al, b[2], b[3]);
         }
       }
       const float skip = p.d_skip[head];
 #pragma unroll
-      for (int j = 0; j < HS_COLS_OUT / 8; ++j) {
-        const int c = c0 + j * 8 + 2 * t;
-        if (c >= p.vdim) continue;
+      for (int r = 0; r < HS_T / 16; ++r) {
+        if (r >= row_tiles) continue;
 #pragma unroll
-        for (int half = 0; half < 2; ++half) {
-          const int row = r0 + g + 8 * half;
-          if (row >= n) continue;
-          const __nv_bfloat162 xv = *reinterpret_cast<const __nv_bfloat162*>(xs + row * C::LDX + j * 8 + 2 * t);
-          *reinterpret_cast<float2*>(p.out + (long long)(begin + row) * p.ld_o + (long long)head * p.vdim + c) =
-              make_float2(fmaf(skip, __bfloat162float(xv.x), acc[j][2 * half]), fmaf(skip, __bfloat162float(xv.y), acc[j][2 * half + 1]));
+        for (int j = 0; j < 2; ++j) {
+          if (j >= cts) continue;
+          const int x_col = warp * 16 + j * 8 + 2 * t, c = c0 + x_col;
+#pragma unroll
+          for (int half = 0; half < 2; ++half) {
+            const int row = r * 16 + g + 8 * half;
+            if (row >= n) continue;
+            const __nv_bfloat162 xv = *reinterpret_cast<const __nv_bfloat162*>(xs + row * C::LDX + x_col);
+            *reinterpret_cast<float2*>(p.out + (long long)(begin + row) * p.ld_o + (long long)head * p.vdim + c) =
+                make_float2(fmaf(skip, __bfloat162float(xv.x), acc[r][j][2 * half]), fmaf(skip, __bfloat162float(xv.y), acc[r][j][2 * half + 1]));
+          }
         }
       }
     }
@@ -444,18 +493,23 @@ int launch_head_scan(HeadScanArgs p, int max_runs, cudaStream_t stream) {
     if (e != cudaSuccess) return hfee_fail(HFEE_ERR_CUDA, "head_scan_mma: cannot get its shared memory: %s", cudaGetErrorString(e));
     configured = true;
   }
-  hfee_launch(head_scan_gates_kernel, dim3((p.heads + 31) / 32, max_runs), dim3(256), 0, stream, p);
+  hfee_launch(head_scan_gates_kernel, dim3((p.heads + HS_GATE_HEADS - 1) / HS_GATE_HEADS, max_runs), dim3(HS_GATE_HEADS * 32), 0, stream, p);
   int rc = hfee_check_launch("head_scan_gates");
   if (rc != HFEE_OK) return rc;
-  hfee_launch(head_scan_states_kernel<NP>, dim3(p.heads, p.requests, (p.vdim + HS_COLS_STATES - 1) / HS_COLS_STATES), dim3(HS_THREADS),
+  hfee_launch(head_scan_states_kernel<NP>, dim3(p.heads, p.requests, (p.vdim + HS_COLS_STATES - 1) / HS_COLS_STATES), dim3(HS_STATES_THREADS),
               StatesCfg<NP>::SMEM, stream, p);
   rc = hfee_check_launch("head_scan_states");
   if (rc != HFEE_OK) return rc;
   const int tiles = (p.vdim + HS_COLS_OUT - 1) / HS_COLS_OUT;
-  // several heads of a group per block share its C . B, as long as the blocks still fill the GPU
-  p.heads_per_block = 1;
-  for (int h : {4, 2})
-    if ((p.heads / p.groups) % h == 0 && (long long)max_runs * (p.heads / h) * tiles >= 2 * hfee_sm_count()) { p.heads_per_block = h; break; }
+  // Several heads of a group per block share its C . B, if the blocks still fill the GPU well: about one head's work for the
+  // shared part and one for each head, times the rounds that the blocks make.
+  const long long slots = (NP <= 128 ? 3 : 2) * (long long)hfee_sm_count();
+  long long best = 0;
+  for (int h : {1, 2, 4}) {
+    if ((p.heads / p.groups) % h != 0) continue;
+    const long long cost = ((long long)max_runs * (p.heads / h) * tiles + slots - 1) / slots * (h + 1);
+    if (best == 0 || cost < best) { best = cost; p.heads_per_block = h; }
+  }
   hfee_launch(head_scan_outputs_kernel<NP>, dim3(max_runs, p.heads / p.heads_per_block, tiles), dim3(HS_THREADS), OutCfg<NP>::SMEM, stream, p);
   return hfee_check_launch("head_scan_outputs");
 }
