@@ -24,6 +24,9 @@
 // last token of the CTA are cleared in shared memory, so that whatever an earlier owner of the page
 // left there (also a NaN) meets no MMA.  Pages of at least 64 tokens (a power of two); other shapes
 // use the mma.sync kernel.  Every barrier wait is bounded.
+// Instances with EXT also take first positions that stay visible behind a window (the blocks that hold them are walked in
+// front of the window's), a cap on the scores, c * tanh(s / c), applied to the row in registers, a sink per query head (one
+// more term exp(sink) of the row sum, added where the row is finished) and a factor on the output.
 // Reference: hostfog/hfee internal/llm/forward.go:146-178, internal/ggml/ops.go:136-150.
 #include "tcgen05.cuh"
 
@@ -58,6 +61,11 @@ struct TcCfg {
   static_assert(SMEM <= 227 * 1024, "shared memory");
 };
 
+// tanh(x) = x P(x^2) on |x| <= 1: P fits tanh(sqrt(u)) / sqrt(u) over the Chebyshev points of 0 .. 1 (largest error of
+// x P(x^2) in float32: 1.4e-7, most of it rounding)
+constexpr int TANH_TERMS = 7;
+constexpr float TANH_P[TANH_TERMS] = {0.999999953f, -0.333328561f, 0.133253981f, -0.0534651838f, 0.0203055276f, -0.00621707439f, 0.0010455543f};
+
 struct TcAttnParams {
   __nv_bfloat16* out; int ld_o;
   const int* block_table; int max_pages; int page_shift; int page_size;
@@ -68,6 +76,13 @@ struct TcAttnParams {
   float scale_log2;
   int window;
   int tokens_per_tile, q_tiles, q_groups;      // q_groups = CTAs along the tokens = ceil(q_tiles / NT)
+  // EXT only
+  int keep_first;              // this many positions from the start stay visible behind the window
+  const float* sink;           // per query head, or null
+  float cap_log2, cap_in;      // > 0: the cap in log2 units, and 2 log2(e) * scale / cap
+  float cap_x;                 // scale / cap
+  float tanh_p[TANH_TERMS];    // TANH_P times the cap in log2 units
+  float out_scale;
 };
 
 __device__ __forceinline__ void tma_load_4d(void* dst, const CUtensorMap* map, int c0, int c1, int c2, int c3,
@@ -129,13 +144,25 @@ __device__ __forceinline__ float2 add2(float2 a, float2 b) {
       : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));
   return d;
 }
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+  float2 d;
+  asm("mul.rn.f32x2 %0, %1, %2;"
+      : "=l"(reinterpret_cast<uint64_t&>(d))
+      : "l"(reinterpret_cast<uint64_t&>(a)), "l"(reinterpret_cast<uint64_t&>(b)));
+  return d;
+}
+__device__ __forceinline__ float fast_reciprocal(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ float max3(float a, float b, float c) {
   float y;
   asm("max.f32 %0, %1, %2, %3;" : "=f"(y) : "f"(a), "f"(b), "f"(c));
   return y;
 }
 
-template <int HD, int NT>
+template <int HD, int NT, bool EXT>
 __global__ void __launch_bounds__(TcCfg<HD, NT>::THREADS, 1)
 attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, TcAttnParams p, int* __restrict__ status) {
@@ -173,7 +200,11 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
   int nb = 0, pos_last_all = 0;
   const int pos_first0 = before + qg * NT * p.tokens_per_tile;
   const int key_lo = (p.window > 0 && pos_first0 + 1 > p.window) ? pos_first0 + 1 - p.window : 0;
-  const int b_lo = key_lo / KB;
+  // the walk's blocks: number j is block j below n_front (kept first positions), block j + skip from there on
+  const int kept = EXT ? min(p.keep_first, key_lo) : 0;
+  const int n_front = EXT ? min((kept + KB - 1) / KB, key_lo / KB) : 0;
+  const int skip = key_lo / KB - n_front;
+  auto block_of = [&](int j) { return EXT && j < n_front ? j : j + skip; };
 #pragma unroll
   for (int t = 0; t < NT; ++t) {
     t_first[t] = (qg * NT + t) * p.tokens_per_tile;
@@ -181,7 +212,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     nb_t[t] = 0;
     if (t_count[t] > 0) {
       const int pos_last = before + t_first[t] + t_count[t] - 1;
-      nb_t[t] = pos_last / KB - b_lo + 1;
+      nb_t[t] = pos_last / KB - skip + 1;
       nb = nb_t[t];
       pos_last_all = pos_last;
     }
@@ -236,7 +267,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
           int page[2], in_page[2];
 #pragma unroll
           for (int c = 0; c < 2; ++c) {                       // two pieces of 64 keys
-            const int key0 = (b_lo + j) * KB + c * 64;
+            const int key0 = block_of(j) * KB + c * 64;
             // a piece beyond the pages the request holds reads page -1: out of range, zero-filled
             page[c] = (key0 >> p.page_shift) < p.max_pages
                           ? p.block_table[(long long)slot * p.max_pages + (key0 >> p.page_shift)] : -1;
@@ -265,7 +296,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         const int j = nb - 1, s = j % ST;
         int done = lane == 0 ? (int)mbar_wait(&v_full[s], (j / ST) & 1u, &abort_flag) : 0;
         done = __shfl_sync(0xffffffffu, done, 0);
-        const int first_row = pos_last_all - (b_lo + j) * KB + 1;       // 1..128
+        const int first_row = pos_last_all - block_of(j) * KB + 1;      // 1..128
         if (done && first_row < KB) {
           unsigned char* v_dst = kv_s + s * 2 * C::KT_BYTES + C::KT_BYTES;
           const int per_slab = (KB - first_row) * 8;                    // 16-byte pieces
@@ -369,7 +400,8 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const uint32_t lane_addr = tmem_base + ((uint32_t)(quad * 32) << 16);
     const uint32_t s_addr = lane_addr + C::S_COL + t * KB, o_addr = lane_addr + C::O_COL + t * HD;
     const uint32_t p_addr = lane_addr + C::P_COL + t * C::P_STRIDE;
-    const float c_log2 = p.scale_log2;
+    const bool capped = EXT && p.cap_log2 > 0.f;           // capped scores are in log2 units already
+    const float c_log2 = capped ? 1.f : p.scale_log2;
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
     // With S_t ready ahead of time the two tiles' softmax threads would run in step and meet in the
@@ -390,7 +422,7 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
 
 #pragma unroll 1
     for (int j = 0; j < my_nb && ok; ++j) {
-      const int key0 = (b_lo + j) * KB;
+      const int key0 = block_of(j) * KB;
       ok = wait_all(&s_full[t], j & 1u);
       tc_fence_after();
       if (!ok) break;
@@ -403,13 +435,39 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         __syncwarp();
         if (lane == 0) mbar_arrive(&s_free[t]);
       }
-      // keys this row may see: [key_min, pos]; blocks wholly inside need no per-element test
+      if constexpr (EXT) {
+        if (capped) {
+          // a cap is wide for nearly every score: where a warp's scores all stay below it, the polynomial (the special-function
+          // unit has an exponential per score to do as it is), else c tanh(x / c) = c - 2 c / (e^(2x / c) + 1)
+          float big = 0.f;
+#pragma unroll
+          for (int i = 0; i < KB; i += 2) big = max3(big, fabsf(v[i]), fabsf(v[i + 1]));
+          if (__all_sync(0xffffffffu, big * p.cap_x <= 1.f)) {
+            const float2 in = make_float2(p.cap_x, p.cap_x);
+#pragma unroll
+            for (int i = 0; i < KB; i += 2) {
+              const float2 x = mul2(make_float2(v[i], v[i + 1]), in), u = mul2(x, x);
+              float2 q = make_float2(p.tanh_p[TANH_TERMS - 1], p.tanh_p[TANH_TERMS - 1]);
+#pragma unroll
+              for (int k = TANH_TERMS - 2; k >= 0; --k) q = fma2(q, u, make_float2(p.tanh_p[k], p.tanh_p[k]));
+              q = mul2(q, x);
+              v[i] = q.x;
+              v[i + 1] = q.y;
+            }
+          } else {
+#pragma unroll
+            for (int i = 0; i < KB; ++i)
+              v[i] = fmaf(-2.f * p.cap_log2, fast_reciprocal(fast_exp2(v[i] * p.cap_in) + 1.f), p.cap_log2);
+          }
+        }
+      }
+      // keys this row may see: [key_min, pos] and the kept ones; blocks wholly inside need no per-element test
       const int key_min = p.window > 0 ? pos - p.window + 1 : -(1 << 30);
       const bool need_mask = __any_sync(0xffffffffu, key0 + KB - 1 > pos || key0 < key_min);
       if (need_mask) {
-        const int hi = pos - key0, lo = key_min - key0;
+        const int hi = pos - key0, lo = key_min - key0, front = EXT ? p.keep_first - key0 : 0;
 #pragma unroll
-        for (int i = 0; i < KB; ++i) v[i] = (i <= hi && i >= lo) ? v[i] : -INFINITY;
+        for (int i = 0; i < KB; ++i) v[i] = (i <= hi && (i >= lo || (EXT && i < front))) ? v[i] : -INFINITY;
       }
       float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -487,7 +545,9 @@ attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     }
     if (ok && my_nb > 0) {
       const int tk = t_first[t] + row / p.group, head = kvh * p.group + row % p.group;
-      const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+      if constexpr (EXT)
+        if (p.sink != nullptr && valid && m_run != -INFINITY) l_run += fast_exp2(p.sink[head] * 1.4426950408889634f - m_run * c_log2);
+      const float inv = l_run > 0.f ? (EXT ? p.out_scale : 1.f) / l_run : 0.f;
       __nv_bfloat16* dst = p.out + (long long)(tok0 + tk) * p.ld_o + (long long)head * HD;
 #pragma unroll
       for (int ch = 0; ch < HD / 32; ++ch) {
@@ -538,20 +598,20 @@ int make_map_4d(CUtensorMap* map, const void* base, const cuuint64_t (&dims)[4],
   return HFEE_OK;
 }
 
-template <int HD, int NT>
+template <int HD, int NT, bool EXT>
 int launch_tc(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, TcAttnParams p, int kv_heads,
               int requests, int* status, cudaStream_t stream) {
   using C = TcCfg<HD, NT>;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<HD, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attention_tc_kernel<HD, NT, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM);
     if (e != cudaSuccess)
       return hfee_fail(HFEE_ERR_CUDA, "attention_tc: cannot get %d bytes of shared memory: %s", C::SMEM, cudaGetErrorString(e));
     configured = true;
   }
   p.q_groups = (p.q_tiles + NT - 1) / NT;
   dim3 grid((unsigned)kv_heads, (unsigned)p.q_groups, (unsigned)requests);
-  hfee_launch(attention_tc_kernel<HD, NT>, grid, dim3(C::THREADS), C::SMEM, stream, mq, mk, mv, p, status);
+  hfee_launch(attention_tc_kernel<HD, NT, EXT>, grid, dim3(C::THREADS), C::SMEM, stream, mq, mk, mv, p, status);
   return hfee_check_launch("attention_tc");
 }
 
@@ -566,13 +626,18 @@ HFEE_API int hfee_attention_tc_supports(int heads, int kv_heads, int head_dim, i
   return 1;
 }
 
-// q [n_tokens, ld_q], out [n_tokens, ld_o]: bfloat16; pools [num_pages, kv_heads, page_size, head_dim].
-HFEE_API int hfee_attention_tc(const void* q, int ld_q, const void* k_pool, const void* v_pool, int num_pages,
+namespace {
+struct TcOptions {
+  int keep_first; float softcap; const float* sink; float out_scale;
+};
+
+int attention_tc_impl(const void* q, int ld_q, const void* k_pool, const void* v_pool, int num_pages,
                                const int* block_table, int max_pages, int page_size, const int* cu_tokens,
                                const int* slots, const int* context_before, void* out, int ld_o, int n_tokens,
                                int requests, int max_new, int heads, int kv_heads, int head_dim, float scale,
-                               int window, int* status, cudaStream_t stream) {
+                               int window, const TcOptions* ext, int* status, cudaStream_t stream) {
   if (n_tokens == 0 || requests == 0) return HFEE_OK;
+  HFEE_REQUIRE(ext == nullptr || ext->keep_first >= 0, "attention_tc: bad mask");
   HFEE_REQUIRE(hfee_attention_tc_supports(heads, kv_heads, head_dim, page_size),
                "attention_tc: needs head_dim 64 or 128, at most 128 query heads per kv head and power-of-two pages "
                ">= 64 (got head_dim %d, heads %d/%d, page_size %d)", head_dim, heads, kv_heads, page_size);
@@ -593,6 +658,13 @@ HFEE_API int hfee_attention_tc(const void* q, int ld_q, const void* k_pool, cons
   p.tokens_per_tile = QM / group;
   p.q_tiles = (max_new + p.tokens_per_tile - 1) / p.tokens_per_tile;
   p.q_groups = 0;
+  p.keep_first = ext ? ext->keep_first : 0;
+  p.sink = ext ? ext->sink : nullptr;
+  p.out_scale = ext ? ext->out_scale : 1.f;
+  p.cap_log2 = ext && ext->softcap > 0.f ? ext->softcap * 1.4426950408889634f : 0.f;
+  p.cap_in = p.cap_log2 > 0.f ? 2.f * p.scale_log2 / ext->softcap : 0.f;
+  p.cap_x = p.cap_log2 > 0.f ? scale / ext->softcap : 0.f;
+  for (int k = 0; k < TANH_TERMS; ++k) p.tanh_p[k] = TANH_P[k] * p.cap_log2;
 
   CUtensorMap mq, mk, mv;
   {
@@ -613,6 +685,37 @@ HFEE_API int hfee_attention_tc(const void* q, int ld_q, const void* k_pool, cons
     rc = make_map_4d(&mv, v_pool, dims, strides, box);
     if (rc != HFEE_OK) return rc;
   }
-  if (head_dim == 64) return launch_tc<64, 2>(mq, mk, mv, p, kv_heads, requests, status, stream);
-  return launch_tc<128, 2>(mq, mk, mv, p, kv_heads, requests, status, stream);
+  if (ext != nullptr) {
+    if (head_dim == 64) return launch_tc<64, 2, true>(mq, mk, mv, p, kv_heads, requests, status, stream);
+    return launch_tc<128, 2, true>(mq, mk, mv, p, kv_heads, requests, status, stream);
+  }
+  if (head_dim == 64) return launch_tc<64, 2, false>(mq, mk, mv, p, kv_heads, requests, status, stream);
+  return launch_tc<128, 2, false>(mq, mk, mv, p, kv_heads, requests, status, stream);
+}
+}  // namespace
+
+// q [n_tokens, ld_q], out [n_tokens, ld_o]: bfloat16; pools [num_pages, kv_heads, page_size, head_dim].
+HFEE_API int hfee_attention_tc(const void* q, int ld_q, const void* k_pool, const void* v_pool, int num_pages,
+                               const int* block_table, int max_pages, int page_size, const int* cu_tokens,
+                               const int* slots, const int* context_before, void* out, int ld_o, int n_tokens,
+                               int requests, int max_new, int heads, int kv_heads, int head_dim, float scale,
+                               int window, int* status, cudaStream_t stream) {
+  return attention_tc_impl(q, ld_q, k_pool, v_pool, num_pages, block_table, max_pages, page_size, cu_tokens, slots,
+                           context_before, out, ld_o, n_tokens, requests, max_new, heads, kv_heads, head_dim, scale, window,
+                           nullptr, status, stream);
+}
+
+// The same with its options: keep_first positions from the start stay visible behind the window, softcap > 0 caps the scaled
+// scores (softcap * tanh(score / softcap)), sink (float32 per query head, or null) is one more term exp(sink) of the row sum,
+// and the output is multiplied by out_scale.
+HFEE_API int hfee_attention_tc_general(const void* q, int ld_q, const void* k_pool, const void* v_pool, int num_pages,
+                                       const int* block_table, int max_pages, int page_size, const int* cu_tokens,
+                                       const int* slots, const int* context_before, void* out, int ld_o, int n_tokens,
+                                       int requests, int max_new, int heads, int kv_heads, int head_dim, float scale,
+                                       int window, int keep_first, float softcap, const float* sink, float out_scale,
+                                       int* status, cudaStream_t stream) {
+  const TcOptions ext{keep_first, softcap, sink, out_scale};
+  return attention_tc_impl(q, ld_q, k_pool, v_pool, num_pages, block_table, max_pages, page_size, cu_tokens, slots,
+                           context_before, out, ld_o, n_tokens, requests, max_new, heads, kv_heads, head_dim, scale, window,
+                           &ext, status, stream);
 }

@@ -43,6 +43,7 @@ _SIGNATURES = {
     "hfee_gemm_ring": [_P, _L, _P, _L, _P, _L, _I, _I, _I, _I, _I, _P, _P],
     "hfee_gemm_ring_supports": [_I, _I, _I, _I],
     "hfee_attention_tc": [_P, _I, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
+    "hfee_attention_tc_general": [_P, _I, _P, _P, _I, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _F, _P, _F, _P, _P],
     "hfee_attention_tc_supports": [_I, _I, _I, _I],
     "hfee_attention_mma": [_P, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P],
     "hfee_attention_mma_rope": [_P, _I, _P, _I, _I, _I, _P, _P, _P, _I, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P, _P],
@@ -1967,8 +1968,9 @@ def softmax_attention(q, k_pool, v_pool, block_table, page_size, step, out, head
     window, an optional ``sink`` (float32 per query head: the denominator also holds exp(sink[h]), a term without key or
     value) and the output times ``out_scale``.  ``keep_first``: that many positions from the start stay visible behind the
     window; ``softcap`` c: a scaled score s becomes c * tanh(s / c).  bfloat16 with key and value sizes that are multiples of 8 (up to 256) runs
-    on the tensor cores (prompt portions, decode steps with their keys split among CTAs when ``scratch`` is given, and
-    mixtures), everything else on the CUDA cores in float32 arithmetic."""
+    on the tensor cores (prompt portions with sizes that :func:`attention_tc` takes on tcgen05, others and decode steps, with
+    their keys split among CTAs when ``scratch`` is given, on ``mma.sync``), everything else on the CUDA cores in float32
+    arithmetic."""
     lib = library()
     group = heads // kv_heads
     assert sink is None or (sink.dtype == torch.float32 and sink.is_contiguous() and sink.numel() == heads)
@@ -1986,6 +1988,14 @@ def softmax_attention(q, k_pool, v_pool, block_table, page_size, step, out, head
                                               value_dim, 0, float(scale), int(window or 0), 0, WEIGHTS_SOFTMAX, None, None, None, 0,
                                               GATE_NONE, None, None, float(out_scale), _ptr(sink), int(keep_first), cap, _dt(q),
                                               _stream()), lib)
+        return
+    if (USE_TC_ATTENTION and head_dim == value_dim and step.max_new * group > 16 and _rows(out, "out") % 8 == 0
+            and out.data_ptr() % 16 == 0 and attention_tc_supports(heads, kv_heads, head_dim, page_size)):
+        _check(lib.hfee_attention_tc_general(q.data_ptr(), _rows(q, "q"), k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[0],
+                                             block_table.data_ptr(), block_table.shape[1], page_size, step.cu_tokens.data_ptr(),
+                                             step.slots.data_ptr(), step.context_before.data_ptr(), out.data_ptr(), _rows(out, "out"),
+                                             step.n, step.r, step.max_new, heads, kv_heads, head_dim, float(scale), int(window or 0),
+                                             int(keep_first), cap, _ptr(sink), float(out_scale), _status().data_ptr(), _stream()), lib)
         return
     splits = 1
     if step.max_new * group <= 16 and scratch is not None:

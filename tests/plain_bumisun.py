@@ -184,9 +184,15 @@ def clamped_expert(w, p, h, limit):
     return (g * sigmoid(1.702 * g) * (u + 1.0)) @ w[p + "down"].T
 
 
+ROUTE_MARGINS = []       # per call: the smallest gap between a chosen logit and the best one left out
+
+
 def choose(logits, top):
     """(experts [T, top], weights [T, top]): the largest logits and the softmax over just those."""
     chosen = np.argsort(-logits, axis=-1, kind="stable")[:, :top]
+    if top < logits.shape[-1]:
+        ranked = np.sort(logits, axis=-1)[:, ::-1]
+        ROUTE_MARGINS.append(float((ranked[:, top - 1] - ranked[:, top]).min()))
     e = np.take_along_axis(logits, chosen, axis=-1)
     e = np.exp(e - e.max(axis=-1, keepdims=True))
     return chosen, e / e.sum(axis=-1, keepdims=True)
