@@ -27,7 +27,10 @@ scan; routed experts with a shared one whose active sizes add up to the dense fe
 attention with a sink, gated linear attention with a decay per key channel; a clamped gated feed-forward in turn with
 group-limited routed experts and a gated shared one; a hashed bigram embedding and layer norms); ``--design fokalorn``
 for a Fokalorn model (a delta rule with a decay per key channel in turn with latent attention over all earlier positions
-with a sink; four residual streams, norms in groups, a token shift, a relu^2 feed-forward), beside a Bamipel model as well.
+with a sink; four residual streams, norms in groups, a token shift, a relu^2 feed-forward), beside a Bamipel model as well;
+``--design bumisun`` for a Bumisun model (windowed attention that keeps the first tokens, with capped scores, a sink and mixed
+values, and a relu-gated feed-forward, in turn with a state-space scan of one decay per head and routed experts), beside a
+Muvetar and a Pupinex model as well.
 ``--breakdown`` prints, instead of the line above, what each class of kernels costs inside the decode
 step at batch 1, 8 and 64 and inside the prompt pass: the step is timed again with that class's
 launches left out (results wrong, timing not), and the difference is the class's cost in place.
@@ -272,11 +275,34 @@ def fokalorn_like(model, layers, streams=4):
             "layers": [kinds[i % 2] for i in range(layers)], "norm": {"eps": 1e-5, "groups": 2}, "embedding": {"scale": 1.0}}
 
 
-DESIGNS = {"fokalorn": fokalorn_like, "dobelix": dobelix_like, "bamipel": bamipel_like, "muvetar": muvetar_like, "pupinex": pupinex_like}
+def bumisun_like(model, layers, experts=16, top=2):
+    """A Bumisun configuration of the layer sizes of the Llama configuration ``model``: in turn attention (the Llama heads, half
+    of every head rotated, a window of 1,024 positions behind which the first four stay visible, scores capped at 30, mixed
+    values) with the dense relu-gated feed-forward, and a scan of twice the width (heads of 64, 128 state entries, as many
+    groups and norm parts as key/value heads, four taps) with ``experts`` routed experts of a quarter of the dense feed-forward
+    each (``top`` chosen) and a gated shared one of half of it."""
+    h, kv, hd = model["num_attention_heads"], model["num_key_value_heads"], model["head_dim"]
+    width, ff = model["hidden_size"], model["intermediate_size"]
+    kinds = [
+        {"type": "attention", "mlp": {"kind": "dense", "ff": ff},
+         "mixer": {"heads": h, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 30.0, "v_mix": True,
+                   "mask": {"size": 1024, "keep_first": 4}, "rot": {"dims": hd // 2, "base": 500000.0}}},
+        {"type": "mamba2",
+         "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": kv, "conv": 4, "norm_groups": kv},
+         "mlp": {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // 4, "limit": 7.0},
+                 "shared": {"ff": ff // 2, "limit": 7.0}}},
+    ]
+    return {"architecture": "Bumisun", "vocab": model["vocab_size"], "width": width, "layers": [kinds[i % 2] for i in range(layers)],
+            "norm": {"eps": 1e-5}, "residual_mult": 0.5, "logit_scale": 1.0}
+
+
+DESIGNS = {"bumisun": bumisun_like, "fokalorn": fokalorn_like, "dobelix": dobelix_like, "bamipel": bamipel_like, "muvetar": muvetar_like, "pupinex": pupinex_like}
 # kernel classes (the names the parts tag their launches with) that only some layers of a design have: class -> the layer
 # types that have it; every other class is counted once per layer ("head": once per model)
-CLOSEST = {"fokalorn": ("bamipel",)}          # designs measured beside this one, after the Llama model
+CLOSEST = {"fokalorn": ("bamipel",), "bumisun": ("muvetar", "pupinex")}          # designs measured beside this one, after the Llama model
 DESIGN_CLASSES = {
+    "bumisun": {"conv": ("mamba2",), "scan": ("mamba2",), "gate": ("mamba2",), "rope": ("attention",), "attention": ("attention",),
+                "router": ("mamba2",), "experts": ("mamba2",)},
     "fokalorn": {"conv": ("channel_delta",), "low_rank": ("channel_delta",), "delta_rule": ("channel_delta",), "gate": ("channel_delta",),
                  "rope": ("latent_attention",), "attention": ("latent_attention",), "fold": ("latent_attention",),
                  "expand": ("latent_attention",)},

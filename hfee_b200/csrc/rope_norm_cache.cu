@@ -279,6 +279,101 @@ attention_prepare_kernel(const T* __restrict__ src, long long ld_src, int q_off,
   }
 }
 
+// attention_prepare without biases and norms for rows that 16-byte accesses can read: a work item is one 16-byte piece of a
+// query, key or value head (with half-split pairing, the piece in the first half of the rotated dimensions and its partner).
+template <typename T, int VEC>
+struct alignas(16) PreparePiece { T v[VEC]; };
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(AP_THREADS)
+attention_prepare_vec_kernel(const T* __restrict__ src, long long ld_src, int q_off, int k_off, int v_off, const float* __restrict__ cs,
+                             int rope_dim, int interleaved, const int* __restrict__ positions, const int* __restrict__ slot_of_token,
+                             T* __restrict__ q_out, long long ld_q, T* __restrict__ k_pool, PagedCache kc, T* __restrict__ v_pool,
+                             PagedCache vc, int heads, int key_dim, T* __restrict__ first_values, long long ld_first, int mix_mode,
+                             float share) {
+  using P = PreparePiece<T, VEC>;
+  const int i = blockIdx.x;
+  const int pos = positions[i], slot = slot_of_token[i];
+  const bool write = k_pool != nullptr;
+  const int page = write ? kc.block_table[(long long)slot * kc.max_pages + (pos >> kc.page_shift)] : 0;
+  const int in_page = pos & (kc.page_size - 1);
+  pdl_wait();
+  pdl_launch_dependents();
+  const T* row = src + (long long)i * ld_src;
+  const float2* csr = reinterpret_cast<const float2*>(cs) + (cs != nullptr ? (long long)i * (rope_dim / 2) : 0);
+  const int kp = key_dim / VEC, vp = write ? vc.head_dim / VEC : 0, half = rope_dim / 2;
+  const int q_items = heads * kp, k_items = write ? kc.kv_heads * kp : 0, v_items = write ? vc.kv_heads * vp : 0;
+  const int stride = AP_THREADS * gridDim.y;
+  for (int w = blockIdx.y * AP_THREADS + threadIdx.x; w < q_items + k_items + v_items; w += stride) {
+    if (w >= q_items + k_items) {                          // a value
+      const int e = w - q_items - k_items, g = e / vp, a = (e - g * vp) * VEC;
+      const int c = g * vc.head_dim + a;
+      P x = *reinterpret_cast<const P*>(row + v_off + c);
+      if (mix_mode == MIX_MIX) {
+        const P f = *reinterpret_cast<const P*>(first_values + (long long)i * ld_first + c);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) x.v[j] = from_f32<T>(fmaf(share, to_f32<T>(f.v[j]), (1.f - share) * to_f32<T>(x.v[j])));
+      }
+      if (mix_mode == MIX_STORE) *reinterpret_cast<P*>(first_values + (long long)i * ld_first + c) = x;
+      *reinterpret_cast<P*>(v_pool + (long long)page * vc.page_stride + ((long long)g * vc.page_size + in_page) * vc.head_dim + a) = x;
+      continue;
+    }
+    const bool is_q = w < q_items;
+    const int e = is_q ? w : w - q_items, h = e / kp, a = (e - h * kp) * VEC;
+    const T* in = row + (is_q ? q_off : k_off) + h * key_dim;
+    T* dst = is_q ? q_out + (long long)i * ld_q + h * key_dim
+                  : k_pool + (long long)page * kc.page_stride + ((long long)h * kc.page_size + in_page) * kc.head_dim;
+    if (cs == nullptr || a >= rope_dim) {
+      *reinterpret_cast<P*>(dst + a) = *reinterpret_cast<const P*>(in + a);
+    } else if (interleaved) {
+      const P x = *reinterpret_cast<const P*>(in + a);
+      P y;
+#pragma unroll
+      for (int j = 0; j < VEC; j += 2) {
+        const float2 c = csr[(a + j) / 2];
+        const float u = to_f32<T>(x.v[j]), v = to_f32<T>(x.v[j + 1]);
+        y.v[j] = from_f32<T>(u * c.x - v * c.y);
+        y.v[j + 1] = from_f32<T>(v * c.x + u * c.y);
+      }
+      *reinterpret_cast<P*>(dst + a) = y;
+    } else if (a < half) {                                 // the partner's piece is done here as well
+      const P x0 = *reinterpret_cast<const P*>(in + a), x1 = *reinterpret_cast<const P*>(in + a + half);
+      P y0, y1;
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        const float2 c = csr[a + j];
+        const float u = to_f32<T>(x0.v[j]), v = to_f32<T>(x1.v[j]);
+        y0.v[j] = from_f32<T>(u * c.x - v * c.y);
+        y1.v[j] = from_f32<T>(v * c.x + u * c.y);
+      }
+      *reinterpret_cast<P*>(dst + a) = y0;
+      *reinterpret_cast<P*>(dst + a + half) = y1;
+    }
+  }
+}
+
+template <typename T>
+bool launch_attention_prepare_vec(const void* src, long long ld_src, int n, int q_off, int k_off, int v_off, const float* cs, int rope_dim,
+                                  int interleaved, const int* positions, const int* slot_of_token, void* q_out, long long ld_q, void* k_pool,
+                                  const PagedCache& kc, void* v_pool, const PagedCache& vc, int heads, int key_dim, void* first_values,
+                                  long long ld_first, int mix_mode, float share, cudaStream_t stream) {
+  constexpr int VEC = 16 / (int)sizeof(T);
+  const auto whole = [](long long e) { return e % VEC == 0; };
+  if (!(whole(ld_src) && whole(q_off) && whole(k_off) && whole(v_off) && whole(ld_q) && whole(key_dim) && whole(vc.head_dim) &&
+        whole(rope_dim) && (interleaved || whole(rope_dim / 2)) && (mix_mode == MIX_NONE || whole(ld_first))))
+    return false;
+  for (const void* p : {src, (const void*)q_out, (const void*)k_pool, (const void*)v_pool, (const void*)first_values})
+    if ((uintptr_t)p % 16 != 0) return false;
+  const int items = heads * (key_dim / VEC) + (k_pool != nullptr ? kc.kv_heads * (key_dim + vc.head_dim) / VEC : 0);
+  // few tokens: one piece per thread; many: a few pieces each
+  const int blocks = (items + AP_THREADS - 1) / AP_THREADS;
+  const dim3 grid((unsigned)n, (unsigned)(n >= 512 ? (blocks + 3) / 4 : blocks));
+  hfee_launch(attention_prepare_vec_kernel<T, VEC>, grid, dim3(AP_THREADS), 0, stream, (const T*)src, ld_src, q_off, k_off, v_off, cs, rope_dim,
+              interleaved, positions, slot_of_token, (T*)q_out, ld_q, (T*)k_pool, kc, (T*)v_pool, vc, heads, key_dim, (T*)first_values, ld_first,
+              mix_mode, share);
+  return true;
+}
+
 template <typename T>
 int launch_rope_norm(const void* src, long long ld_src, int n, const float* cs, int rope_dim, float norm_eps,
                      const int* positions, const int* slot_of_token, const HeadGroup& qg, void* q_out, long long ld_q,
@@ -371,6 +466,15 @@ HFEE_API int hfee_attention_prepare(const void* src, long long ld_src, int dtype
   const size_t smem = sizeof(float) * ((size_t)heads * key_dim + (k_pool != nullptr ? (size_t)kv_heads * (key_dim + value_dim) : 0));
   HFEE_REQUIRE(smem <= 48 * 1024, "attention_prepare: a token's projections (%zu bytes as float32) exceed 48 KB", smem);
   if (cs == nullptr) rope_dim = 0;
+  if (bq == nullptr && bk == nullptr && bv == nullptr && wq == nullptr && wk == nullptr) {
+    const bool done = dtype == HFEE_F32
+        ? launch_attention_prepare_vec<float>(src, ld_src, n, q_off, k_off, v_off, cs, rope_dim, interleaved, positions, slot_of_token, q_out, ld_q,
+                                              k_pool, kc, v_pool, vc, heads, key_dim, first_values, ld_first, mix_mode, share, stream)
+        : dtype == HFEE_BF16 &&
+          launch_attention_prepare_vec<__nv_bfloat16>(src, ld_src, n, q_off, k_off, v_off, cs, rope_dim, interleaved, positions, slot_of_token, q_out,
+                                                      ld_q, k_pool, kc, v_pool, vc, heads, key_dim, first_values, ld_first, mix_mode, share, stream);
+    if (done) return hfee_check_launch("attention_prepare");
+  }
   if (dtype == HFEE_F32)
     hfee_launch(attention_prepare_kernel<float>, dim3(n), dim3(AP_THREADS), smem, stream, (const float*)src, ld_src, q_off, k_off, v_off,
                 bq, bk, bv, wq, wk, eps, cs, rope_dim, interleaved, positions, slot_of_token, (float*)q_out, ld_q, (float*)k_pool, kc,

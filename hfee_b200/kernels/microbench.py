@@ -500,10 +500,18 @@ def _bumisun_rows(args) -> dict:
     o = torch.empty(n, inner, dtype=torch.bfloat16, device=DEV)
     logits, bias = torch.randn(n, args.experts + 1, device=DEV), torch.randn(args.experts, device=DEV)
     choice, weight = torch.empty(n, args.top, dtype=torch.int32, device=DEV), torch.empty(n, args.top, device=DEV)
+    h, kv, hd = args.heads, args.kv_heads, args.head_dim
+    hq, hk, step = h * hd, kv * hd, _batch_of([0], [n])
+    qkv, qo = torch.randn(n, hq + 2 * hk, device=DEV).to(torch.bfloat16), torch.empty(n, hq, dtype=torch.bfloat16, device=DEV)
+    fv, cs = torch.randn(n, hk, device=DEV).to(torch.bfloat16), torch.randn(n, hd // 4, 2, device=DEV)
+    kp, vp = (torch.empty(-(-n // 64), kv, 64, hd, dtype=torch.bfloat16, device=DEV) for _ in range(2))
+    pages = torch.arange(-(-n // 64), dtype=torch.int32, device=DEV)[None].contiguous()
     cases = {
         "embed_norm": (lambda i: ops.embed_norm(table, tok, w, 1e-5, x), n * k * 6),
         "gate_parts_norm": (lambda i: ops.gate_parts_norm(y, z, wi, 1e-5, 1, o), n * inner * 8),
         "gate_parts_norm_8": (lambda i: ops.gate_parts_norm(y, z, wi, 1e-5, 8, o), n * inner * 8),
+        "attention_prepare": (lambda i: ops.attention_prepare(qkv, 0, hq, hq + hk, h, kv, hd, hd, step, qo, kp, vp, pages, 64, cs, hd // 2, False,
+                                                              first_values=fv, value_mix=ops.VALUES_MIX, share=0.5), n * (2 * (hq + 2 * hk) + hk) * 2),
         "moe_route_chosen": (lambda i: ops.moe_route_chosen(logits, args.experts, args.top, 1.0, choice, weight, bias), n * args.experts * 4),
     }
     res = {"kernel": "bumisun_rows", "tokens": n, "width": k, "inner": inner}

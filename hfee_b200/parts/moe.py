@@ -85,7 +85,10 @@ class RoutedExperts(Part):
             # with a stride, the softmax router over all experts does not
             if self.router == "softmax":
                 raise ValueError("a gated shared expert goes with the sigmoid_groups or the softmax_chosen router")
-            self.w_router = torch.cat([tensors["router"], tensors["shared.sg"]], dim=0).contiguous()
+            # (and rows of zeros up to a multiple of eight: the products like their columns so)
+            rows = [tensors["router"], tensors["shared.sg"]]
+            pad = pad8(self.experts + 1) - self.experts - 1
+            self.w_router = torch.cat(rows + [torch.zeros_like(rows[1])] * pad, dim=0).contiguous()
         pairs = rt.max_tokens * self.top
         self.grouped = ops.moe_experts_grouped_ok(rt.dtype, self.width, self.inner)
         self.tiles = ops.moe_tiles_grouped(pairs, self.experts) if self.grouped else ops.moe_max_tiles(pairs, self.experts)
@@ -127,7 +130,7 @@ class RoutedExperts(Part):
             ops.moe_route_chosen(logits, self.experts, top, self.router_scale, choice, weight, self.router_bias)
         else:
             ops.moe_route(logits, top, self.router_scale, choice, weight)
-        gate_col = logits[:, self.experts:] if self.shared_gate else None
+        gate_col = logits[:, self.experts:self.experts + 1] if self.shared_gate else None
         place = None
         if self.grouped:
             rows = self.tiles * ops.GROUPED_TILE_ROWS

@@ -265,3 +265,44 @@ def test_head_scan_without_a_write_leaves_the_state():
         ops.head_scan(buf[:, :32], buf[:, 32:40], buf[:, 40:], z, one, -one, one, S, make_step([n], lengths=[3], slots=[1]), out, 2, 1, 8, 16,
                       False, ws)
         assert torch.equal(S, before)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("interleaved", [False, True])
+@pytest.mark.parametrize("heads,kv,dim,vdim,rope", [(4, 2, 32, 24, 16), (6, 2, 64, 16, 64), (2, 1, 16, 8, 8), (3, 3, 8, 40, 0), (2, 2, 128, 64, 32), (5, 1, 24, 16, 6)])
+def test_attention_prepare_in_whole_pieces(dtype, interleaved, heads, kv, dim, vdim, rope):
+    """Without biases and norms the preparation moves 16-byte pieces where it can; few tokens and many, over pages in any order."""
+    from hfee_b200.kernels import ops
+    rng = np.random.default_rng(heads * dim + rope)
+    qc, kc, vc = heads * dim, kv * dim, kv * vdim
+    for n, n0, page in ((1, 37, 16), (13, 21, 16), (600, 5, 64)):
+        src = dev(rng.normal(size=(n, qc + kc + vc)), dtype)
+        x = wide(src)
+        pages = -(-(n0 + n) // page)
+        order = rng.permutation(pages)
+        table = torch.full((3, pages + 1), -1, dtype=torch.int32, device=DEV)
+        table[1, :pages] = dev(order, torch.int32)
+        step = make_step([n], lengths=[n0], slots=[1])
+        cs = None
+        if rope:
+            inv = torch.tensor([300.0 ** (-2.0 * i / rope) for i in range(rope // 2)], dtype=torch.float64, device=DEV)
+            cs = torch.empty((n, rope // 2, 2), device=DEV)
+            ops.rope_table(step.positions, inv, cs)
+        kp, vp = (torch.zeros((pages, kv, page, d), dtype=dtype, device=DEV) for d in (dim, vdim))
+        q_out = torch.empty((n, qc), dtype=dtype, device=DEV)
+        ops.attention_prepare(src, 0, qc, qc + kc, heads, kv, dim, vdim, step, q_out, kp, vp, table, page, cs, rope, interleaved)
+
+        def rotated(t, h):
+            t = t.reshape(n, h, dim).copy()
+            a = (np.arange(n0, n0 + n)[:, None] * 300.0 ** (-2.0 * np.arange(rope // 2) / max(rope, 1)))[:, None, :]
+            first, second = ((slice(0, rope, 2), slice(1, rope, 2)) if interleaved else (slice(0, rope // 2), slice(rope // 2, rope)))
+            u, v = t[..., first].copy(), t[..., second].copy()
+            t[..., first], t[..., second] = u * np.cos(a) - v * np.sin(a), v * np.cos(a) + u * np.sin(a)
+            return t
+        tol = 1e-6 if dtype == torch.float32 else 5e-3
+        assert close(wide(q_out), rotated(x[:, :qc], heads).reshape(n, qc), tol)
+        at = np.arange(n0, n0 + n)
+        pg = order[at // page]
+        assert close(wide(kp)[pg, :, at % page], rotated(x[:, qc:qc + kc], kv), tol)
+        assert np.array_equal(wide(vp)[pg, :, at % page].reshape(n, vc), x[:, qc + kc:])
+        assert torch.count_nonzero(kp[int(order[0])][:, :n0 % page if n0 < page else 0]) == 0
