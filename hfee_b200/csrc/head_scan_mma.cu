@@ -24,7 +24,7 @@
 namespace {
 
 constexpr int HS_T = 64;            // tokens of a run
-constexpr int HS_WARPS = 4;         // of a block of outputs
+constexpr int HS_WARPS = 8;         // of a block of outputs
 constexpr int HS_THREADS = HS_WARPS * 32;
 constexpr int HS_COLS_STATES = 32;  // columns of x per block of the walk
 constexpr int HS_COLS_OUT = 64;     // and of the outputs
@@ -293,8 +293,9 @@ head_scan_states_kernel(HeadScanArgs p) {
 }
 
 // ------------------------------------------------------------------------------------------ (3) outputs
-// Warp w owns the run's tokens 16 w .. + 15 for C . B and the weights made of it, which meet in shared memory, and the
-// columns 16 w .. + 15 of the outputs of all of the run's tokens, so that a fragment of the state is read once per block.
+// C . B and the weights made of it: warp w has the run's tokens 16 (w & 3) .. + 15 against every second tile of 16 tokens
+// in front of them (from w >> 2 on); they meet in shared memory.  Outputs: warp w has the columns 16 (w & 3) .. + 15 of two
+// of the run's four tiles of 16 tokens, the outer ones or the inner ones (as many tiles in front of them either way).
 template <int NP> struct OutCfg {
   static constexpr int TILES = NP / 16;
   static constexpr int LDB = NP + HS_PAD, LDX = HS_COLS_OUT + HS_PAD, LDP = HS_T + HS_PAD;
@@ -304,8 +305,10 @@ template <int NP> struct OutCfg {
   static constexpr int SMEM = HS_T * LDB * 2 + SHARED + 2 * X_STAGE;
 };
 
+constexpr int HS_OUT_BLOCKS = 2;     // resident per SM
+
 template <int NP>
-__global__ void __launch_bounds__(HS_THREADS, NP <= 128 ? 3 : 2)
+__global__ void __launch_bounds__(HS_THREADS, HS_OUT_BLOCKS)
 head_scan_outputs_kernel(HeadScanArgs p) {
   using C = OutCfg<NP>;
   extern __shared__ __align__(16) unsigned char smem_raw[];
@@ -334,9 +337,11 @@ head_scan_outputs_kernel(HeadScanArgs p) {
       const bool ok = s < n && c0 + c < p.vdim;
       hs_copy16(xd + s * C::LDX + c, ok ? p.x + (long long)(begin + s) * p.ld + (long long)head * p.vdim + c0 + c : p.x, ok);
     }
-    const int s = tid % HS_T;
-    const float* src = (tid < HS_T ? p.gate_s : p.gate_dt) + (long long)head * p.n_tokens + begin;
-    hs_copy4(sd + tid, s < n ? src + s : p.gate_s, s < n);
+    if (tid < 2 * HS_T) {
+      const int s = tid % HS_T;
+      const float* src = (tid < HS_T ? p.gate_s : p.gate_dt) + (long long)head * p.n_tokens + begin;
+      hs_copy4(sd + tid, s < n ? src + s : p.gate_s, s < n);
+    }
     hs_commit();
   };
 #pragma unroll
@@ -351,35 +356,39 @@ head_scan_outputs_kernel(HeadScanArgs p) {
   hs_wait_all();
   __syncthreads();
 
-  // C . B of the warp's 16 tokens with the tokens up to the diagonal, for all heads of the block
-  const int r0 = warp * 16;
-  float cb[HS_T / 8][4];
+  // C . B, for all heads of the block
+  const int quarter = warp & 3, side = warp >> 2;
+  const int r0 = quarter * 16;
+  float cb[2][2][4];                                       // tiles side and side + 2 of 16 tokens, by 8
 #pragma unroll
-  for (int j = 0; j < HS_T / 8; ++j) cb[j][0] = cb[j][1] = cb[j][2] = cb[j][3] = 0.f;
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int q = 0; q < 2; ++q) cb[i][q][0] = cb[i][q][1] = cb[i][q][2] = cb[i][q][3] = 0.f;
 #pragma unroll
   for (int kk = 0; kk < C::TILES; ++kk) {
     uint32_t a[4];
     load_a(a, cs, C::LDB, r0, kk * 16, lane);
 #pragma unroll
-    for (int kt = 0; kt < HS_T / 16; ++kt) {
-      if (kt <= warp) {
+    for (int i = 0; i < 2; ++i) {
+      const int kt = side + 2 * i;
+      if (kt <= quarter) {
         uint32_t b[4];
         load_b_pair(b, bs, C::LDB, kt * 16, kk * 16, lane);
-        mma_bf16(cb[2 * kt], a, b[0], b[1]);
-        mma_bf16(cb[2 * kt + 1], a, b[2], b[3]);
+        mma_bf16(cb[i][0], a, b[0], b[1]);
+        mma_bf16(cb[i][1], a, b[2], b[3]);
       }
     }
   }
   __syncthreads();                                         // B is used up: its place takes the weights
-  const int ct0 = c0 / 8 + 2 * warp;                       // the warp's two tiles of 8 columns
+  const int ct0 = c0 / 8 + 2 * quarter;                    // the warp's two tiles of 8 columns
   const int cts = min(2, p.ctiles - ct0);                  // 0 or less: none of them exists
-  const int row_tiles = (n + 15) / 16;
+  const int row_tile[2] = {side, 3 - side};
   for (int hh = 0; hh < p.heads_per_block; ++hh) {
     const int head = head0 + hh, st = hh & 1;
     if (hh + 1 < p.heads_per_block) load_head(head + 1, st ^ 1);
     // the state in front of the run: requested before the weights are computed
     const uint4* S = p.carried + ((long long)(blockIdx.x) * p.heads + head) * (C::TILES * p.ctiles * 32) + ct0 * 32 + lane;
-    constexpr int AHEAD = C::TILES < 8 ? C::TILES : 8;
+    constexpr int AHEAD = C::TILES < 4 ? C::TILES : 4;
     uint4 f[AHEAD][2];
 #pragma unroll
     for (int kk = 0; kk < AHEAD; ++kk)
@@ -392,38 +401,42 @@ head_scan_outputs_kernel(HeadScanArgs p) {
     // weights e^(s_t - s_u) dt_u (C_t . B_u)
     const float s_lo = ss[r0 + g], s_hi = ss[r0 + g + 8];
 #pragma unroll
-    for (int q = 0; q < HS_T / 8; ++q) {
-      if (q < 2 * (warp + 1)) {
-        const int u = q * 8 + 2 * t;
-        const float2 su = *reinterpret_cast<const float2*>(ss + u), du = *reinterpret_cast<const float2*>(sdt + u);
-        const int lo_row = r0 + g, hi_row = r0 + g + 8;
-        const float w0 = u <= lo_row ? cb[q][0] * (hs_exp2(s_lo - su.x) * du.x) : 0.f;
-        const float w1 = u + 1 <= lo_row ? cb[q][1] * (hs_exp2(s_lo - su.y) * du.y) : 0.f;
-        const float w2 = u <= hi_row ? cb[q][2] * (hs_exp2(s_hi - su.x) * du.x) : 0.f;
-        const float w3 = u + 1 <= hi_row ? cb[q][3] * (hs_exp2(s_hi - su.y) * du.y) : 0.f;
-        uint32_t hi, lo;
-        split_pair(w0, w1, hi, lo);
-        *reinterpret_cast<uint32_t*>(w_hi + lo_row * C::LDP + u) = hi;
-        *reinterpret_cast<uint32_t*>(w_lo + lo_row * C::LDP + u) = lo;
-        split_pair(w2, w3, hi, lo);
-        *reinterpret_cast<uint32_t*>(w_hi + hi_row * C::LDP + u) = hi;
-        *reinterpret_cast<uint32_t*>(w_lo + hi_row * C::LDP + u) = lo;
+    for (int i = 0; i < 2; ++i) {
+      const int kt = side + 2 * i;
+      if (kt <= quarter) {
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          const int u = kt * 16 + q * 8 + 2 * t;
+          const float2 su = *reinterpret_cast<const float2*>(ss + u), du = *reinterpret_cast<const float2*>(sdt + u);
+          const int lo_row = r0 + g, hi_row = r0 + g + 8;
+          const float w0 = u <= lo_row ? cb[i][q][0] * (hs_exp2(s_lo - su.x) * du.x) : 0.f;
+          const float w1 = u + 1 <= lo_row ? cb[i][q][1] * (hs_exp2(s_lo - su.y) * du.y) : 0.f;
+          const float w2 = u <= hi_row ? cb[i][q][2] * (hs_exp2(s_hi - su.x) * du.x) : 0.f;
+          const float w3 = u + 1 <= hi_row ? cb[i][q][3] * (hs_exp2(s_hi - su.y) * du.y) : 0.f;
+          uint32_t hi, lo;
+          split_pair(w0, w1, hi, lo);
+          *reinterpret_cast<uint32_t*>(w_hi + lo_row * C::LDP + u) = hi;
+          *reinterpret_cast<uint32_t*>(w_lo + lo_row * C::LDP + u) = lo;
+          split_pair(w2, w3, hi, lo);
+          *reinterpret_cast<uint32_t*>(w_hi + hi_row * C::LDP + u) = hi;
+          *reinterpret_cast<uint32_t*>(w_lo + hi_row * C::LDP + u) = lo;
+        }
       }
     }
     __syncthreads();
     if (cts > 0) {
-      float acc[HS_T / 16][2][4];
+      float acc[2][2][4];
 #pragma unroll
-      for (int r = 0; r < HS_T / 16; ++r)
+      for (int r = 0; r < 2; ++r)
 #pragma unroll
         for (int j = 0; j < 2; ++j) acc[r][j][0] = acc[r][j][1] = acc[r][j][2] = acc[r][j][3] = 0.f;
       // what the state in front of the run gives
 #pragma unroll
       for (int kk = 0; kk < C::TILES; ++kk) {
 #pragma unroll
-        for (int r = 0; r < HS_T / 16; ++r) {
+        for (int r = 0; r < 2; ++r) {
           uint32_t a[4];
-          load_a(a, cs, C::LDB, r * 16, kk * 16, lane);
+          load_a(a, cs, C::LDB, row_tile[r] * 16, kk * 16, lane);
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
             mma_bf16(acc[r][j], a, f[kk % AHEAD][j].x, f[kk % AHEAD][j].y);
@@ -437,21 +450,23 @@ head_scan_outputs_kernel(HeadScanArgs p) {
         }
       }
 #pragma unroll
-      for (int r = 0; r < HS_T / 16; ++r) {
-        const float e_lo = hs_exp2(ss[r * 16 + g]), e_hi = hs_exp2(ss[r * 16 + g + 8]);
+      for (int r = 0; r < 2; ++r) {
+        const float e_lo = hs_exp2(ss[row_tile[r] * 16 + g]), e_hi = hs_exp2(ss[row_tile[r] * 16 + g + 8]);
 #pragma unroll
         for (int j = 0; j < 2; ++j) { acc[r][j][0] *= e_lo; acc[r][j][1] *= e_lo; acc[r][j][2] *= e_hi; acc[r][j][3] *= e_hi; }
       }
       // what the run's own tokens give
 #pragma unroll
       for (int kt = 0; kt < HS_T / 16; ++kt) {
+        if (kt > row_tile[1]) continue;                    // row_tile[1] is the later of the two
         uint32_t b[4];
-        load_b_pair_trans(b, xs, C::LDX, warp * 16, kt * 16, lane);
+        load_b_pair_trans(b, xs, C::LDX, quarter * 16, kt * 16, lane);
 #pragma unroll
-        for (int r = kt; r < HS_T / 16; ++r) {
+        for (int r = 0; r < 2; ++r) {
+          if (kt > row_tile[r]) continue;
           uint32_t ah[4], al[4];
-          load_a(ah, w_hi, C::LDP, r * 16, kt * 16, lane);
-          load_a(al, w_lo, C::LDP, r * 16, kt * 16, lane);
+          load_a(ah, w_hi, C::LDP, row_tile[r] * 16, kt * 16, lane);
+          load_a(al, w_lo, C::LDP, row_tile[r] * 16, kt * 16, lane);
           mma_bf16(acc[r][0], ah, b[0], b[1]);
           mma_bf16(acc[r][1], ah, b[2], b[3]);
           mma_bf16(acc[r][0], al, b[0], b[1]);
@@ -460,15 +475,14 @@ head_scan_outputs_kernel(HeadScanArgs p) {
       }
       const float skip = p.d_skip[head];
 #pragma unroll
-      for (int r = 0; r < HS_T / 16; ++r) {
-        if (r >= row_tiles) continue;
+      for (int r = 0; r < 2; ++r) {
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           if (j >= cts) continue;
-          const int x_col = warp * 16 + j * 8 + 2 * t, c = c0 + x_col;
+          const int x_col = quarter * 16 + j * 8 + 2 * t, c = c0 + x_col;
 #pragma unroll
           for (int half = 0; half < 2; ++half) {
-            const int row = r * 16 + g + 8 * half;
+            const int row = row_tile[r] * 16 + g + 8 * half;
             if (row >= n) continue;
             const __nv_bfloat162 xv = *reinterpret_cast<const __nv_bfloat162*>(xs + row * C::LDX + x_col);
             *reinterpret_cast<float2*>(p.out + (long long)(begin + row) * p.ld_o + (long long)head * p.vdim + c) =
@@ -503,7 +517,7 @@ int launch_head_scan(HeadScanArgs p, int max_runs, cudaStream_t stream) {
   const int tiles = (p.vdim + HS_COLS_OUT - 1) / HS_COLS_OUT;
   // Several heads of a group per block share its C . B, if the blocks still fill the GPU well: about one head's work for the
   // shared part and one for each head, times the rounds that the blocks make.
-  const long long slots = (NP <= 128 ? 3 : 2) * (long long)hfee_sm_count();
+  const long long slots = HS_OUT_BLOCKS * (long long)hfee_sm_count();
   long long best = 0;
   for (int h : {1, 2, 4}) {
     if ((p.heads / p.groups) % h != 0) continue;
